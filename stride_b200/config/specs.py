@@ -102,7 +102,8 @@ class LayerSpec:
     """kind ``pre_norm``: x += m * mixer(norm(x)); x += m * ffn(norm(x)); then every part of ``after`` adds
     m * part(x, tokens). ``residual_mult`` is m (1 where an architecture has none); ``feed_forward`` and
     ``ffn_norm`` may be None for a layer without a feed-forward. kind ``sandwich`` has a second norm on either
-    sublayer's output (``mixer_out_norm``, ``ffn_out_norm``): x += m * out_norm(mixer(norm(x)))."""
+    sublayer's output (``mixer_out_norm``, ``ffn_out_norm``): x += m * out_norm(mixer(norm(x))). kind ``copies`` runs on a
+    residual stream in several copies (``ModelSpec.copies``; see ``parts/copies.py`` for its ``params``)."""
     kind: str
     mixer: MixerSpec
     feed_forward: Optional[FeedForwardSpec]
@@ -112,6 +113,7 @@ class LayerSpec:
     after: tuple = ()           # of StreamInputSpec
     mixer_out_norm: Optional[NormSpec] = None
     ffn_out_norm: Optional[NormSpec] = None
+    params: tuple = ()          # free-form (key, value) pairs of an arrangement
 
 
 @dataclass(frozen=True)
@@ -181,6 +183,7 @@ class ModelSpec:
     embedding: Optional[EmbeddingSpec] = None
     head: Optional[HeadSpec] = None
     pass_input: Optional[PassInputSpec] = None      # for schedules whose entries name ``enters_pass``
+    copies: int = 0                                 # the residual stream is kept in this many copies (layers of kind ``copies``); 0: it is one
 
     def embedding_spec(self) -> EmbeddingSpec:
         return self.embedding or EmbeddingSpec("lookup", self.vocab, self.hidden, self.embed_name)

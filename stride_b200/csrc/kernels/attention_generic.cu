@@ -16,7 +16,8 @@
 // learned number whose exponential joins the softmax's denominator (it has no key and no value and is not scaled): it
 // enters the running maximum and sum after the last group of keys, so the order of the sums stays a function of p.
 // Values may be narrower or wider than keys (`vd` beside `hd`), and a head may take a penalty off a score in proportion
-// to the key's distance: s <- s - slope_h (p - j), the slopes given per query head.
+// to the key's distance: s <- s - slope_h (p - j), the slopes given per query head, or gain a learned number that depends on
+// the distance: s <- s + rel[h, min(p - j, rel_len - 1)] (a table per query head whose last entry serves all farther keys).
 #include "common.cuh"
 
 namespace stride {
@@ -70,7 +71,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restr
                                const T* __restrict__ v_pages, const int32_t* __restrict__ block_table, int table_width,
                                const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ positions, int nq,
                                int nkv, int hd, int vd, int page_size, float scale, int window, float softcap,
-                               const float* __restrict__ sinks, const float* __restrict__ slopes) {
+                               const float* __restrict__ sinks, const float* __restrict__ slopes, const float* __restrict__ rel, int rel_len) {
     pdl_trigger();
     pdl_wait();
     __shared__ __align__(16) float q_smem[kWarps][kMaxHeadDim];
@@ -110,6 +111,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restr
             s = dot_row<T>(qs, k_row, hd) * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
             if (slopes) s = __fadd_rn(s, -__fmul_rn(slope, static_cast<float>(pos - key)));
+            if (rel) s = __fadd_rn(s, rel[static_cast<size_t>(head) * rel_len + min(pos - key, rel_len - 1)]);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float p = ok ? expf(s - m_new) : 0.f;
@@ -159,8 +161,9 @@ extern "C" int stride_paged_attention_generic(const void* q, int q_stride, void*
                                               const int32_t* block_table, int table_width, const int32_t* seq_of_token,
                                               const int32_t* positions, int tokens, int nq, int nkv, int hd, int vd, int page_size,
                                               float scale, int window, float softcap, const float* sinks, const float* slopes,
-                                              int dtype, cudaStream_t stream) {
-    if (tokens < 0 || nq <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || softcap < 0.f) return STRIDE_BAD_ARGUMENT;
+                                              const float* rel, int rel_len, int dtype, cudaStream_t stream) {
+    if (tokens < 0 || nq <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || softcap < 0.f ||
+        (rel && rel_len <= 0)) return STRIDE_BAD_ARGUMENT;
     if (nq % nkv) return STRIDE_BAD_ARGUMENT;
     if (hd > kMaxHeadDim || vd > kMaxHeadDim) return STRIDE_UNSUPPORTED;
     if (tokens == 0) return 0;
@@ -168,12 +171,12 @@ extern "C" int stride_paged_attention_generic(const void* q, int q_stride, void*
     if (dtype == STRIDE_DTYPE_F32)
         stride::launch(paged_attention_generic_kernel<float>, dim3(grid), dim3(kWarps * 32), 0, stream, 
             static_cast<const float*>(q), q_stride, static_cast<float*>(out), static_cast<const float*>(k_pages),
-            static_cast<const float*>(v_pages), block_table, table_width, seq_of_token, positions, nq, nkv, hd, vd, page_size, scale, window, softcap, sinks, slopes);
+            static_cast<const float*>(v_pages), block_table, table_width, seq_of_token, positions, nq, nkv, hd, vd, page_size, scale, window, softcap, sinks, slopes, rel, rel_len);
     else if (dtype == STRIDE_DTYPE_BF16)
         stride::launch(paged_attention_generic_kernel<__nv_bfloat16>, dim3(grid), dim3(kWarps * 32), 0, stream, 
             static_cast<const __nv_bfloat16*>(q), q_stride, static_cast<__nv_bfloat16*>(out),
             static_cast<const __nv_bfloat16*>(k_pages), static_cast<const __nv_bfloat16*>(v_pages), block_table, table_width,
-            seq_of_token, positions, nq, nkv, hd, vd, page_size, scale, window, softcap, sinks, slopes);
+            seq_of_token, positions, nq, nkv, hd, vd, page_size, scale, window, softcap, sinks, slopes, rel, rel_len);
     else
         return STRIDE_BAD_ARGUMENT;
     return STRIDE_LAUNCH_STATUS();

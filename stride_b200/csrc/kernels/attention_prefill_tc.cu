@@ -59,7 +59,8 @@ constexpr long long kStaggerCycles = 1000;
 // HEADS query heads of one key head per CTA (1 or 2). One head: 4 service warps (keys, products, values, Q) and 4
 // softmax warps, two CTAs per SM. Two heads: 8 service warps (three for keys, products, three for values, Q) and
 // 8 softmax warps, one CTA per SM: a single warp cannot issue a tile's copies as fast as two heads consume them.
-template <int HD, int HEADS, bool TMA_KV>
+// REL: with a table of learned numbers per head and distance.
+template <int HD, int HEADS, bool TMA_KV, bool REL>
 __global__ void __launch_bounds__(HEADS == 1 ? 256 : 512, HEADS == 1 ? 2 : 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const __nv_bfloat16* __restrict__ k_pages,
@@ -67,7 +68,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const int32_t* __restrict__ block_table, int table_width, const int32_t* __restrict__ q_start,
                        const int32_t* __restrict__ q_len, const int32_t* __restrict__ ctx_len, int num_seqs, int nq, int nkv,
                        int page_shift, float scale_log2e, int window, float cap_in, const float* __restrict__ sinks,
-                       const float* __restrict__ slopes, int* __restrict__ status) {
+                       const float* __restrict__ slopes, const float* __restrict__ rel, int rel_len, int* __restrict__ status) {
     constexpr int HALVES = HD / 64;                       // 64-column boxes per row
     constexpr int HALF_BYTES = kQRows * 128;              // a [128 rows x 64 columns] bf16 box of Q
     constexpr int KV_HALF_BYTES = kKeys * 128;            // [64 keys x 64 columns] of K or V
@@ -307,6 +308,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         float m_ref = -INFINITY, l = 0.f;                    // m_ref in log2 units (scaled scores)
         // A penalty on the key's distance, slope (pos - key), in the units of the raw scores (which scale_log2e multiplies).
         const float slope_raw = slopes != nullptr ? slopes[head] * 1.4426950408889634f / scale_log2e : 0.f;
+        // A learned number per head and distance, from a table whose last entry serves all farther keys: added to the raw
+        // scores in their units. A tile all of whose (row, key) pairs lie that far costs one addition a score.
+        const float rel_unit = 1.4426950408889634f / scale_log2e;
+        const float* rel_h = REL ? rel + static_cast<size_t>(head) * rel_len : nullptr;
+        const float rel_far = REL ? rel_h[rel_len - 1] * rel_unit : 0.f;
         // The output product of tile x has finished when phase x / 2 of s_free[x & 1] has: the phase before it
         // (tile x - 2) is known to be over whenever this is asked, because the scores of tile x could only be issued
         // after it, so the parity cannot be mistaken.
@@ -338,6 +344,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 const float d0 = static_cast<float>(k0 - pos_r);
 #pragma unroll
                 for (int i = 0; i < 64; ++i) sv[i] = fmaf(slope_raw, d0 + static_cast<float>(i), sv[i]);
+            }
+            if (REL) {
+                if (pos0 - (k0 + kKeys - 1) >= rel_len - 1) {
+#pragma unroll
+                    for (int i = 0; i < 64; ++i) sv[i] += rel_far;
+                } else {
+                    const int n0 = pos_r - k0;
+#pragma unroll
+                    for (int i = 0; i < 64; ++i) sv[i] = fmaf(__ldg(rel_h + max(0, min(n0 - i, rel_len - 1))), rel_unit, sv[i]);
+                }
             }
             if (edge) {
 #pragma unroll
@@ -456,27 +472,31 @@ template <int HD, int HEADS>
 int launch_attn(const CUtensorMap* map_q, const CUtensorMap* map_k, const CUtensorMap* map_v, const __nv_bfloat16* k_pages, const __nv_bfloat16* v_pages, __nv_bfloat16* out,
                 const int32_t* block_table, int table_width, const int32_t* q_start, const int32_t* q_len, const int32_t* ctx_len,
                 int num_seqs, int max_tiles, int nq, int nkv, int page_shift, float scale, int window, float softcap,
-                const float* sinks, const float* slopes, int* status, cudaStream_t stream) {
+                const float* sinks, const float* slopes, const float* rel, int rel_len, int* status, cudaStream_t stream) {
     constexpr int stages = HEADS == 1 ? 2 : 4;
     constexpr int smem = (HD / 64) * (HEADS * kQRows * 128 + 2 * stages * kKeys * 128) + 1024;      // Q tiles, key ring, value ring
     static bool configured[64] = {};        // the shared-memory limit is set per kernel and device
     int device = 0;
     if (cudaGetDevice(&device) != cudaSuccess || device < 0 || device >= 64) return STRIDE_BAD_ARGUMENT;
     if (!configured[device]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, HEADS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, HEADS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e != cudaSuccess) return static_cast<int>(e);
+        const void* kernels[4] = {reinterpret_cast<const void*>(attn_prefill_tc_kernel<HD, HEADS, true, false>),
+                                  reinterpret_cast<const void*>(attn_prefill_tc_kernel<HD, HEADS, false, false>),
+                                  reinterpret_cast<const void*>(attn_prefill_tc_kernel<HD, HEADS, true, true>),
+                                  reinterpret_cast<const void*>(attn_prefill_tc_kernel<HD, HEADS, false, true>)};
+        for (const void* k : kernels) {
+            const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+            if (e != cudaSuccess) return static_cast<int>(e);
+        }
         configured[device] = true;
     }
     const dim3 grid(nq / HEADS, max_tiles), block(HEADS == 1 ? 256 : 512);
-    if (map_k != nullptr && map_v != nullptr)
-        stride::launch(attn_prefill_tc_kernel<HD, HEADS, true>, grid, block, smem, stream, *map_q, *map_k, *map_v, k_pages, v_pages, out,
-                       block_table, table_width, q_start, q_len, ctx_len, num_seqs, nq, nkv, page_shift,
-                       (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes, status);
-    else
-        stride::launch(attn_prefill_tc_kernel<HD, HEADS, false>, grid, block, smem, stream, *map_q, *map_q, *map_q, k_pages, v_pages, out,
-                       block_table, table_width, q_start, q_len, ctx_len, num_seqs, nq, nkv, page_shift,
-                       (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes, status);
+    const bool tma = map_k != nullptr && map_v != nullptr;
+    const auto kernel = rel != nullptr ? (tma ? attn_prefill_tc_kernel<HD, HEADS, true, true> : attn_prefill_tc_kernel<HD, HEADS, false, true>)
+                                       : (tma ? attn_prefill_tc_kernel<HD, HEADS, true, false> : attn_prefill_tc_kernel<HD, HEADS, false, false>);
+    stride::launch(kernel, grid, block, smem, stream, *map_q, tma ? *map_k : *map_q, tma ? *map_v : *map_q, k_pages, v_pages, out,
+                   block_table, table_width, q_start, q_len, ctx_len, num_seqs, nq, nkv, page_shift,
+                   (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes, rel,
+                   rel_len, status);
     return STRIDE_LAUNCH_STATUS();
 }
 
@@ -509,15 +529,17 @@ static bool kv_tma() {
 // than 64 and 128, page sizes that are no power of two from 4 to 64, unaligned strides); the caller
 // then uses the mma.sync kernel. softcap c > 0 caps the scaled scores at c tanh(s / c) (with the hardware's tanh); sinks
 // (float32 [nq] or null) adds exp(sink) of the head to the softmax's denominator; slopes (float32 [nq] or null) takes
-// slope_h times the key's distance off every score of head h.
+// slope_h times the key's distance off every score of head h; rel (float32 [nq, rel_len] or null) adds rel[h, min(distance,
+// rel_len - 1)] to every score of head h.
 extern "C" int stride_paged_prefill_attention_tc(const void* q, int q_stride, void* out, const void* k_pages, const void* v_pages,
                                                  int num_pages, const int32_t* block_table, int table_width,
                                                  const int32_t* q_start, const int32_t* q_len, const int32_t* ctx_len,
                                                  int num_seqs, int tokens, int nq, int nkv, int hd, int page_size, float scale,
-                                                 int window, float softcap, const float* sinks, const float* slopes, int* status,
+                                                 int window, float softcap, const float* sinks, const float* slopes, const float* rel,
+                                                 int rel_len, int* status,
                                                  cudaStream_t stream) {
     if (tokens < 0 || num_seqs < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || num_pages <= 0 ||
-        softcap < 0.f)
+        softcap < 0.f || (rel && rel_len <= 0))
         return STRIDE_BAD_ARGUMENT;
     if (nq % nkv || status == nullptr) return STRIDE_BAD_ARGUMENT;
     if ((hd != 64 && hd != 128) || page_size > tc::kKeys || page_size < 4 || q_stride % 8 || nq > 65535) return STRIDE_UNSUPPORTED;
@@ -549,7 +571,7 @@ extern "C" int stride_paged_prefill_attention_tc(const void* q, int q_stride, vo
     }
 #define STRIDE_ATTN_LAUNCH(HD_, HEADS_)                                                                                          \
     tc::launch_attn<HD_, HEADS_>(map_q, map_k, map_v, kp, vp, op, block_table, table_width, q_start, q_len, ctx_len, num_seqs, max_tiles, nq, \
-                                 nkv, page_shift, scale, window, softcap, sinks, slopes, status, stream)
+                                 nkv, page_shift, scale, window, softcap, sinks, slopes, rel, rel_len, status, stream)
     if (hd == 64) return pair ? STRIDE_ATTN_LAUNCH(64, 2) : STRIDE_ATTN_LAUNCH(64, 1);
     return pair ? STRIDE_ATTN_LAUNCH(128, 2) : STRIDE_ATTN_LAUNCH(128, 1);
 #undef STRIDE_ATTN_LAUNCH

@@ -1,0 +1,448 @@
+// Linear attention with a fading memory: per head a matrix S [D, DV] in float32 from zero and, per token,
+//
+//   channel decays     S <- diag(alpha_t) S + k v^T ;  o = S^T (q D^-1/2),  alpha_t = sigmoid(z_t + b)^(1 / tau) per key channel
+//                      (Yang et al., "Gated Linear Attention Transformers with Hardware-Efficient Training")
+//   constant decay     S <- decay_h S + silu(k) silu(v)^T ;  o = S^T silu(q)
+//                      (Qin et al., "Lightning Attention-2: A Free Lunch for Handling Unlimited Sequence Lengths in Large
+//                      Language Models")
+//
+// Two forms of the same recurrence:
+//
+//   decay_scan    one token after the other (memory_scan.cuh): decoding, short portions, and the whole 32-bit path, where a
+//                 token's output must not depend on how its prompt was cut.
+//   decay_chunks  long portions, chunks of 64 tokens side by side. With g_t the running product of decays inside a chunk (from
+//                 its first token on, so g <= 1), G the chunk's whole product and S_c the memory before the chunk:
+//                     o_i = (q_i g_i)^T S_c + sum_{j <= i} ((q_i g_i) . (k_j / g_j)) v_j
+//                     S_(c+1) = G S_c + sum_j (k_j G / g_j) v_j^T
+//                 Four launches: the running logarithms of the decays (channel decays only), every chunk's own sum, the
+//                 memories at the chunks' starts (memory_scan.cuh: pieces_combine), the outputs. All of it in float32 on the FMA
+//                 pipe (the memory, the decays and what enters them are float32 by the designs' own rule, so the tensor cores,
+//                 which would round the operands, are left out), as register-tiled products from shared memory.
+//                 1 / g_j can overflow where a channel forgets nearly everything within a chunk: a CTA whose chunk has a
+//                 channel with g below e^-60 forms its scores with exp(log g_i - log g_j) per channel instead, which only
+//                 costs time. A constant decay never divides: decay^(i - j) is taken from a table of powers.
+#include "memory_scan.cuh"
+
+namespace stride {
+
+constexpr int kChunk = 64;              // tokens a chunk
+constexpr int kChunkCols = 128;         // columns of S a CTA works on
+constexpr int kChunkThreads = 256;
+constexpr int kLd = kChunk + 4;         // row stride of the transposed tiles: 16-byte reads, stores without bank conflicts
+constexpr float kSafeLog = -60.f;
+
+struct ChunkArgs {
+    const void* q;          // [tokens, ld], head h at column h * D
+    const void* k;
+    const void* v;          // head h at column h * DV
+    int ld, in_bf16;
+    float* cum;             // channel decays: [tokens, H * D], the running logarithm of the decays inside the chunk
+    const float* bias;      // channel decays: [H * D]
+    const float* powers;    // constant decay: [H, kChunk + 1], decay^n
+    float q_scale, inv_tau;
+    float* o;               // [tokens, H * DV]
+    float* piece_s;         // [seqs * max_pieces, H, D, DV]
+    float* piece_p;         // [seqs * max_pieces, H, D]
+    const int32_t* q_start;
+    const int32_t* q_len;
+    int H, D, DV, max_pieces;
+};
+
+// z -> running sums of log(sigmoid(z + b)) / tau over the chunk's tokens, in place. One thread a (head, channel).
+static __global__ void __launch_bounds__(128)
+chunk_decay_kernel(const ChunkArgs p) {
+    pdl_trigger();
+    pdl_wait();
+    const int z = blockIdx.y, seq = z / p.max_pieces, first = (z % p.max_pieces) * kChunk;
+    const int nt = min(p.q_len[seq] - first, kChunk);
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, HD = p.H * p.D;
+    if (nt <= 0 || c >= HD) return;
+    float* at = p.cum + static_cast<size_t>(p.q_start[seq] + first) * HD + c;
+    const float b = p.bias[c];
+    float sum = 0.f;
+    for (int t0 = 0; t0 < nt; t0 += 8) {
+        float l[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) l[u] = t0 + u < nt ? at[static_cast<size_t>(t0 + u) * HD] : 0.f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) l[u] = log_sigmoid_f(l[u] + b) * p.inv_tau;
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (t0 + u < nt) {
+                sum += l[u];
+                at[static_cast<size_t>(t0 + u) * HD] = sum;
+            }
+    }
+}
+
+// piece_s[z, h] = sum_j (k_j G / g_j) v_j^T, piece_p[z, h] = G. DP: D padded. Grid (column tiles, heads, chunks).
+template <int DP, int RULE>
+__global__ void __launch_bounds__(kChunkThreads)
+chunk_sum_kernel(const ChunkArgs p) {
+    constexpr int PASS_ROWS = DP < 128 ? DP : 128, R = PASS_ROWS / 8;       // rows of S a warp holds at a time
+    extern __shared__ __align__(16) float smem[];
+    float* ks = smem;                       // [kChunk][DP]
+    float* vs = smem + kChunk * DP;         // [kChunk][kChunkCols]
+    pdl_trigger();
+    const int z = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * kChunkCols;
+    const int seq = z / p.max_pieces, first = (z % p.max_pieces) * kChunk;
+    const int nt = min(p.q_len[seq] - first, kChunk);
+    if (nt <= 0) return;
+    pdl_wait();
+    const int D = p.D, DV = p.DV, HD = p.H * D;
+    const size_t row0 = static_cast<size_t>(p.q_start[seq] + first);
+    const float* powers = RULE == kConstantDecay ? p.powers + h * (kChunk + 1) : nullptr;
+    for (int idx = threadIdx.x; idx < nt * DP; idx += kChunkThreads) {
+        const int j = idx / DP, d = idx - j * DP;
+        float k = 0.f;
+        if (d < D) {
+            k = load_any(p.k, (row0 + j) * p.ld + h * D + d, p.in_bf16);
+            if (RULE == kConstantDecay) {
+                k = silu_f(k) * powers[nt - 1 - j];
+            } else {
+                const float* cum = p.cum + row0 * HD + h * D + d;
+                k *= expf(cum[static_cast<size_t>(nt - 1) * HD] - cum[static_cast<size_t>(j) * HD]);
+            }
+        }
+        ks[idx] = k;
+    }
+    for (int idx = threadIdx.x; idx < nt * kChunkCols; idx += kChunkThreads) {
+        const int j = idx / kChunkCols, c = idx - j * kChunkCols;
+        float v = 0.f;
+        if (col0 + c < DV) {
+            v = load_any(p.v, (row0 + j) * p.ld + h * DV + col0 + c, p.in_bf16);
+            if (RULE == kConstantDecay) v = silu_f(v);
+        }
+        vs[idx] = v;
+    }
+    if (blockIdx.x == 0)
+        for (int d = threadIdx.x; d < D; d += kChunkThreads)
+            p.piece_p[(static_cast<size_t>(z) * p.H + h) * D + d] =
+                RULE == kConstantDecay ? powers[nt] : expf(p.cum[(row0 + nt - 1) * HD + h * D + d]);
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* out = p.piece_s + (static_cast<size_t>(z) * p.H + h) * D * DV;
+    for (int pass = 0; pass < DP / PASS_ROWS; ++pass) {
+        const int r0 = pass * PASS_ROWS + warp * R;
+        float acc[R][4];
+#pragma unroll
+        for (int r = 0; r < R; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+#pragma unroll 2
+        for (int j = 0; j < nt; ++j) {
+            const float4 b = *reinterpret_cast<const float4*>(vs + j * kChunkCols + 4 * lane);
+#pragma unroll
+            for (int r = 0; r < R; r += 4) {
+                const float4 a4 = *reinterpret_cast<const float4*>(ks + j * DP + r0 + r);
+                const float a[4] = {a4.x, a4.y, a4.z, a4.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    acc[r + e][0] = fmaf(a[e], b.x, acc[r + e][0]);
+                    acc[r + e][1] = fmaf(a[e], b.y, acc[r + e][1]);
+                    acc[r + e][2] = fmaf(a[e], b.z, acc[r + e][2]);
+                    acc[r + e][3] = fmaf(a[e], b.w, acc[r + e][3]);
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r0 + r >= D) continue;
+            float* dst = out + static_cast<size_t>(r0 + r) * DV + col0 + 4 * lane;
+            if (DV % 4 == 0) {
+                if (col0 + 4 * lane < DV) *reinterpret_cast<float4*>(dst) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (col0 + 4 * lane + e < DV) dst[e] = acc[r][e];
+            }
+        }
+    }
+}
+
+// Outputs of a chunk from the memory at its start (piece_s by now). Grid as above.
+template <int DP>
+constexpr int chunk_out_floats() {
+    return DP * kLd + (DP * kLd > kChunk * kChunkCols ? DP * kLd : kChunk * kChunkCols) + kChunk * kLd;
+}
+
+template <int DP, int RULE>
+__global__ void __launch_bounds__(kChunkThreads)
+chunk_out_kernel(const ChunkArgs p) {
+    constexpr int SECOND = DP * kLd > kChunk * kChunkCols ? DP * kLd : kChunk * kChunkCols;
+    constexpr int SLAB = DP * kLd / kChunkCols < DP / 2 ? DP / 4 : DP / 2;      // rows of S staged at a time
+    extern __shared__ __align__(16) float smem[];
+    float* qT = smem;                       // [DP][kLd]: column i is token i's query (times g_i)
+    float* kT = qT + DP * kLd;              // [DP][kLd]; later slabs of S [SLAB][kChunkCols], then the values [kChunk][kChunkCols]
+    float* aT = kT + SECOND;                // [kChunk j][kLd i]: scores
+    pdl_trigger();
+    const int z = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * kChunkCols;
+    const int seq = z / p.max_pieces, first = (z % p.max_pieces) * kChunk;
+    const int nt = min(p.q_len[seq] - first, kChunk);
+    if (nt <= 0) return;
+    pdl_wait();
+    const int D = p.D, DV = p.DV, HD = p.H * D;
+    const size_t row0 = static_cast<size_t>(p.q_start[seq] + first);
+    const float* powers = RULE == kConstantDecay ? p.powers + h * (kChunk + 1) : nullptr;
+    const float* cum = RULE == kChannelDecay ? p.cum + row0 * HD + h * D : nullptr;
+    bool safe = true;
+    if (RULE == kChannelDecay) {
+        int low = 0;
+        for (int d = threadIdx.x; d < D; d += kChunkThreads) low |= cum[static_cast<size_t>(nt - 1) * HD + d] < kSafeLog;
+        safe = !__syncthreads_or(low);
+    }
+    // lanes of a warp: 8 neighbouring channels of 4 neighbouring tokens, so that the transposed stores hit 32 banks
+    for (int idx = threadIdx.x; idx < kChunk * DP; idx += kChunkThreads) {
+        const int sub = idx & 31, blk = idx >> 5;
+        const int d = (blk % (DP / 8)) * 8 + (sub & 7), i = (blk / (DP / 8)) * 4 + (sub >> 3);
+        float q = 0.f, k = 0.f;
+        if (d < D && i < nt) {
+            const size_t at = (row0 + i) * p.ld + h * D + d;
+            q = load_any(p.q, at, p.in_bf16);
+            k = load_any(p.k, at, p.in_bf16);
+            if (RULE == kConstantDecay) {
+                q = silu_f(q);
+                k = silu_f(k);
+            } else {
+                q *= p.q_scale;
+                if (safe) {
+                    const float c = cum[static_cast<size_t>(i) * HD + d];
+                    q *= expf(c);
+                    k *= expf(-c);
+                }
+            }
+        }
+        qT[d * kLd + i] = q;
+        kT[d * kLd + i] = k;
+    }
+    __syncthreads();
+    {   // scores: thread (ty, tx) tokens i = 4 ty .. + 3 against j = 4 tx .. + 3
+        const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+        float a[4][4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e][0] = a[e][1] = a[e][2] = a[e][3] = 0.f;
+        if (RULE == kConstantDecay || safe) {
+            if (tx <= ty) {
+#pragma unroll 4
+                for (int d = 0; d < DP; ++d) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(qT + d * kLd + 4 * ty);
+                    const float4 k4 = *reinterpret_cast<const float4*>(kT + d * kLd + 4 * tx);
+                    const float qv[4] = {q4.x, q4.y, q4.z, q4.w}, kv[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+#pragma unroll
+                        for (int f = 0; f < 4; ++f) a[e][f] = fmaf(qv[e], kv[f], a[e][f]);
+                }
+            }
+        } else if (tx <= ty) {
+            for (int d = 0; d < D; ++d) {
+                float ci[4], cj[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    ci[e] = 4 * ty + e < nt ? cum[static_cast<size_t>(4 * ty + e) * HD + d] : 0.f;
+                    cj[e] = 4 * tx + e < nt ? cum[static_cast<size_t>(4 * tx + e) * HD + d] : 0.f;
+                }
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+#pragma unroll
+                    for (int f = 0; f < 4; ++f)
+                        if (4 * tx + f <= 4 * ty + e) a[e][f] = fmaf(qT[d * kLd + 4 * ty + e] * expf(ci[e] - cj[f]), kT[d * kLd + 4 * tx + f], a[e][f]);
+            }
+        }
+#pragma unroll
+        for (int f = 0; f < 4; ++f) {
+            float w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int n = 4 * ty + e - (4 * tx + f);
+                w[e] = n < 0 ? 0.f : RULE == kConstantDecay ? a[e][f] * powers[n] : a[e][f];
+            }
+            *reinterpret_cast<float4*>(aT + (4 * tx + f) * kLd + 4 * ty) = make_float4(w[0], w[1], w[2], w[3]);
+        }
+    }
+    __syncthreads();
+    if (RULE == kChannelDecay && !safe) {
+        for (int idx = threadIdx.x; idx < kChunk * DP; idx += kChunkThreads) {
+            const int sub = idx & 31, blk = idx >> 5;
+            const int d = (blk % (DP / 8)) * 8 + (sub & 7), i = (blk / (DP / 8)) * 4 + (sub >> 3);
+            if (d < D && i < nt) qT[d * kLd + i] *= expf(cum[static_cast<size_t>(i) * HD + d]);
+        }
+    }
+    // outputs: warp w tokens 8 w .. + 7, lane columns 4 lane .. + 3
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float acc[8][4];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+    auto step = [&](const float* a_row, const float* b_row) {
+        const float4 lo = *reinterpret_cast<const float4*>(a_row), hi = *reinterpret_cast<const float4*>(a_row + 4);
+        const float4 b = *reinterpret_cast<const float4*>(b_row);
+        const float a[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+            acc[r][0] = fmaf(a[r], b.x, acc[r][0]);
+            acc[r][1] = fmaf(a[r], b.y, acc[r][1]);
+            acc[r][2] = fmaf(a[r], b.z, acc[r][2]);
+            acc[r][3] = fmaf(a[r], b.w, acc[r][3]);
+        }
+    };
+    const float* S = p.piece_s + (static_cast<size_t>(z) * p.H + h) * D * DV;
+    for (int d0 = 0; d0 < DP && d0 < D; d0 += SLAB) {
+        if (DV % 4 == 0) {
+            for (int idx = threadIdx.x; idx < SLAB * kChunkCols / 4; idx += kChunkThreads) {
+                const int d = idx / (kChunkCols / 4), c = (idx % (kChunkCols / 4)) * 4;
+                float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (d0 + d < D && col0 + c < DV) s = *reinterpret_cast<const float4*>(S + static_cast<size_t>(d0 + d) * DV + col0 + c);
+                *reinterpret_cast<float4*>(kT + d * kChunkCols + c) = s;
+            }
+        } else {
+            for (int idx = threadIdx.x; idx < SLAB * kChunkCols; idx += kChunkThreads) {
+                const int d = idx / kChunkCols, c = idx % kChunkCols;
+                kT[idx] = d0 + d < D && col0 + c < DV ? S[static_cast<size_t>(d0 + d) * DV + col0 + c] : 0.f;
+            }
+        }
+        __syncthreads();
+#pragma unroll 2
+        for (int d = 0; d < SLAB; ++d) step(qT + (d0 + d) * kLd + 8 * warp, kT + d * kChunkCols + 4 * lane);
+        __syncthreads();
+    }
+    if (RULE == kConstantDecay) {
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+            const float f = powers[8 * warp + r + 1];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[r][e] *= f;
+        }
+    }
+    for (int idx = threadIdx.x; idx < nt * kChunkCols; idx += kChunkThreads) {
+        const int j = idx / kChunkCols, c = idx - j * kChunkCols;
+        float v = 0.f;
+        if (col0 + c < DV) {
+            v = load_any(p.v, (row0 + j) * p.ld + h * DV + col0 + c, p.in_bf16);
+            if (RULE == kConstantDecay) v = silu_f(v);
+        }
+        kT[idx] = v;
+    }
+    __syncthreads();
+    const int last = min(nt, 8 * warp + 8);         // later tokens have no weight in this warp's rows
+#pragma unroll 2
+    for (int j = 0; j < last; ++j) step(aT + j * kLd + 8 * warp, kT + j * kChunkCols + 4 * lane);
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+        const int i = 8 * warp + r;
+        if (i >= nt) break;
+        float* dst = p.o + ((row0 + i) * p.H + h) * DV + col0 + 4 * lane;
+        if (DV % 4 == 0) {
+            if (col0 + 4 * lane < DV) *reinterpret_cast<float4*>(dst) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (col0 + 4 * lane + e < DV) dst[e] = acc[r][e];
+        }
+    }
+}
+
+template <typename... A>
+cudaError_t more_shared_memory(void (*kernel)(A...), int bytes) {
+    return bytes > 48 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) : cudaSuccess;
+}
+
+template <int DP, int RULE>
+int launch_chunks(const ChunkArgs& p, float* state, long long state_stride, const int32_t* state_slot, int num_seqs, cudaStream_t stream) {
+    const int zs = num_seqs * p.max_pieces;
+    const dim3 grid((p.DV + kChunkCols - 1) / kChunkCols, p.H, zs), block(kChunkThreads);
+    constexpr int sum_bytes = (kChunk * DP + kChunk * kChunkCols) * 4, out_bytes = chunk_out_floats<DP>() * 4;
+    cudaError_t e = more_shared_memory(chunk_sum_kernel<DP, RULE>, sum_bytes);
+    if (e == cudaSuccess) e = more_shared_memory(chunk_out_kernel<DP, RULE>, out_bytes);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    if (RULE == kChannelDecay) stride::launch(chunk_decay_kernel, dim3((p.H * p.D + 127) / 128, zs), dim3(128), 0, stream, p);
+    stride::launch(chunk_sum_kernel<DP, RULE>, grid, block, sum_bytes, stream, p);
+    stride::launch(pieces_combine_kernel, dim3((p.H * p.D * p.DV + 255) / 256, num_seqs), dim3(256), 0, stream, p.piece_s,
+                   static_cast<const float*>(p.piece_p), state, state_stride, p.q_len, state_slot, p.H, p.D, p.DV, kChunk, p.max_pieces);
+    stride::launch(chunk_out_kernel<DP, RULE>, grid, block, out_bytes, stream, p);
+    return STRIDE_LAUNCH_STATUS();
+}
+
+template <int RULE>
+int dispatch_chunks(const ChunkArgs& p, float* state, long long state_stride, const int32_t* state_slot, int num_seqs, cudaStream_t stream) {
+    if (p.D <= 32) return launch_chunks<32, RULE>(p, state, state_stride, state_slot, num_seqs, stream);
+    if (p.D <= 64) return launch_chunks<64, RULE>(p, state, state_stride, state_slot, num_seqs, stream);
+    if (p.D <= 128) return launch_chunks<128, RULE>(p, state, state_stride, state_slot, num_seqs, stream);
+    if (p.D <= 256) return launch_chunks<256, RULE>(p, state, state_stride, state_slot, num_seqs, stream);
+    return STRIDE_UNSUPPORTED;
+}
+
+}  // namespace stride
+
+using namespace stride;
+
+extern "C" {
+
+// One token after the other. q, k [tokens, ld] with head h at column h * D, v with head h at column h * DV, all in the compute
+// type. fade (constant decay): [H] float32, the decay minus one; null: channel decays from logit [tokens, H * D] and bias
+// [H * D], float32. o [tokens, H * DV] float32; state: S of head h at h * D * DV floats into a slot's row.
+int stride_decay_scan(const void* q, const void* k, const void* v, int ld, const float* logit, const float* bias, const float* fade,
+                      float q_scale, float inv_tau, float* o, float* state, long long state_stride, const int32_t* q_start,
+                      const int32_t* q_len, const int32_t* state_slot, int num_seqs, int H, int D, int DV, int dtype, cudaStream_t stream) {
+    if (num_seqs < 0 || H <= 0 || D <= 0 || DV <= 0 || (!fade && (!logit || !bias))) return STRIDE_BAD_ARGUMENT;
+    if (state_stride < static_cast<long long>(H) * D * DV) return STRIDE_BAD_ARGUMENT;
+    if (dtype != STRIDE_DTYPE_F32 && dtype != STRIDE_DTYPE_BF16) return STRIDE_BAD_ARGUMENT;
+    if (num_seqs > 65535 || H > 65535) return STRIDE_UNSUPPORTED;
+    if (num_seqs == 0) return 0;
+    ScanArgs p = {};
+    p.a = q;
+    p.k = k;
+    p.v = v;
+    p.lda = p.ldv = ld;
+    p.w = logit;
+    p.w0 = bias;
+    p.fade = fade;
+    p.q_scale = q_scale;
+    p.inv_tau = inv_tau;
+    p.o = o;
+    p.state = state;
+    p.state_stride = state_stride;
+    p.q_start = q_start;
+    p.q_len = q_len;
+    p.state_slot = state_slot;
+    p.H = H;
+    p.group = 1;
+    p.D = D;
+    p.DV = DV;
+    p.in_bf16 = dtype == STRIDE_DTYPE_BF16 ? 1 : 0;
+    return fade ? launch_scan<kConstantDecay>(p, num_seqs, stream) : launch_scan<kChannelDecay>(p, num_seqs, stream);
+}
+
+// Chunk by chunk. powers (constant decay): [H, 65] float32, decay^0 .. decay^64; null: channel decays, whose logits are
+// overwritten. scratch: float32, num_seqs * max_pieces * H * D * (DV + 1), max_pieces = ceil(longest portion / 64).
+int stride_decay_chunks(const void* q, const void* k, const void* v, int ld, float* logit, const float* bias, const float* powers,
+                        float q_scale, float inv_tau, float* o, float* state, long long state_stride, const int32_t* q_start,
+                        const int32_t* q_len, const int32_t* state_slot, int num_seqs, int H, int D, int DV, int dtype, int max_pieces,
+                        float* scratch, cudaStream_t stream) {
+    if (num_seqs < 0 || H <= 0 || D <= 0 || DV <= 0 || max_pieces <= 0 || !scratch || (!powers && (!logit || !bias))) return STRIDE_BAD_ARGUMENT;
+    if (state_stride < static_cast<long long>(H) * D * DV) return STRIDE_BAD_ARGUMENT;
+    if (dtype != STRIDE_DTYPE_F32 && dtype != STRIDE_DTYPE_BF16) return STRIDE_BAD_ARGUMENT;
+    if (static_cast<long long>(num_seqs) * max_pieces > 65535 || H > 65535 || reinterpret_cast<uintptr_t>(scratch) % 16) return STRIDE_UNSUPPORTED;
+    if (num_seqs == 0) return 0;
+    ChunkArgs p = {};
+    p.q = q;
+    p.k = k;
+    p.v = v;
+    p.ld = ld;
+    p.in_bf16 = dtype == STRIDE_DTYPE_BF16 ? 1 : 0;
+    p.cum = logit;
+    p.bias = bias;
+    p.powers = powers;
+    p.q_scale = q_scale;
+    p.inv_tau = inv_tau;
+    p.o = o;
+    p.piece_s = scratch;
+    p.piece_p = scratch + static_cast<size_t>(num_seqs) * max_pieces * H * D * DV;
+    p.q_start = q_start;
+    p.q_len = q_len;
+    p.H = H;
+    p.D = D;
+    p.DV = DV;
+    p.max_pieces = max_pieces;
+    return powers ? dispatch_chunks<kConstantDecay>(p, state, state_stride, state_slot, num_seqs, stream)
+                  : dispatch_chunks<kChannelDecay>(p, state, state_stride, state_slot, num_seqs, stream);
+}
+
+}  // extern "C"

@@ -13,10 +13,11 @@ namespace stride {
 
 // ----------------------------------------------------------------- embedding
 // out[t, :] = table[ids[t], :] as float32 (python/stride_worker/model.py:252).
-// Padded tokens (seq_of_token < 0) get zeros.
+// Padded tokens (seq_of_token < 0) get zeros. With a position table: out[t, :] = mult * table[ids[t], :] + pos[positions[t], :].
 template <typename T>
 __global__ void embed_gather_kernel(const int32_t* __restrict__ ids, const int32_t* __restrict__ seq_of_token,
-                                    const T* __restrict__ table, float* __restrict__ out, int hidden, int vocab) {
+                                    const T* __restrict__ table, float* __restrict__ out, int hidden, int vocab, float mult,
+                                    const T* __restrict__ pos_table, const int32_t* __restrict__ positions, int num_positions) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -25,7 +26,11 @@ __global__ void embed_gather_kernel(const int32_t* __restrict__ ids, const int32
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // ids are validated on the host; never read outside the table
     const T* row = table + static_cast<size_t>(id) * hidden;
     float* dst = out + static_cast<size_t>(t) * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = live ? to_f32(row[i]) : 0.f;
+    const T* pos = pos_table && live ? pos_table + static_cast<size_t>(min(positions[t], num_positions - 1)) * hidden : nullptr;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+        const float x = __fmul_rn(mult, to_f32(row[i]));
+        dst[i] = live ? (pos ? __fadd_rn(x, to_f32(pos[i])) : x) : 0.f;
+    }
 }
 
 // ------------------------------------------------------- residual add + RMSNorm
@@ -481,7 +486,8 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ in, T* __restrict__ ou
 // embed_gather_kernel with 16-byte reads of the table (hidden % V == 0).
 template <typename T>
 __global__ void embed_gather_vec_kernel(const int32_t* __restrict__ ids, const int32_t* __restrict__ seq_of_token,
-                                        const T* __restrict__ table, float* __restrict__ out, int hidden, int vocab) {
+                                        const T* __restrict__ table, float* __restrict__ out, int hidden, int vocab, float mult,
+                                    const T* __restrict__ pos_table, const int32_t* __restrict__ positions, int num_positions) {
     pdl_trigger();
     pdl_wait();
     constexpr int V = Pack<T>::V;
@@ -491,9 +497,16 @@ __global__ void embed_gather_vec_kernel(const int32_t* __restrict__ ids, const i
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
     const T* row = table + static_cast<size_t>(id) * hidden;
     float* dst = out + static_cast<size_t>(t) * hidden;
+    const T* pos = pos_table && live ? pos_table + static_cast<size_t>(min(positions[t], num_positions - 1)) * hidden : nullptr;
     for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {
-        Pack<T> p;
+        Pack<T> p, q;
         if (live) p.load(row + i);
+        if (pos) q.load(pos + i);
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+            p.v[j] = __fmul_rn(mult, p.v[j]);
+            if (pos) p.v[j] = __fadd_rn(p.v[j], q.v[j]);
+        }
 #pragma unroll
         for (int j = 0; j < V; j += 4)
             *reinterpret_cast<float4*>(dst + i + j) =
@@ -548,21 +561,26 @@ using namespace stride;
 extern "C" {
 
 int stride_embed_gather(const int32_t* ids, const int32_t* seq_of_token, const void* table, float* out, int tokens,
-                        int hidden, int vocab, int dtype, cudaStream_t stream) {
-    if (tokens < 0 || hidden <= 0 || vocab <= 0) return STRIDE_BAD_ARGUMENT;
+                        int hidden, int vocab, float mult, const void* pos_table, const int32_t* positions, int num_positions, int dtype,
+                        cudaStream_t stream) {
+    if (tokens < 0 || hidden <= 0 || vocab <= 0 || (pos_table && (!positions || num_positions <= 0))) return STRIDE_BAD_ARGUMENT;
     if (tokens == 0) return 0;
     const int threads = hidden >= 1024 ? 256 : 128;
-    const bool aligned = (reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+    const bool aligned = (reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(pos_table)) % 16 == 0;
     if (dtype == STRIDE_DTYPE_F32) {
         if (aligned && hidden % 4 == 0)
-            stride::launch(embed_gather_vec_kernel<float>, dim3(tokens), dim3(128), 0, stream, ids, seq_of_token, static_cast<const float*>(table), out, hidden, vocab);
+            stride::launch(embed_gather_vec_kernel<float>, dim3(tokens), dim3(128), 0, stream, ids, seq_of_token, static_cast<const float*>(table), out, hidden, vocab, mult,
+                           static_cast<const float*>(pos_table), positions, num_positions);
         else
-            stride::launch(embed_gather_kernel<float>, dim3(tokens), dim3(threads), 0, stream, ids, seq_of_token, static_cast<const float*>(table), out, hidden, vocab);
+            stride::launch(embed_gather_kernel<float>, dim3(tokens), dim3(threads), 0, stream, ids, seq_of_token, static_cast<const float*>(table), out, hidden, vocab, mult,
+                           static_cast<const float*>(pos_table), positions, num_positions);
     } else if (dtype == STRIDE_DTYPE_BF16) {
         if (aligned && hidden % 8 == 0)
-            stride::launch(embed_gather_vec_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, ids, seq_of_token, static_cast<const __nv_bfloat16*>(table), out, hidden, vocab);
+            stride::launch(embed_gather_vec_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, ids, seq_of_token, static_cast<const __nv_bfloat16*>(table), out, hidden, vocab, mult,
+                           static_cast<const __nv_bfloat16*>(pos_table), positions, num_positions);
         else
-            stride::launch(embed_gather_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream, ids, seq_of_token, static_cast<const __nv_bfloat16*>(table), out, hidden, vocab);
+            stride::launch(embed_gather_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream, ids, seq_of_token, static_cast<const __nv_bfloat16*>(table), out, hidden, vocab, mult,
+                           static_cast<const __nv_bfloat16*>(pos_table), positions, num_positions);
     } else {
         return STRIDE_BAD_ARGUMENT;
     }

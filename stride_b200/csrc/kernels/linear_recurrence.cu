@@ -25,17 +25,9 @@
 //                   start), one per consumer; the portion's last input goes into the state
 //   head_norm_gate  o / rms(o) * weight * gate per head, into the compute type for the output projection
 // The scans end by writing S back and, for the delta rule, by moving the convolution's tail in the state forward.
-#include "common.cuh"
+#include "memory_scan.cuh"
 
 namespace stride {
-
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
-
-__device__ __forceinline__ float load_any(const void* p, size_t i, int is_bf16) {
-    return is_bf16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p)[i]) : static_cast<const float*>(p)[i];
-}
 
 // ------------------------------------------------------------------------------------------------ delta_prepare
 // proj [tokens, ld] (compute type): columns [0, GD) q, [GD, 2GD) k, [2GD, 2GD + HV) v, then H columns of beta's
@@ -183,302 +175,6 @@ head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ wei
     }
 }
 
-// --------------------------------------------------------------------------------------------------------- scans
-constexpr int kScanThreads = 128;
-
-struct ScanArgs {
-    const void* a;          // queries (delta) / receptance (memory with bonus): [tokens, lda], head h at column (h / group) * D
-    const void* k;          // keys, the same layout
-    const float* w;         // [tokens, H * D]: the decay minus one (delta), or its double logarithm before w0 (bonus rule)
-    const void* v;          // values [tokens, ldv], head h at column h * DV
-    const float* beta;      // [tokens, H] (delta) or null
-    const float* w0;        // [H * D] added to w before exp(-exp(.)) (bonus rule) or null
-    const float* bonus;     // [H * D] (bonus rule) or null
-    float* o;               // [tokens, H * DV] float32
-    float* state;           // [slots, state_stride]; S of head h at h * D * DV
-    long long state_stride;
-    const int32_t* q_start;
-    const int32_t* q_len;
-    const int32_t* state_slot;
-    int lda, ldv, H, group, D, DV, in_bf16;
-    // the convolution's tail (delta rule; taps 0: none): the last taps - 1 rows of proj's first C columns
-    const void* proj;
-    int ld_proj, C, taps, proj_bf16;
-    long long tail_off;
-    // pieces (mode 0: none, a request's tokens in one chain). A piece is `piece` consecutive tokens of a request; grid z is
-    // request * max_pieces + piece. Mode 1 runs every piece from a zero memory, writes no output, and leaves the piece's
-    // memory in piece_s [z, H, D, DV] and the product of its decays in piece_p [z, H, D]; mode 2 runs every piece from
-    // piece_s (by then the memory at the piece's start), writes the outputs and leaves the state alone.
-    // init (mode 1): 1 starts every column from zero, 2 from the unit matrix (column j holds a one in row j): with no values
-    // (v null) the memory of a piece then ends as the matrix that carries any memory across the piece.
-    int mode, piece, max_pieces, init;
-    float* piece_s;
-    float* piece_p;
-};
-
-// LANES lanes share a column, each with R of its rows (R a multiple of 4): D <= LANES * R. A thread works on NC columns
-// at once (COLS apart), CHUNK tokens are staged at a time. One token follows the other and a warp issues in order, so what
-// sets the pace of a prompt is the chain of dependent instructions a token costs a warp (shared-memory reads, the sums,
-// the shuffles), not the amount of arithmetic: the rows are spread over as many lanes as the head size allows, and the NC
-// columns of a thread are independent chains that fill one another's waits (they also share the reads of k, q and the decay).
-// PIECES false: the one chain only (mode 0), with nothing of the pieces' bookkeeping in its loop.
-template <int LANES, int R, int NC, int CHUNK, int RULE, bool PIECES>      // RULE 0: gated delta rule, 1: decayed memory with a bonus
-__global__ void __launch_bounds__(kScanThreads)
-scan_kernel(const ScanArgs p) {
-    // Launched without programmatic dependent launch (launch_alone): no trigger, and nothing to wait for.
-    const int mode = PIECES ? p.mode : 0;
-    constexpr int DP = R * LANES;                           // rows with padding
-    constexpr int THREADS = kScanThreads;
-    constexpr int COLS = THREADS / LANES;                   // columns of one pass over the threads
-    constexpr int CTA_COLS = COLS * NC;                     // columns of this CTA
-    constexpr int ROW_ITEMS = CHUNK * DP / THREADS;         // entries of each [chunk, DP] array a thread fetches
-    constexpr int V_ITEMS = (CHUNK * CTA_COLS + THREADS - 1) / THREADS;
-    static_assert(R % 4 == 0 && (CHUNK * DP) % THREADS == 0 && CHUNK <= THREADS, "chunks are shared out evenly");
-    // two buffers: while the tokens of one chunk are worked through, the next chunk's inputs are on their way from
-    // global memory into registers; they are stored (the decay's exponentials applied) when the chunk is done
-    __shared__ __align__(16) float s_a[2][CHUNK][DP], s_k[2][CHUNK][DP], s_w[2][CHUNK][DP];
-    __shared__ float s_v[2][CHUNK][CTA_COLS], s_beta[2][CHUNK];
-    __shared__ __align__(16) float s_bonus[DP], s_w0[DP];
-    const int seq = mode ? blockIdx.z / p.max_pieces : blockIdx.z, h = blockIdx.y;
-    const int first = mode ? (blockIdx.z % p.max_pieces) * p.piece : 0;         // this CTA's tokens of the request: [first, len)
-    const int len = mode ? min(p.q_len[seq], first + p.piece) : p.q_len[seq];
-    if (len <= first) return;
-    const int start = p.q_start[seq];
-    const int il = threadIdx.x & (LANES - 1), jc = threadIdx.x / LANES;
-    const int j0 = blockIdx.x * CTA_COLS + jc;              // this thread's columns: j0 + c * COLS
-    const int D = p.D, DV = p.DV, H = p.H;
-    const int hk = h / p.group;
-    float* S_g = mode ? p.piece_s + (static_cast<size_t>(blockIdx.z) * H + h) * D * DV
-                        : p.state + static_cast<size_t>(p.state_slot[seq]) * p.state_stride + static_cast<size_t>(h) * D * DV;
-    // lane il of a column's lanes holds rows 4 LANES g + 4 il + e (g < R / 4, e < 4) in S[.][4 g + e]: four neighbouring rows
-    // are one 16-byte read of shared memory, and the lanes read consecutive 16 bytes
-    auto row_of = [&](int r) { return 4 * LANES * (r >> 2) + 4 * il + (r & 3); };
-    float S[NC][R];
-#pragma unroll
-    for (int c = 0; c < NC; ++c)
-#pragma unroll
-        for (int r = 0; r < R; ++r) {
-            const int i = row_of(r), j = j0 + c * COLS;
-            S[c][r] = mode == 1 ? ((p.init == 2 && i == j && i < D) ? 1.f : 0.f)
-                                  : ((i < D && j < DV) ? S_g[static_cast<size_t>(i) * DV + j] : 0.f);
-        }
-    float decayed[R];           // mode 1: the product of the decays of this thread's rows over the piece
-#pragma unroll
-    for (int r = 0; r < R; ++r) decayed[r] = 1.f;
-    if (RULE == 1)
-        for (int i = threadIdx.x; i < DP; i += blockDim.x) {
-            s_bonus[i] = i < D ? p.bonus[h * D + i] : 0.f;
-            s_w0[i] = i < D ? p.w0[h * D + i] : 0.f;
-        }
-
-    float fa[ROW_ITEMS], fk[ROW_ITEMS], fw[ROW_ITEMS], fv[V_ITEMS], fb = 0.f;
-    auto fetch = [&](int c0) {          // the chunk from token c0 on, into registers (zeros past the request's end)
-#pragma unroll
-        for (int n = 0; n < ROW_ITEMS; ++n) {
-            const int idx = n * THREADS + threadIdx.x;
-            const int tt = idx / DP, i = idx - tt * DP;
-            fa[n] = fk[n] = fw[n] = 0.f;
-            if (c0 + tt < len && i < D) {
-                const size_t row = static_cast<size_t>(start + c0 + tt);
-                fa[n] = load_any(p.a, row * p.lda + hk * D + i, p.in_bf16);
-                fk[n] = load_any(p.k, row * p.lda + hk * D + i, p.in_bf16);
-                fw[n] = p.w[row * H * D + h * D + i];
-            }
-        }
-#pragma unroll
-        for (int n = 0; n < V_ITEMS; ++n) {
-            const int idx = n * THREADS + threadIdx.x;
-            const int tt = idx / CTA_COLS, c = idx - tt * CTA_COLS;
-            const int col = blockIdx.x * CTA_COLS + c;
-            fv[n] = ((!PIECES || p.v != nullptr) && tt < CHUNK && c0 + tt < len && col < DV)
-                        ? load_any(p.v, static_cast<size_t>(start + c0 + tt) * p.ldv + h * DV + col, p.in_bf16) : 0.f;
-        }
-        if (RULE == 0 && threadIdx.x < CHUNK)
-            fb = c0 + threadIdx.x < len ? p.beta[static_cast<size_t>(start + c0 + threadIdx.x) * H + h] : 0.f;
-    };
-    auto stash = [&](int buf) {
-#pragma unroll
-        for (int n = 0; n < ROW_ITEMS; ++n) {
-            const int idx = n * THREADS + threadIdx.x;
-            const int tt = idx / DP, i = idx - tt * DP;
-            float w = fw[n];
-            if (RULE == 1) w = i < D ? expm1f(-expf(w + s_w0[i])) : 0.f;
-            s_a[buf][tt][i] = fa[n];
-            s_k[buf][tt][i] = fk[n];
-            s_w[buf][tt][i] = w;
-        }
-#pragma unroll
-        for (int n = 0; n < V_ITEMS; ++n) {
-            const int idx = n * THREADS + threadIdx.x;
-            if (idx < CHUNK * CTA_COLS) s_v[buf][idx / CTA_COLS][idx % CTA_COLS] = fv[n];
-        }
-        if (RULE == 0 && threadIdx.x < CHUNK) s_beta[buf][threadIdx.x] = fb;
-    };
-
-    fetch(first);
-    __syncthreads();            // s_w0 is there
-    stash(0);
-    __syncthreads();
-    int buf = 0;
-    for (int c0 = first; c0 < len; c0 += CHUNK, buf ^= 1) {
-        const int nt = min(CHUNK, len - c0);
-        const bool more = c0 + CHUNK < len;
-        if (more) fetch(c0 + CHUNK);
-        for (int tt = 0; tt < nt; ++tt) {
-            const float4* w4 = reinterpret_cast<const float4*>(&s_w[buf][tt][4 * il]);
-            const float4* k4 = reinterpret_cast<const float4*>(&s_k[buf][tt][4 * il]);
-            const float4* a4 = reinterpret_cast<const float4*>(&s_a[buf][tt][4 * il]);
-            float vj[NC], out[NC];
-#pragma unroll
-            for (int c = 0; c < NC; ++c) vj[c] = s_v[buf][tt][jc + c * COLS];
-            // four partial sums a read (fixed order): a single chain of R dependent additions would set the pace
-            if (RULE == 0) {
-                float d[NC][4], kk[R];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) d[c][0] = d[c][1] = d[c][2] = d[c][3] = 0.f;
-#pragma unroll
-                for (int g = 0; g < R / 4; ++g) {
-                    const float4 w = w4[LANES * g], k = k4[LANES * g];
-                    const float wv[4] = {w.x, w.y, w.z, w.w};
-                    kk[4 * g] = k.x; kk[4 * g + 1] = k.y; kk[4 * g + 2] = k.z; kk[4 * g + 3] = k.w;
-#pragma unroll
-                    for (int c = 0; c < NC; ++c)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            S[c][4 * g + e] = fmaf(S[c][4 * g + e], wv[e], S[c][4 * g + e]);
-                            d[c][e] = fmaf(S[c][4 * g + e], kk[4 * g + e], d[c][e]);
-                        }
-                }
-                float u[NC];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) u[c] = (d[c][0] + d[c][1]) + (d[c][2] + d[c][3]);
-#pragma unroll
-                for (int o = 1; o < LANES; o <<= 1)
-#pragma unroll
-                    for (int c = 0; c < NC; ++c) u[c] += __shfl_xor_sync(0xffffffffu, u[c], o);
-                const float beta = s_beta[buf][tt];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) u[c] = beta * (vj[c] - u[c]);
-                float acc[NC][4];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
-#pragma unroll
-                for (int g = 0; g < R / 4; ++g) {
-                    const float4 q = a4[LANES * g];
-                    const float qv[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-                    for (int c = 0; c < NC; ++c)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            S[c][4 * g + e] = fmaf(kk[4 * g + e], u[c], S[c][4 * g + e]);
-                            acc[c][e] = fmaf(S[c][4 * g + e], qv[e], acc[c][e]);
-                        }
-                }
-#pragma unroll
-                for (int c = 0; c < NC; ++c) out[c] = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
-            } else {
-                const float4* b4 = reinterpret_cast<const float4*>(&s_bonus[4 * il]);
-                float acc[NC][4];
-#pragma unroll
-                for (int c = 0; c < NC; ++c) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
-#pragma unroll
-                for (int g = 0; g < R / 4; ++g) {
-                    const float4 w = w4[LANES * g], k = k4[LANES * g], rr = a4[LANES * g], b = b4[LANES * g];
-                    const float wv[4] = {w.x, w.y, w.z, w.w}, kv4[4] = {k.x, k.y, k.z, k.w}, rv[4] = {rr.x, rr.y, rr.z, rr.w},
-                                bv[4] = {b.x, b.y, b.z, b.w};
-                    if (mode == 1) {
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) decayed[4 * g + e] = fmaf(wv[e], decayed[4 * g + e], decayed[4 * g + e]);
-                    }
-#pragma unroll
-                    for (int c = 0; c < NC; ++c)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const float kv = kv4[e] * vj[c];
-                            acc[c][e] = fmaf(rv[e], fmaf(bv[e], kv, S[c][4 * g + e]), acc[c][e]);
-                            S[c][4 * g + e] = fmaf(wv[e], S[c][4 * g + e], S[c][4 * g + e]) + kv;
-                        }
-                }
-#pragma unroll
-                for (int c = 0; c < NC; ++c) out[c] = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
-            }
-#pragma unroll
-            for (int o = 1; o < LANES; o <<= 1)
-#pragma unroll
-                for (int c = 0; c < NC; ++c) out[c] += __shfl_xor_sync(0xffffffffu, out[c], o);
-            if (il == 0 && mode != 1) {
-#pragma unroll
-                for (int c = 0; c < NC; ++c)
-                    if (j0 + c * COLS < DV) p.o[(static_cast<size_t>(start + c0 + tt) * H + h) * DV + j0 + c * COLS] = out[c];
-            }
-        }
-        if (more) stash(buf ^ 1);       // nobody reads that buffer: its chunk was finished before the last barrier
-        __syncthreads();
-    }
-    if (mode != 2) {
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-            for (int r = 0; r < R; ++r) {
-                const int i = row_of(r), j = j0 + c * COLS;
-                if (i < D && j < DV) S_g[static_cast<size_t>(i) * DV + j] = S[c][r];
-            }
-    }
-    if (mode == 1) {
-        if (RULE == 1 && blockIdx.x == 0 && jc == 0) {
-#pragma unroll
-            for (int r = 0; r < R; ++r)
-                if (row_of(r) < D) p.piece_p[(static_cast<size_t>(blockIdx.z) * H + h) * D + row_of(r)] = decayed[r];
-        }
-        return;
-    }
-    if (mode == 2 && first != 0) return;          // the CTAs of a request's first piece move the tail
-    // The convolution's tail: row m of the new tail is the input of local token len - (taps - 1) + m, which lies in
-    // this step or, for a short step, further up in the old tail. Channels are shared out over the CTAs of the request;
-    // a channel's rows move in ascending order, so a row is read before it is overwritten.
-    if (p.taps > 1) {
-        const int keep = p.taps - 1;
-        const int all = PIECES ? p.q_len[seq] : len;        // the whole request's tokens, whatever this CTA's piece
-        float* tail = p.state + static_cast<size_t>(p.state_slot[seq]) * p.state_stride + p.tail_off;
-        const int cta = blockIdx.y * gridDim.x + blockIdx.x, ctas = gridDim.x * gridDim.y;
-        for (int c = cta * blockDim.x + threadIdx.x; c < p.C; c += ctas * blockDim.x)
-            for (int m = 0; m < keep; ++m) {
-                const int src = all - keep + m;
-                tail[static_cast<size_t>(m) * p.C + c] = src >= 0 ? load_any(p.proj, static_cast<size_t>(start + src) * p.ld_proj + c, p.proj_bf16)
-                                                                 : tail[static_cast<size_t>(m + all) * p.C + c];
-            }
-    }
-}
-
-// Between the two passes over pieces, for a memory whose decay is diagonal: piece_s [z, H, D, DV] holds what every piece
-// adds from a zero memory, piece_p [z, H, D] the product of its decays. One thread an entry of S walks the request's pieces
-// in order: the memory at a piece's start takes the place of the piece's own sum, and the memory after the last piece goes
-// into the state.
-__global__ void __launch_bounds__(256)
-pieces_combine_kernel(float* __restrict__ piece_s, const float* __restrict__ piece_p, float* __restrict__ state, long long state_stride,
-                      const int32_t* __restrict__ q_len, const int32_t* __restrict__ state_slot, int H, int D, int DV, int piece,
-                      int max_pieces) {
-    pdl_trigger();
-    pdl_wait();
-    const int seq = blockIdx.y;
-    const int len = q_len[seq];
-    if (len <= 0) return;
-    const int entry = blockIdx.x * blockDim.x + threadIdx.x;          // over H * D * DV
-    if (entry >= H * D * DV) return;
-    const int row = entry / DV;                                          // h * D + i
-    float* S_g = state + static_cast<size_t>(state_slot[seq]) * state_stride + entry;
-    float S = *S_g;
-    const int pieces = (len + piece - 1) / piece;
-    for (int c = 0; c < pieces; ++c) {
-        const size_t z = static_cast<size_t>(seq) * max_pieces + c;
-        float* at = piece_s + z * H * D * DV + entry;
-        const float own = *at;
-        *at = S;
-        S = fmaf(piece_p[z * H * D + row], S, own);
-    }
-    *S_g = S;
-}
-
 // The same for the delta rule, whose pieces carry a memory across by a full matrix: piece_t [z, H, D, D] holds it, piece_s
 // [z, H, D, DV] what the piece adds from a zero memory; S_next = T S + B. A CTA owns 16 columns of S of one head of one
 // request and walks the pieces in order; T comes through shared memory in slabs of 16 columns. The memory at a piece's
@@ -556,32 +252,51 @@ delta_pieces_combine_kernel(float* __restrict__ piece_s, const float* __restrict
     }
 }
 
-template <int LANES, int R, int CHUNK, int RULE>
-int launch_scan_as(const ScanArgs& p, int num_seqs, cudaStream_t stream) {
-    constexpr int COLS = kScanThreads / LANES;
-    // four columns a thread where the head is wide enough to fill them
-    if (p.mode) num_seqs *= p.max_pieces;
-    if (p.DV >= 4 * COLS) {
-        const dim3 grid((p.DV + 4 * COLS - 1) / (4 * COLS), p.H, num_seqs);
-        if (p.mode) stride::launch_alone(scan_kernel<LANES, R, 4, CHUNK, RULE, true>, grid, dim3(kScanThreads), 0, stream, p);
-        else stride::launch_alone(scan_kernel<LANES, R, 4, CHUNK, RULE, false>, grid, dim3(kScanThreads), 0, stream, p);
-    } else {
-        const dim3 grid((p.DV + COLS - 1) / COLS, p.H, num_seqs);
-        if (p.mode) stride::launch_alone(scan_kernel<LANES, R, 1, CHUNK, RULE, true>, grid, dim3(kScanThreads), 0, stream, p);
-        else stride::launch_alone(scan_kernel<LANES, R, 1, CHUNK, RULE, false>, grid, dim3(kScanThreads), 0, stream, p);
+// The same with a CTA a (token, head), for heads so wide that a warp would walk them for long (one norm over all heads of a
+// token counts as one head). V columns a thread and turn.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict__ weight, int w_head_stride, const void* __restrict__ gate,
+                           int ld_gate, int gate_kind, T* __restrict__ out, int H, int DV, float eps) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x / H, h = blockIdx.x % H;
+    const float* row = o + (static_cast<size_t>(t) * H + h) * DV;
+    const size_t g0 = static_cast<size_t>(t) * ld_gate + h * DV;
+    float ss = 0.f;
+    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
+        alignas(16) float x[V];
+        if constexpr (V == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+        else x[0] = row[j];
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
     }
-    return STRIDE_LAUNCH_STATUS();
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / static_cast<float>(DV) + eps);
+    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
+        alignas(16) float x[V];
+        alignas(16) float w[V];
+        alignas(16) T g[V];
+        alignas(16) T y[V];
+        if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+            *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(weight + h * w_head_stride + j);
+        } else {
+            x[0] = row[j];
+            w[0] = weight[h * w_head_stride + j];
+        }
+        struct alignas(V * sizeof(T)) Pack { T v[V]; };
+        if (gate_kind) *reinterpret_cast<Pack*>(g) = *reinterpret_cast<const Pack*>(static_cast<const T*>(gate) + g0 + j);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float z = gate_kind ? to_f32(g[e]) : static_cast<const float*>(gate)[g0 + j + e];
+            y[e] = from_f32<T>(x[e] * inv * w[e] * (gate_kind == 1 ? silu_f(z) : sigmoid_f(z)));
+        }
+        *reinterpret_cast<Pack*>(out + (static_cast<size_t>(t) * H + h) * DV + j) = *reinterpret_cast<Pack*>(y);
+    }
 }
 
-template <int RULE>
-int launch_scan(const ScanArgs& p, int num_seqs, cudaStream_t stream) {
-    if (p.D <= 16) return launch_scan_as<4, 4, 16, RULE>(p, num_seqs, stream);
-    if (p.D <= 32) return launch_scan_as<8, 4, 16, RULE>(p, num_seqs, stream);
-    if (p.D <= 64) return launch_scan_as<16, 4, 16, RULE>(p, num_seqs, stream);
-    if (p.D <= 128) return launch_scan_as<16, 8, 8, RULE>(p, num_seqs, stream);
-    if (p.D <= 256) return launch_scan_as<16, 16, 4, RULE>(p, num_seqs, stream);
-    return STRIDE_UNSUPPORTED;
-}
+constexpr int kWideHead = 512;
 
 }  // namespace stride
 
@@ -748,6 +463,18 @@ int stride_head_norm_gate(const float* o, const float* weight, int w_head_stride
     if (tokens < 0 || H <= 0 || DV <= 0 || gate_kind < 0 || gate_kind > 2) return STRIDE_BAD_ARGUMENT;
     if (tokens == 0) return 0;
     const long long pairs = static_cast<long long>(tokens) * H;
+    if (DV >= kWideHead && pairs < 0x7fffffff && (dtype == STRIDE_DTYPE_F32 || dtype == STRIDE_DTYPE_BF16)) {
+        auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+        const bool vec = DV % 4 == 0 && ld_gate % 4 == 0 && aligned(o) && aligned(weight) && aligned(gate) && aligned(out) && w_head_stride % 4 == 0;
+        const dim3 cta(DV / (vec ? 4 : 1) >= 256 ? 256 : 128), each(static_cast<unsigned>(pairs));
+        if (dtype == STRIDE_DTYPE_F32)
+            stride::launch(vec ? head_norm_gate_wide_kernel<float, 4> : head_norm_gate_wide_kernel<float, 1>, each, cta, 0, stream, o, weight,
+                           w_head_stride, gate, ld_gate, gate_kind, static_cast<float*>(out), H, DV, eps);
+        else
+            stride::launch(vec ? head_norm_gate_wide_kernel<__nv_bfloat16, 4> : head_norm_gate_wide_kernel<__nv_bfloat16, 1>, each, cta, 0,
+                           stream, o, weight, w_head_stride, gate, ld_gate, gate_kind, static_cast<__nv_bfloat16*>(out), H, DV, eps);
+        return STRIDE_LAUNCH_STATUS();
+    }
     const dim3 grid(static_cast<unsigned>((pairs + 7) / 8)), block(256);
     if (dtype == STRIDE_DTYPE_F32)
         stride::launch(head_norm_gate_kernel<float>, grid, block, 0, stream, o, weight, w_head_stride, gate, ld_gate, gate_kind,

@@ -478,7 +478,24 @@ moe_combine_kernel(const float* __restrict__ Y, const int32_t* __restrict__ row_
     }
 }
 
-// relu(x)^2 in place, for the shared expert (the routed experts apply it in their product's epilogue)
+// relu(x)^2 in place, for the shared expert and for dense feed-forwards without a gate (the routed experts apply it in their
+// product's epilogue). The packed form: one 16-byte pack a thread.
+template <typename T>
+__global__ void relu_squared_vec_kernel(uint4* __restrict__ x, size_t packs) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+    if (i >= packs) return;
+    uint4 r = x[i];
+    T* v = reinterpret_cast<T*>(&r);
+#pragma unroll
+    for (int e = 0; e < static_cast<int>(16 / sizeof(T)); ++e) {
+        const float f = fmaxf(to_f32(v[e]), 0.f);
+        v[e] = from_f32<T>(f * f);
+    }
+    x[i] = r;
+}
+
 template <typename T>
 __global__ void relu_squared_kernel(T* __restrict__ x, size_t n) {
     pdl_trigger();
@@ -596,6 +613,13 @@ int stride_relu_squared(void* x, long long n, int dtype, cudaStream_t stream) {
     if (n < 0) return STRIDE_BAD_ARGUMENT;
     if (n == 0) return 0;
     const unsigned blocks = static_cast<unsigned>(n / 256 >= 4096 ? 4096 : (n + 255) / 256);
+    const int pack = dtype == STRIDE_DTYPE_F32 ? 4 : 8;
+    const long long packs = n / pack;
+    if (n % pack == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0 && (packs + 255) / 256 < 0x7fffffff && (dtype == STRIDE_DTYPE_F32 || dtype == STRIDE_DTYPE_BF16)) {
+        stride::launch(dtype == STRIDE_DTYPE_F32 ? relu_squared_vec_kernel<float> : relu_squared_vec_kernel<__nv_bfloat16>,
+                       dim3(static_cast<unsigned>((packs + 255) / 256)), dim3(256), 0, stream, static_cast<uint4*>(x), static_cast<size_t>(packs));
+        return STRIDE_LAUNCH_STATUS();
+    }
     if (dtype == STRIDE_DTYPE_F32)
         stride::launch(relu_squared_kernel<float>, dim3(blocks), dim3(256), 0, stream, static_cast<float*>(x), static_cast<size_t>(n));
     else if (dtype == STRIDE_DTYPE_BF16)

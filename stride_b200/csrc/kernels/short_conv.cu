@@ -13,9 +13,14 @@
 //   conv_tail        afterwards, the tails move on: row m of the new tail is the projected row of local token
 //                    len - (taps - 1) + m, which lies in this step or, for a short step, further up in the old tail.
 //                    A thread owns a channel and reads all it needs before it writes.
+//   conv_row_norm    the same with one norm over all query channels of a token and one over all its key channels (weights of
+//                    those widths) instead of a norm a head, and a factor on the queries that grows with the token's position p:
+//                    1 + coef ln(floor((p + 1) / every) + 1) (every 0: none). One CTA a token.
 // One warp a (token, head); float32 arithmetic; sums in an order that depends on the head's width only. Heads of whole
 // 16-byte packs on 16-byte boundaries take the packed form: a lane holds whole packs of its head (8 bfloat16 or 4 float32
 // channels), a warp serves one head of up to 32 packs or two heads of up to 16, and every row of a tap is one 16-byte read.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace stride {
@@ -217,6 +222,116 @@ conv_head_norm_vec_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out
     }
 }
 
+// One CTA a token. A thread works on packs of V channels (16 bytes of the compute type, or one channel where sizes or pointers
+// are not multiples of a pack) and keeps their convolved values in shared memory until the two sums of squares are known.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+conv_row_norm_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out, int ld_out, const float* __restrict__ conv_w, int taps,
+                     const float* __restrict__ state, long long state_stride, long long tail_off,
+                     const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ q_start, const int32_t* __restrict__ state_slot,
+                     const int32_t* __restrict__ positions, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                     float temp_coef, int temp_every, const int32_t* __restrict__ slot_mapping, T* __restrict__ k_pages,
+                     T* __restrict__ v_pages, int nq, int nkv, int hd, int vd, int page_size) {
+    extern __shared__ __align__(16) float y_row[];      // C floats
+    __shared__ float part[2][8];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int seq = seq_of_token[t];
+    if (seq < 0) return;
+    const int q_dim = nq * hd, k_dim = nkv * hd, C = q_dim + k_dim + nkv * vd;
+    const int start = q_start[seq], local = t - start;
+    const float* tail = state ? state + static_cast<size_t>(state_slot[seq]) * state_stride + tail_off : nullptr;
+    auto load = [](const auto* p, float* v) {
+        if constexpr (V == 1) v[0] = to_f32(*p);
+        else ConvPack<std::remove_cv_t<std::remove_reference_t<decltype(*p)>>>::load(p, v);
+    };
+    auto load_floats = [](const float* p, float* v) {
+        if constexpr (V == 1) v[0] = *p;
+        else {
+#pragma unroll
+            for (int e = 0; e < V; e += 4) ConvPack<float>::load(p + e, v + e);
+        }
+    };
+    float sq_q = 0.f, sq_k = 0.f;
+    for (int c = threadIdx.x * V; c < C; c += blockDim.x * V) {
+        float y[V];
+        if (conv_w && taps > 1) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = 0.f;
+            for (int j = 0; j < taps; ++j) {
+                const int src = local - (taps - 1) + j;
+                float u[V], w[V];
+                if (src >= 0) load(raw + static_cast<size_t>(start + src) * ld + c, u);
+                else load_floats(tail + static_cast<size_t>(taps - 1 + src) * C + c, u);
+                load_floats(conv_w + static_cast<size_t>(j) * C + c, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e) y[e] = fmaf(w[e], u[e], y[e]);
+            }
+        } else {
+            load(raw + static_cast<size_t>(t) * ld + c, y);
+            if (conv_w) {
+#pragma unroll
+                for (int e = 0; e < V; ++e) y[e] *= conv_w[c + e];
+            }
+        }
+        float sq = 0.f;
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            y_row[c + e] = y[e];
+            sq = fmaf(y[e], y[e], sq);
+        }
+        if (c < q_dim) sq_q += sq;
+        else if (c < q_dim + k_dim) sq_k += sq;
+    }
+    sq_q = warp_sum(sq_q);
+    sq_k = warp_sum(sq_k);
+    if ((threadIdx.x & 31) == 0) {
+        part[0][threadIdx.x >> 5] = sq_q;
+        part[1][threadIdx.x >> 5] = sq_k;
+    }
+    __syncthreads();
+    sq_q = sq_k = 0.f;
+    for (int w = 0; w < (blockDim.x >> 5); ++w) {
+        sq_q += part[0][w];
+        sq_k += part[1][w];
+    }
+    const float inv_q = wq ? rsqrtf(sq_q / static_cast<float>(q_dim) + eps) : 1.f;
+    const float inv_k = wk ? rsqrtf(sq_k / static_cast<float>(k_dim) + eps) : 1.f;
+    const float factor = temp_every > 0 ? fmaf(temp_coef, logf(static_cast<float>((positions[t] + 1) / temp_every + 1)), 1.f) : 1.f;
+    const int slot = slot_mapping ? slot_mapping[t] : -1;
+    for (int c = threadIdx.x * V; c < C; c += blockDim.x * V) {
+        float y[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = y_row[c + e];
+        const bool is_q = c < q_dim, is_v = c >= q_dim + k_dim;
+        const float* weight = is_q ? wq : is_v ? nullptr : wk;
+        if (weight) {
+            float w[V];
+            load_floats(weight + (is_q ? c : c - q_dim), w);
+            const float inv = is_q ? inv_q : inv_k;
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = __fmul_rn(__fmul_rn(y[e], inv), w[e]);
+        }
+        if (is_q) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] *= factor;
+        }
+        T* dst[2] = {out + static_cast<size_t>(t) * ld_out + c, nullptr};
+        if (slot >= 0 && !is_q) {
+            const int at = is_v ? c - q_dim - k_dim : c - q_dim, width = is_v ? vd : hd, kvh = at / width;
+            dst[1] = (is_v ? v_pages : k_pages) +
+                     ((static_cast<size_t>(slot / page_size) * nkv + kvh) * page_size + slot % page_size) * width + (at - kvh * width);
+        }
+#pragma unroll
+        for (int o = 0; o < 2; ++o)
+            if (dst[o]) {
+                if constexpr (V == 1) *dst[o] = from_f32<T>(y[0]);
+                else ConvPack<T>::store(dst[o], y);
+            }
+    }
+}
+
 // grid (sequence slots of the step, channel blocks)
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -286,6 +401,44 @@ int stride_conv_head_norm(const void* raw, int ld, void* out, int ld_out, const 
     else
         return STRIDE_BAD_ARGUMENT;
     return STRIDE_LAUNCH_STATUS();
+}
+
+int stride_conv_row_norm(const void* raw, int ld, void* out, int ld_out, const float* conv_w, int taps, const float* state,
+                         long long state_stride, long long tail_off, const int32_t* seq_of_token, const int32_t* q_start,
+                         const int32_t* state_slot, const int32_t* positions, const float* wq, const float* wk, float eps, float temp_coef,
+                         int temp_every, const int32_t* slot_mapping, void* k_pages, void* v_pages, int tokens, int nq, int nkv, int hd,
+                         int vd, int page_size, int dtype, cudaStream_t stream) {
+    const long long C = static_cast<long long>(nq + nkv) * hd + static_cast<long long>(nkv) * vd;
+    if (tokens < 0 || nq <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || ld < C || ld_out < C || taps < 1 || temp_every < 0)
+        return STRIDE_BAD_ARGUMENT;
+    if (taps > 1 && (!conv_w || !state || !q_start || !state_slot || state_stride < tail_off + (taps - 1) * C)) return STRIDE_BAD_ARGUMENT;
+    if ((slot_mapping != nullptr && (k_pages == nullptr || v_pages == nullptr)) || (temp_every > 0 && !positions)) return STRIDE_BAD_ARGUMENT;
+    const long long bytes = C * 4;
+    if (taps > kConvMaxTaps || bytes > 200 * 1024) return STRIDE_UNSUPPORTED;
+    if (tokens == 0) return 0;
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const int pack = dtype == STRIDE_DTYPE_F32 ? 4 : 8;
+    const bool vec = hd % pack == 0 && vd % pack == 0 && ld % pack == 0 && ld_out % pack == 0 && aligned(raw) && aligned(out) &&
+                     aligned(k_pages) && aligned(v_pages) && aligned(wq) && aligned(wk) && aligned(state) && aligned(conv_w) &&
+                     state_stride % 4 == 0 && tail_off % 4 == 0;
+    auto run = [&](auto kernel, auto* typed_raw) {
+        using T = std::remove_cv_t<std::remove_pointer_t<decltype(typed_raw)>>;
+        if (bytes > 48 * 1024) {
+            const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes));
+            if (e != cudaSuccess) return static_cast<int>(e);
+        }
+        const long long items = vec ? C / pack : C;
+        const int threads = items >= 256 ? 256 : static_cast<int>((items + 31) / 32 * 32);
+        stride::launch(kernel, dim3(tokens), dim3(threads), static_cast<size_t>(bytes), stream, typed_raw, ld, static_cast<T*>(out), ld_out,
+                       conv_w, taps, state, state_stride, tail_off, seq_of_token, q_start, state_slot, positions, wq, wk, eps, temp_coef,
+                       temp_every, slot_mapping, static_cast<T*>(k_pages), static_cast<T*>(v_pages), nq, nkv, hd, vd, page_size);
+        return STRIDE_LAUNCH_STATUS();
+    };
+    if (dtype == STRIDE_DTYPE_F32)
+        return run(vec ? conv_row_norm_kernel<float, 4> : conv_row_norm_kernel<float, 1>, static_cast<const float*>(raw));
+    if (dtype == STRIDE_DTYPE_BF16)
+        return run(vec ? conv_row_norm_kernel<__nv_bfloat16, 8> : conv_row_norm_kernel<__nv_bfloat16, 1>, static_cast<const __nv_bfloat16*>(raw));
+    return STRIDE_BAD_ARGUMENT;
 }
 
 int stride_conv_tail(const void* raw, int ld, float* state, long long state_stride, long long tail_off, const int32_t* q_start,

@@ -29,7 +29,8 @@ _bound: dict[str, ctypes._CFuncPtr] = {}
 
 _SIGNATURES = {
     # name: (library, argtypes)
-    "stride_embed_gather": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_embed_gather": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
+                                            c_int, c_void_p]),
     "stride_add_rmsnorm": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p]),
     "stride_add_residual": ("elementwise", [c_void_p, c_void_p, c_longlong, c_int, c_void_p]),
     "stride_zero_fresh_state": ("elementwise", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
@@ -41,7 +42,7 @@ _SIGNATURES = {
     "stride_gemm_nt_f32": ("gemm_f32", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_paged_attention_generic": ("attention_generic", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                              c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                                             c_int, c_float, c_void_p, c_void_p, c_int, c_void_p]),
+                                                             c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "stride_gemm_tc_skinny": ("gemm_bf16_tc", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_longlong,
                                                c_void_p, c_int, c_void_p, c_void_p]),
     "stride_gemm_tc_clustered": ("gemm_bf16_tc", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
@@ -73,12 +74,17 @@ _SIGNATURES = {
     "stride_paged_decode_attention_gated": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                                                  c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
                                                                  c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p]),
+    "stride_paged_decode_attention_biased": ("attention_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                                                  c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int,
+                                                                  c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                                                  c_int, c_void_p, c_void_p]),
     "stride_paged_prefill_attention": ("attention_prefill", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                                             c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p]),
+                                                             c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
     "stride_paged_prefill_attention_tc": ("attention_prefill_tc", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                                    c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                                                   c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p]),
+                                                                   c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int,
+                                                                   c_void_p, c_void_p]),
     "stride_sample_ranked": ("sampling_ranked", [c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                                  c_void_p, c_void_p, c_longlong, c_void_p]),
     "stride_sample_rows": ("sampling", [c_void_p, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -138,6 +144,16 @@ _SIGNATURES = {
                                              c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_conv_tail": ("short_conv", [c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                         c_int, c_void_p]),
+    "stride_conv_row_norm": ("short_conv", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
+                                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p, c_void_p,
+                                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_copies_step": ("stream_copies", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
+                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_decay_scan": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                           c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_decay_chunks": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                             c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                             c_void_p, c_void_p]),
     "stride_mlstm_scan": ("mlstm", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
                                     c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_pointwise": ("pointwise", [c_void_p, c_void_p, c_int, c_float, c_longlong, c_int, c_void_p]),
@@ -195,6 +211,9 @@ _CLASS_OF = {
     "stride_stream_concat": "repeated block: input", "stride_add_row_vector": "repeated block: input",
     "stride_rms_norm_cols": "latent norm", "stride_conv_head_norm": "convolution + head norms + cache write",
     "stride_conv_tail": "convolution + head norms + cache write", "stride_mlstm_scan": "matrix LSTM: recurrence",
+    "stride_conv_row_norm": "convolution + row norms + cache write", "stride_copies_step": "residual copies + norm",
+    "stride_decay_scan": "fading memory: recurrence", "stride_decay_chunks": "fading memory: recurrence",
+    "stride_paged_decode_attention_biased": "attention (decode)",
 }
 
 
@@ -284,6 +303,16 @@ def _opt(t, name: str, dtype=None) -> int | None:
     return None if t is None else _dev(t, name, dtype)
 
 
+def _state_rows(state) -> tuple:
+    """(pointer, floats from row to row) of per-request state [slots, n] float32. The rows may be a column block of wider
+    ones: mixers that share a request's slot each see their own part."""
+    if not state.is_cuda:
+        raise KernelError("state must live on a CUDA device; stride_b200 has no CPU path")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1:
+        raise KernelError("state must be float32 [slots, n] with the floats of a row side by side")
+    return state.data_ptr(), state.stride(0)
+
+
 def _code(dtype: torch.dtype) -> int:
     try:
         return DTYPE_CODE[dtype]
@@ -298,11 +327,15 @@ def require_device() -> None:
 
 
 # ------------------------------------------------------------------ elementwise
-def embed_gather(ids, seq_of_token, table, out) -> None:
+def embed_gather(ids, seq_of_token, table, out, mult: float = 1.0, pos_table=None, positions=None) -> None:
+    """``out[t] = mult * table[ids[t]]`` (+ ``pos_table[positions[t]]``) in float32; zeros for padded rows."""
     tokens, hidden = out.shape
+    if pos_table is not None and (pos_table.dtype != table.dtype or pos_table.shape[1] != hidden):
+        raise KernelError("embed_gather: the position table must have the embedding's width and element type")
     _check(_fn("stride_embed_gather")(_dev(ids, "ids", torch.int32), _opt(seq_of_token, "seq_of_token", torch.int32),
                                       _dev(table, "table"), _dev(out, "out", torch.float32), tokens, hidden,
-                                      table.shape[0], _code(table.dtype), _stream()), "embed_gather")
+                                      table.shape[0], float(mult), _opt(pos_table, "pos_table"), _opt(positions, "positions", torch.int32),
+                                      0 if pos_table is None else pos_table.shape[0], _code(table.dtype), _stream()), "embed_gather")
 
 
 def add_rmsnorm(residual, delta, weight, out, eps: float, rows=None) -> None:
@@ -466,7 +499,7 @@ def delta_prepare(proj, conv_w, low, a_log, dt_bias, state, tail_off: int, seq_o
         raise KernelError("delta_prepare: shapes do not agree")
     _check(_fn("stride_delta_prepare")(
         _dev(proj, "proj"), proj.shape[1], _dev(conv_w, "conv_w", torch.float32), _dev(low, "low", torch.float32), low.shape[1],
-        _dev(a_log, "a_log", torch.float32), _dev(dt_bias, "dt_bias", torch.float32), _dev(state, "state", torch.float32), state.shape[1],
+        _dev(a_log, "a_log", torch.float32), _dev(dt_bias, "dt_bias", torch.float32), *_state_rows(state),
         int(tail_off), _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32),
         _dev(state_slot, "state_slot", torch.int32), _dev(qk, "qk", torch.float32), _dev(v, "v", torch.float32),
         _dev(beta, "beta", torch.float32), _dev(decay, "decay", torch.float32), tokens, G, H, D, DV, taps, float(unit_eps),
@@ -488,7 +521,7 @@ def delta_scan(qk, v, beta, decay, o, state, tail_off: int, proj, q_start, q_len
         raise KernelError("delta_scan: the scratch is too small")
     _check(_fn("stride_delta_scan")(
         _dev(qk, "qk", torch.float32), _dev(v, "v", torch.float32), _dev(beta, "beta", torch.float32), _dev(decay, "decay", torch.float32),
-        _dev(o, "o", torch.float32), _dev(state, "state", torch.float32), state.shape[1], int(tail_off), _dev(proj, "proj"), proj.shape[1],
+        _dev(o, "o", torch.float32), *_state_rows(state), int(tail_off), _dev(proj, "proj"), proj.shape[1],
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32), num_seqs,
         G, H, D, DV, taps, _code(proj.dtype), piece, max_pieces, _opt(scratch, "scratch", torch.float32), _stream()), "delta_scan")
 
@@ -511,7 +544,7 @@ def bonus_scan(r, k, v, wlog, w0, bonus, o, state, q_start, q_len, state_slot, n
         raise KernelError("bonus_scan: the scratch is too small")
     _check(_fn("stride_bonus_scan")(
         _dev(r, "r"), _dev(k, "k"), _dev(v, "v"), _dev(wlog, "wlog", torch.float32), _dev(w0, "w0", torch.float32),
-        _dev(bonus, "bonus", torch.float32), _dev(o, "o", torch.float32), _dev(state, "state", torch.float32), state.shape[1],
+        _dev(bonus, "bonus", torch.float32), _dev(o, "o", torch.float32), *_state_rows(state),
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32), num_seqs,
         H, D, _code(r.dtype), piece, max_pieces, _opt(scratch, "scratch", torch.float32), _stream()), "bonus_scan")
 
@@ -524,7 +557,7 @@ def shift_mix(x, mu, state, prev_off: int, seq_of_token, q_start, q_len, state_s
     if out.shape != (mixes, tokens, width) or out.dtype != x.dtype or mu.shape[1] != width:
         raise KernelError("shift_mix: shapes do not agree")
     _check(_fn("stride_shift_mix")(
-        _dev(x, "x"), _dev(mu, "mu", torch.float32), _dev(state, "state", torch.float32), state.shape[1], int(prev_off),
+        _dev(x, "x"), _dev(mu, "mu", torch.float32), *_state_rows(state), int(prev_off),
         _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
         _dev(state_slot, "state_slot", torch.int32), _dev(out, "out"), tokens, width, mixes, _code(x.dtype), _stream()), "shift_mix")
 
@@ -557,9 +590,93 @@ def mlstm_scan(proj, q_off: int, k_off: int, v_off: int, gates, bias_i, bias_f, 
     _check(_fn("stride_mlstm_scan")(
         _dev(proj, "proj"), proj.shape[1], int(q_off), int(k_off), int(v_off), _dev(gates, "gates", torch.float32), gates.shape[1],
         _dev(bias_i, "bias_i", torch.float32), _dev(bias_f, "bias_f", torch.float32), float(cap), float(q_scale),
-        _dev(o, "o", torch.float32), _dev(state, "state", torch.float32), state.shape[1], _dev(q_start, "q_start", torch.int32),
+        _dev(o, "o", torch.float32), *_state_rows(state), _dev(q_start, "q_start", torch.int32),
         _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype),
         _stream()), "mlstm_scan")
+
+
+# ------------------------------------------------------------ fading memories (linear attention with decay)
+DECAY_CHUNK = 64        # tokens a chunk of ``decay_chunks``
+# Portions of at least this many tokens run chunk by chunk in bfloat16 models (float32 models keep the one chain, whose sums do
+# not depend on the cutting). 0: never.
+DECAY_CHUNKS_MIN_TOKENS = int(_os.environ.get("STRIDE_B200_DECAY_CHUNKS_MIN", "96"))
+
+
+def _decay_args(proj, q_off, k_off, v_off, logit, bias, H, D, DV, o):
+    if proj.shape[1] < max(q_off + H * D, k_off + H * D, v_off + H * DV) or o.shape != (proj.shape[0], H * DV):
+        raise KernelError("fading memory: the projection or the output has the wrong width")
+    if logit is not None and (logit.shape != (proj.shape[0], H * D) or bias.numel() != H * D):
+        raise KernelError("fading memory: one decay logit per token, head and key channel is needed")
+    base, item = _dev(proj, "proj"), proj.element_size()
+    return base + q_off * item, base + k_off * item, base + v_off * item, proj.shape[1]
+
+
+def decay_scan(proj, q_off: int, k_off: int, v_off: int, logit, bias, fade, q_scale: float, inv_tau: float, o, state, q_start, q_len,
+               state_slot, num_seqs: int, H: int, D: int, DV: int) -> None:
+    """A matrix memory that fades, over every request of the step in token order. ``proj`` [tokens, ld] holds q, k ([H, D]) and v
+    ([H, DV]) from the given columns on. Channel decays (``fade`` None): ``S = diag(sigmoid(logit + bias)^inv_tau) S + k v^T``,
+    ``o = q_scale S^T q`` (``logit`` float32 [tokens, H * D], ``bias`` float32 [H * D]). Constant decay (``fade`` float32 [H], the
+    decay minus one): ``S = (1 + fade) S + silu(k) silu(v)^T``, ``o = S^T silu(q)``. ``o`` [tokens, H * DV] float32; S in ``state``."""
+    if state.shape[1] < H * D * DV:
+        raise KernelError("decay_scan: the state rows are too short")
+    _check(_fn("stride_decay_scan")(
+        *_decay_args(proj, q_off, k_off, v_off, logit, bias, H, D, DV, o), _opt(logit, "logit", torch.float32),
+        _opt(bias, "bias", torch.float32), _opt(fade, "fade", torch.float32), float(q_scale), float(inv_tau), _dev(o, "o", torch.float32),
+        *_state_rows(state), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
+        _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype), _stream()), "decay_scan")
+
+
+def decay_chunks_scratch_floats(num_seqs: int, max_q_len: int, H: int, D: int, DV: int) -> int:
+    return num_seqs * -(-max_q_len // DECAY_CHUNK) * H * D * (DV + 1)
+
+
+def decay_chunks(proj, q_off: int, k_off: int, v_off: int, logit, bias, powers, q_scale: float, inv_tau: float, o, state, q_start, q_len,
+                 state_slot, num_seqs: int, H: int, D: int, DV: int, max_q_len: int, scratch) -> None:
+    """``decay_scan`` with the chunks of every portion side by side (sums in another order). ``powers`` (float32 [H, 65]):
+    decay^0 .. decay^64 in place of ``fade``; ``logit`` is overwritten; ``scratch``: ``decay_chunks_scratch_floats``."""
+    if state.shape[1] < H * D * DV or scratch.numel() < decay_chunks_scratch_floats(num_seqs, max_q_len, H, D, DV):
+        raise KernelError("decay_chunks: the state rows or the scratch are too short")
+    if powers is not None and powers.shape != (H, DECAY_CHUNK + 1):
+        raise KernelError("decay_chunks: powers must hold decay^0 .. decay^64 per head")
+    _check(_fn("stride_decay_chunks")(
+        *_decay_args(proj, q_off, k_off, v_off, logit, bias, H, D, DV, o), _opt(logit, "logit", torch.float32),
+        _opt(bias, "bias", torch.float32), _opt(powers, "powers", torch.float32), float(q_scale), float(inv_tau),
+        _dev(o, "o", torch.float32), *_state_rows(state), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
+        _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype), -(-max_q_len // DECAY_CHUNK),
+        _dev(scratch, "scratch", torch.float32), _stream()), "decay_chunks")
+
+
+# ------------------------------------------------------------ a residual stream in several copies
+def copies_step(src, dst, delta, scale, mix, out_w, in_w, norm_w, eps: float, out=None, sum_out=None, rows=None, copies: int = 0) -> None:
+    """The write behind one sublayer and the read in front of the next. ``src`` float32 [tokens, copies * hidden] (or [tokens,
+    hidden]: all copies equal). With ``delta``: every copy ``b`` becomes ``sum_a mix[a, b] X_a + out_w[b] * scale * delta``.
+    ``dst`` (or None) receives the copies; ``u = sum_a in_w[a] X_a`` (``in_w`` None: the plain sum) goes to ``sum_out`` (float32)
+    and, as an RMS norm with ``norm_w`` and ``eps``, to ``out``. ``rows`` (int32): only these source rows, into row i of the outputs."""
+    result = out if out is not None else sum_out
+    if dst is not None:
+        hidden = dst.shape[1] // copies
+    elif result is not None:
+        hidden = result.shape[1]
+    else:
+        raise KernelError("copies_step: nothing to produce")
+    n_src = src.shape[1] // hidden
+    num_rows = rows.shape[0] if rows is not None else src.shape[0]
+    if src.shape[1] != n_src * hidden or (dst is not None and dst.shape != (src.shape[0], copies * hidden)):
+        raise KernelError("copies_step: the copies must be [tokens, copies * hidden]")
+    for name, t in (("out", out), ("sum_out", sum_out)):
+        if t is not None and t.shape != (num_rows, hidden):
+            raise KernelError(f"copies_step: {name} must be [rows, hidden]")
+    if (norm_w is None) != (out is None) or (delta is not None and (delta.shape != (src.shape[0], hidden) or (out is not None and out.dtype != delta.dtype))):
+        raise KernelError("copies_step: a norm needs an output of the delta's element type")
+    for t, count in ((scale, hidden), (mix, copies * copies), (out_w, copies), (in_w, copies), (norm_w, hidden)):
+        if t is not None and t.numel() != count:
+            raise KernelError("copies_step: a coefficient has the wrong size")
+    dtype = delta.dtype if delta is not None else out.dtype if out is not None else torch.float32
+    _check(_fn("stride_copies_step")(
+        _dev(src, "src", torch.float32), n_src, _opt(dst, "dst", torch.float32), _opt(delta, "delta"), _opt(scale, "scale", torch.float32),
+        _opt(mix, "mix", torch.float32), _opt(out_w, "out_w", torch.float32), _opt(in_w, "in_w", torch.float32),
+        _opt(norm_w, "norm_w", torch.float32), float(eps), _opt(out, "out"), _opt(sum_out, "sum_out", torch.float32),
+        _opt(rows, "rows", torch.int32), num_rows, copies, hidden, _code(dtype), _stream()), "copies_step")
 
 
 # ------------------------------------------------------------ short convolution with head norms
@@ -575,17 +692,36 @@ def conv_head_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start
         raise KernelError("conv_head_norm: raw and out must agree in rows and element type")
     _check(_fn("stride_conv_head_norm")(
         _dev(raw, "raw"), raw.shape[1], _dev(out, "out"), out.shape[1], _opt(conv_w, "conv_w", torch.float32), taps,
-        _opt(state, "state", torch.float32), 0 if state is None else state.shape[1], int(tail_off),
+        *(_state_rows(state) if state is not None else (None, 0)), int(tail_off),
         _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32), _dev(state_slot, "state_slot", torch.int32),
         _opt(wq, "wq", torch.float32), _opt(wk, "wk", torch.float32), float(eps), _opt(slot_mapping, "slot_mapping", torch.int32),
         _opt(k_pages, "k_pages", raw.dtype), _opt(v_pages, "v_pages", raw.dtype), raw.shape[0], nq, nkv, hd, vd, page_size,
         _code(raw.dtype), _stream()), "conv_head_norm")
 
 
+def conv_row_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start, state_slot, positions, wq, wk, eps: float, temp_coef: float,
+                  temp_every: int, slot_mapping, k_pages, v_pages, nq: int, nkv: int, hd: int, vd: int, page_size: int) -> None:
+    """``conv_head_norm`` with one RMS norm over a token's whole query projection (weight ``wq`` [nq * hd]) and one over its whole
+    key projection (``wk`` [nkv * hd]) in place of a norm a head, and queries multiplied by
+    ``1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)`` at position p (``temp_every`` 0: not)."""
+    taps = 1 if conv_w is None else conv_w.shape[0]
+    if out.dtype != raw.dtype or out.shape[0] != raw.shape[0]:
+        raise KernelError("conv_row_norm: raw and out must agree in rows and element type")
+    if (wq is not None and wq.numel() != nq * hd) or (wk is not None and wk.numel() != nkv * hd):
+        raise KernelError("conv_row_norm: the norms' weights must have the projections' widths")
+    _check(_fn("stride_conv_row_norm")(
+        _dev(raw, "raw"), raw.shape[1], _dev(out, "out"), out.shape[1], _opt(conv_w, "conv_w", torch.float32), taps,
+        *(_state_rows(state) if state is not None else (None, 0)), int(tail_off),
+        _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32), _dev(state_slot, "state_slot", torch.int32),
+        _dev(positions, "positions", torch.int32), _opt(wq, "wq", torch.float32), _opt(wk, "wk", torch.float32), float(eps), float(temp_coef),
+        int(temp_every), _opt(slot_mapping, "slot_mapping", torch.int32), _opt(k_pages, "k_pages", raw.dtype),
+        _opt(v_pages, "v_pages", raw.dtype), raw.shape[0], nq, nkv, hd, vd, page_size, _code(raw.dtype), _stream()), "conv_row_norm")
+
+
 def conv_tail(raw, state, tail_off: int, q_start, q_len, state_slot, num_seqs: int, channels: int, taps: int) -> None:
     """Moves every request's convolution tail on by the step's rows of ``raw`` (its first ``channels`` columns)."""
     _check(_fn("stride_conv_tail")(
-        _dev(raw, "raw"), raw.shape[1], _dev(state, "state", torch.float32), state.shape[1], int(tail_off),
+        _dev(raw, "raw"), raw.shape[1], *_state_rows(state), int(tail_off),
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32),
         int(num_seqs), int(channels), int(taps), _code(raw.dtype), _stream()), "conv_tail")
 
@@ -1322,13 +1458,22 @@ def linear(x, weight, out) -> None:
 
 
 # -------------------------------------------------------------------- attention
+def _rel_args(rel, nq: int) -> tuple:
+    if rel is None:
+        return None, 0
+    if rel.dim() != 2 or rel.shape[0] != nq:
+        raise KernelError("rel must hold one row per query head")
+    return _dev(rel, "rel", torch.float32), rel.shape[1]
+
+
 def paged_attention(q, q_stride: int, out, k_pages, v_pages, block_table, seq_of_token, positions, nq: int, nkv: int,
                     hd: int, page_size: int, scale: float, window: int = 0, softcap: float = 0.0, sinks=None, slopes=None,
-                    vd: int | None = None) -> None:
+                    vd: int | None = None, rel=None) -> None:
     """Attention of every token in the flat batch over its request's pages.
     ``q`` holds head h of token t at ``q[t * q_stride + h * hd]``. ``softcap`` c > 0 caps the scaled scores at
     c tanh(s / c); ``sinks`` (float32 [nq]) adds exp(sink) of the head to the softmax's denominator; ``slopes`` (float32
-    [nq]) takes slope_h times the key's distance off every score; ``vd`` is the values' width where it is not ``hd``."""
+    [nq]) takes slope_h times the key's distance off every score; ``vd`` is the values' width where it is not ``hd``;
+    ``rel`` (float32 [nq, n]) adds ``rel[h, min(distance, n - 1)]`` to every score of head h."""
     tokens = out.shape[0]
     vd = hd if vd is None else int(vd)
     if out.shape[1] != nq * vd or k_pages.shape[-1] != hd or v_pages.shape[-1] != vd:
@@ -1337,7 +1482,8 @@ def paged_attention(q, q_stride: int, out, k_pages, v_pages, block_table, seq_of
         _dev(q, "q"), q_stride, _dev(out, "out"), _dev(k_pages, "k_pages"), _dev(v_pages, "v_pages"),
         _dev(block_table, "block_table", torch.int32), block_table.shape[1], _dev(seq_of_token, "seq_of_token", torch.int32),
         _dev(positions, "positions", torch.int32), tokens, nq, nkv, hd, vd, page_size, float(scale), int(window), float(softcap),
-        _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), _code(q.dtype), _stream()), "paged_attention")
+        _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), _code(q.dtype), _stream()),
+        "paged_attention")
 
 
 def fast_attention_supported(dtype, nq: int, nkv: int, hd: int) -> bool:
@@ -1358,21 +1504,21 @@ def decode_scratch_floats(tokens: int, nq: int, nkv: int, hd: int, max_context: 
 
 def paged_attention_decode(q, q_stride: int, out, k_pages, v_pages, block_table, seq_of_token, positions, scratch, nq: int,
                            nkv: int, hd: int, page_size: int, scale: float, window: int, max_context: int, softcap: float = 0.0,
-                           sinks=None, slopes=None, gate_col: int = -1) -> None:
+                           sinks=None, slopes=None, gate_col: int = -1, rel=None) -> None:
     """Attention for single decoded tokens (one query per row), split over the keys;
     ``scratch`` (float32, zero when first used) holds the ticket counters and the
     partial results of the splits. ``softcap``, ``sinks`` and ``slopes`` as for ``paged_attention``. ``gate_col`` >= 0: columns
     ``gate_col .. gate_col + nq - 1`` of a row of ``q`` hold one logit per head, and head h's output leaves the kernel
-    multiplied by the sigmoid of its logit."""
+    multiplied by the sigmoid of its logit. ``rel`` as for ``paged_attention``."""
     tokens = out.shape[0]
     if out.shape[1] != nq * hd:
         raise KernelError("attention output has the wrong width")
-    _check(_fn("stride_paged_decode_attention_gated")(
+    _check(_fn("stride_paged_decode_attention_biased")(
         _dev(q, "q", torch.bfloat16), q_stride, _dev(out, "out", torch.bfloat16), _dev(k_pages, "k_pages", torch.bfloat16),
         _dev(v_pages, "v_pages", torch.bfloat16), k_pages.shape[0], _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], _dev(seq_of_token, "seq_of_token", torch.int32), _dev(positions, "positions", torch.int32),
         _dev(scratch, "scratch", torch.float32), scratch.numel(), tokens, nq, nkv, hd, page_size, float(scale), int(window),
-        float(softcap), _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), int(gate_col), int(max_context),
+        float(softcap), _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), int(gate_col), int(max_context),
         _tc_buffers(q.device, 0)["status"].data_ptr(), _stream()),
         "paged_attention_decode")
 
@@ -1382,7 +1528,7 @@ TC_ATTENTION = _os.environ.get("STRIDE_B200_TC_ATTENTION", "1") != "0"
 
 def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_table, q_start, q_len, ctx_len, num_seqs: int,
                                nq: int, nkv: int, hd: int, page_size: int, scale: float, window: int, softcap: float = 0.0,
-                               sinks=None, slopes=None) -> bool:
+                               sinks=None, slopes=None, rel=None) -> bool:
     """The tcgen05 version of ``paged_attention_prefill`` (same arguments). Returns False
     when it does not take the sizes; the caller then uses the mma.sync kernel."""
     tokens = out.shape[0]
@@ -1394,7 +1540,7 @@ def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_ta
         _dev(v_pages, "v_pages", torch.bfloat16), k_pages.shape[0], _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
         _dev(ctx_len, "ctx_len", torch.int32), num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), float(softcap),
-        _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), st["status"].data_ptr(), _stream())
+        _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), st["status"].data_ptr(), _stream())
     if code == -2:
         return False
     _check(code, "paged_attention_prefill_tc")
@@ -1403,7 +1549,7 @@ def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_ta
 
 def paged_attention_prefill(q, q_stride: int, out, k_pages, v_pages, block_table, q_start, q_len, ctx_len, num_seqs: int,
                             nq: int, nkv: int, hd: int, page_size: int, scale: float, window: int, softcap: float = 0.0,
-                            sinks=None, slopes=None) -> None:
+                            sinks=None, slopes=None, rel=None) -> None:
     """Attention for the first ``num_seqs`` requests of the step (portions of any
     length), which own the rows of ``out``. ``softcap`` and ``sinks`` as for ``paged_attention``."""
     tokens = out.shape[0]
@@ -1414,7 +1560,7 @@ def paged_attention_prefill(q, q_stride: int, out, k_pages, v_pages, block_table
         _dev(v_pages, "v_pages", torch.bfloat16), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(ctx_len, "ctx_len", torch.int32),
         num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), float(softcap), _opt(sinks, "sinks", torch.float32),
-        _opt(slopes, "slopes", torch.float32), _stream()), "paged_attention_prefill")
+        _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), _stream()), "paged_attention_prefill")
 
 
 # --------------------------------------------------------------------- sampling

@@ -31,6 +31,14 @@ Spec params, all optional:
 * ``qk_norm`` ``weighted``: every query and key head goes through an RMS norm with a weight of the head's size shared by the
   heads (tensors ``q.norm``, ``k.norm``; ``norm_eps`` inside the root), after the convolution. One kernel does the
   convolution, the norms and the write into the pages; a second one moves the tails on.
+* ``qk_norm`` ``rows``: an RMS norm over a token's whole query projection and one over its whole key projection (tensors ``q.norm``
+  [heads * head_dim], ``k.norm`` [kv_heads * head_dim]), after the convolution, before the heads are told apart.
+* ``query_factor`` (coef, every), with ``qk_norm`` ``rows``: the query at position p is multiplied by
+  ``1 + coef ln(floor((p + 1) / every) + 1)`` after its norm.
+* ``distance_table`` (buckets B, largest D, positions): a tensor ``rel`` [B, heads]; ``rel[bucket(i - j), h]`` is added to the scaled score
+  of query i and key j. Distances below B / 2 have a bucket each, the others share the rest logarithmically up to D, beyond which
+  all fall into the last (the bucketing of Raffel et al., "Exploring the Limits of Transfer Learning with a Unified Text-to-Text
+  Transformer"). The kernels get the number of every distance from 0 to D, worked out when the tensor is bound.
 * ``sinks`` ``zero``: no tensor; every head's denominator gains exp(0) = 1.
 * ``borrowed_kv``: the mixer has no key and value projections and reads the pages of the cache slot it is given, which
   another layer's mixer of the same shape writes.
@@ -43,11 +51,31 @@ stored order back.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..csrc import ops
 from .runtime import sequence_slots
 from .base import CacheRequest, Mixer, Projection, StateRequest, TensorDecl, build_part, register_part
+
+
+def distance_bucket(n: int, buckets: int, largest: int) -> int:
+    """The bucket of distance n: n itself below half, else ``half + floor(log_(largest / half)(n / half) * (buckets - half))``, at
+    most the last. The floor is taken exactly, in integers: ``log >= r / m`` is ``n^m half^r >= largest^r half^m``."""
+    half = buckets // 2
+    if n < half:
+        return n
+    if n >= largest:
+        return buckets - 1
+    m = buckets - half
+    r = min(m, max(0, math.floor(math.log(n / half) / math.log(largest / half) * m)))
+    reaches = lambda r: n ** m * half ** r >= largest ** r * half ** m
+    while r > 0 and not reaches(r):
+        r -= 1
+    while r < m and reaches(r + 1):
+        r += 1
+    return min(buckets - 1, half + r)
 
 
 class PagedAttention(Mixer):
@@ -73,6 +101,17 @@ class PagedAttention(Mixer):
         self.zero_sinks = p.get("sinks") == "zero"
         self.has_sinks, self.gated = bool(p.get("sinks", False)) and not self.zero_sinks, bool(p.get("output_gate", False))
         self.taps, self.weighted_qk = int(p.get("conv", 0)), p.get("qk_norm") == "weighted"
+        self.row_norm = p.get("qk_norm") == "rows"
+        self.q_coef, self.q_every = p.get("query_factor") or (0.0, 0)
+        if self.q_every and not self.row_norm:
+            raise ValueError("a factor on the queries goes with norms over whole projections")
+        self.buckets = self.largest = 0
+        if p.get("distance_table"):
+            self.buckets, self.largest, self.table_positions = (int(v) for v in p["distance_table"])
+            if self.buckets < 2 or self.largest <= self.buckets // 2:
+                raise ValueError(f"a distance table needs its number of buckets (read off the checkpoint, or given in the configuration) and a "
+                                 f"largest distance beyond half of it, got {self.buckets} and {self.largest}")
+        self.rel = self.stored_rel = None
         self.short_names = p.get("names") == "short"
         self.vd = int(p.get("value_dim", self.hd))
         self.unit_qk, self.unit_v = p.get("qk_norm") == "unit", p.get("v_norm") == "unit"
@@ -87,10 +126,10 @@ class PagedAttention(Mixer):
         # what the plain path (projection, then the position part's rotation and cache write) cannot do goes through
         # the head-norm kernel, which adds the bias, norms and writes the pages itself when there is no rotation
         self.plain_position = s.position is None or s.position.kind == "none"
-        self.conv_path = self.taps > 0 or self.weighted_qk
+        self.conv_path = self.taps > 0 or self.weighted_qk or self.row_norm
         if self.conv_path and (self.unit_qk or self.unit_v or self.borrows or s.bias or self.head_gate or not self.plain_position
                                or not self.short_names or self.taps > 16):
-            raise ValueError("a convolution or weighted head norms go with no rotation, no biases, no unit norms, no borrowed pages, "
+            raise ValueError("a convolution, weighted head norms or norms over whole projections go with no rotation, no biases, no unit norms, no borrowed pages, "
                              "no per-head gate, short tensor names and at most 16 taps")
         self.own_prepare = self.unit_qk or self.unit_v or self.vd != self.hd or self.borrows or self.conv_path
         if self.own_prepare and not self.plain_position and (self.vd != self.hd or self.borrows):
@@ -147,6 +186,10 @@ class PagedAttention(Mixer):
             d.update({f"{p}{n}.conv": TensorDecl((rows, self.taps), "vector") for n, rows in (("q", self.q_dim), ("k", self.kv_dim), ("v", self.v_dim))})
         if self.weighted_qk:
             d.update({f"{p}{n}.norm": TensorDecl((self.hd,), "vector") for n in "qk"})
+        if self.row_norm:
+            d.update({p + "q.norm": TensorDecl((self.q_dim,), "vector"), p + "k.norm": TensorDecl((self.kv_dim,), "vector")})
+        if self.buckets:
+            d[p + "rel"] = TensorDecl((self.buckets, self.nq), "vector")
         d.update(self.position.declare())          # a position encoding may have tensors of its own
         return d
 
@@ -177,6 +220,7 @@ class PagedAttention(Mixer):
             self.w_gate = self._reorder(weights[w["g"]]) if self.values_are_keys else weights[w["g"]]
         if self.has_sinks:
             self.sinks = weights[w["sink"]]
+        self._bind_rel(weights)
         self.position.bind(weights)
 
     def _bind_own(self, weights, w, b):
@@ -202,9 +246,19 @@ class PagedAttention(Mixer):
         if self.taps:
             # [taps, channels]: a tap's weights of neighbouring channels side by side, as the kernel reads them
             self.conv_w = torch.cat([weights[f"{p}{n}.conv"] for n in "qkv"], dim=0).t().contiguous()
-        if self.weighted_qk:
+        if self.weighted_qk or self.row_norm:
             self.wq_norm, self.wk_norm = weights[p + "q.norm"], weights[p + "k.norm"]
+        self._bind_rel(weights)
         self.position.bind(weights)
+
+    def _bind_rel(self, weights):
+        """The distance table as the kernels read it: [heads, distances], the last entry for every farther key."""
+        if not self.buckets:
+            return
+        self.stored_rel = weights[self.spec.prefix + "rel"]
+        distances = min(self.largest, self.table_positions - 1) + 1
+        index = torch.tensor([distance_bucket(n, self.buckets, self.largest) for n in range(distances)], device=self.stored_rel.device)
+        self.rel = self.stored_rel.index_select(0, index).t().contiguous()
 
     def _named_own(self):
         w, b = self._names()
@@ -225,8 +279,10 @@ class PagedAttention(Mixer):
             q, k = self.q_dim, self.q_dim + self.kv_dim
             stored = self.conv_w.t()
             out.update({p + "q.conv": stored[:q], p + "k.conv": stored[q:k], p + "v.conv": stored[k:]})
-        if self.weighted_qk:
+        if self.weighted_qk or self.row_norm:
             out.update({p + "q.norm": self.wq_norm, p + "k.norm": self.wk_norm})
+        if self.buckets:
+            out[p + "rel"] = self.stored_rel
         out.update(self.position.named_tensors())
         return out
 
@@ -250,6 +306,8 @@ class PagedAttention(Mixer):
             out[w["sink"]] = self.sinks
         if self.has_output_bias:
             out[b["o"]] = self.output_bias
+        if self.buckets:
+            out[self.spec.prefix + "rel"] = self.stored_rel
         out.update(self.position.named_tensors())
         return out
 
@@ -310,12 +368,22 @@ class PagedAttention(Mixer):
 
 
     def _convolve_and_store(self, raw, qkv, ctx, cache, tokens):
-        """Convolution over time, weighted head norms and the pages in one kernel; then the tails of the step's requests move on."""
+        """Convolution over time, the norms of queries and keys and the pages in one kernel; then the tails of the step's requests move on."""
         slots = ctx.slot_mapping[cache.group][:tokens] if cache.writes else None
         state = cache.state if self.taps > 1 else None
+        if self.row_norm:
+            ops.conv_row_norm(raw, qkv, self.conv_w, state, 0, ctx.seq_of_token[:tokens], ctx.q_start, ctx.state_slot, ctx.positions[:tokens],
+                              self.wq_norm, self.wk_norm, self.norm_eps, self.q_coef, self.q_every, slots,
+                              cache.k_pages if cache.writes else None, cache.v_pages if cache.writes else None, self.nq, self.nkv, self.hd,
+                              self.vd, cache.page_size)
+            self._move_tails(raw, state, ctx)
+            return
         ops.conv_head_norm(raw, qkv, self.conv_w, state, 0, ctx.seq_of_token[:tokens], ctx.q_start, ctx.state_slot, self.wq_norm, self.wk_norm,
                            self.norm_eps, slots, cache.k_pages if cache.writes else None, cache.v_pages if cache.writes else None, self.nq,
                            self.nkv, self.hd, self.vd, cache.page_size)
+        self._move_tails(raw, state, ctx)
+
+    def _move_tails(self, raw, state, ctx):
         if state is not None:
             ops.conv_tail(raw, state, 0, ctx.q_start, ctx.q_len, ctx.state_slot, sequence_slots(ctx), self.qkv_dim, self.taps)
 
@@ -358,12 +426,12 @@ class PagedAttention(Mixer):
         if not self._fast:
             # the exact kernel: the whole 32-bit path, and bfloat16 sizes the tensor-core kernels refuse
             ops.paged_attention(qkv, self.qkv_dim, attn, cache.k_pages, cache.v_pages, table, ctx.seq_of_token[:tokens],
-                                ctx.positions[:tokens], *geometry, self.softcap, self.sinks, self.slopes, self.vd)
+                                ctx.positions[:tokens], *geometry, self.softcap, self.sinks, self.slopes, self.vd, self.rel)
             return tokens
         split = min(ctx.decode_tail_start, tokens)          # portions before, single decoded tokens after
         if split > 0:
             args = (qkv[:split], self.qkv_dim, attn[:split], cache.k_pages, cache.v_pages, table, ctx.q_start, ctx.q_len,
-                    ctx.ctx_len, ctx.decode_tail_seq, *geometry, self.softcap, self.sinks, self.slopes)
+                    ctx.ctx_len, ctx.decode_tail_seq, *geometry, self.softcap, self.sinks, self.slopes, self.rel)
             # tcgen05 kernel first; the mma.sync kernel takes what it refuses (odd page sizes)
             if not (ops.TC_ATTENTION and ops.paged_attention_prefill_tc(*args)):
                 ops.paged_attention_prefill(*args)
@@ -373,7 +441,7 @@ class PagedAttention(Mixer):
             ops.paged_attention_decode(qkv[split:tokens], self.qkv_dim, attn[split:tokens], cache.k_pages, cache.v_pages, table,
                                        ctx.seq_of_token[split:tokens], ctx.positions[split:tokens], scratch, *geometry,
                                        ctx.context_bound, self.softcap, self.sinks, self.slopes,
-                                       self.q_dim + self.kv_cols if self.fused_gate else -1)
+                                       self.q_dim + self.kv_cols if self.fused_gate else -1, self.rel)
             return split if self.fused_gate else tokens
         return tokens
 

@@ -6,7 +6,8 @@ the compute dtype and returned in float32; a head whose spec names no tensor sha
 (python/stride_worker/model.py:127-130, 322-341). An architecture that scales its embedding, adds a bias to its
 head registers another kind; the model itself does not change. ``lookup`` with the param ``sinusoid`` b adds the fixed
 position vector of Vaswani et al., "Attention Is All You Need", in neighbouring pairs: entry 2i gets sin(p b^(-2i / hidden)),
-entry 2i + 1 the cosine of the same angle, formed in float64 on the device. A ``linear`` head whose spec gives the param
+entry 2i + 1 the cosine of the same angle, formed in float64 on the device; with ``scale`` f the row is multiplied by f; with
+``positions`` (name, count) a learned vector per position, row p of the tensor ``name`` [count, hidden], is added (not scaled). A ``linear`` head whose spec gives the param
 ``softcap`` c caps its logits at c tanh(logits / c).
 """
 
@@ -20,6 +21,9 @@ class LookupEmbedding(Embedding):
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.weight = None
+        self.scale = float(dict(spec.params).get("scale", 1.0))
+        self.pos_name, self.pos_count = dict(spec.params).get("positions") or (None, 0)
+        self.pos = None
         base = dict(spec.params).get("sinusoid")
         self.freq = None
         if base:
@@ -28,20 +32,25 @@ class LookupEmbedding(Embedding):
             self.freq = (float(base) ** (-2.0 * pairs / spec.hidden)).to(runtime.device)
 
     def declare(self):
-        return {self.spec.name: TensorDecl((self.spec.vocab, self.spec.hidden))}
+        d = {self.spec.name: TensorDecl((self.spec.vocab, self.spec.hidden))}
+        if self.pos_name:
+            d[self.pos_name] = TensorDecl((self.pos_count, self.spec.hidden))
+        return d
 
     def bind(self, weights):
         self.weight = weights[self.spec.name]
+        self.pos = weights[self.pos_name] if self.pos_name else None
 
     def named_tensors(self):
-        return {self.spec.name: self.weight}
+        return {self.spec.name: self.weight, **({self.pos_name: self.pos} if self.pos_name else {})}
 
     def table(self):
         return self.weight
 
     def forward(self, ctx, out):
         tokens = out.shape[0]
-        ops.embed_gather(ctx.token_ids[:tokens], ctx.seq_of_token[:tokens], self.weight, out)
+        ops.embed_gather(ctx.token_ids[:tokens], ctx.seq_of_token[:tokens], self.weight, out, self.scale, self.pos,
+                         ctx.positions[:tokens] if self.pos is not None else None)
         if self.freq is not None:
             ops.add_sinusoid(out, None, ctx.positions[:tokens], ctx.seq_of_token[:tokens], self.freq)
 

@@ -18,6 +18,7 @@ import torch
 from ..csrc import ops
 from ..weights import check_source, load_weights
 from .base import build_part
+from .copies import CopiedStream
 from .runtime import ResidualStream, Runtime
 
 
@@ -31,6 +32,9 @@ class DecoderModel:
         self.final_norm = build_part("norm", spec.final_norm, runtime)
         self.head = build_part("head", spec.head_spec(), runtime)
         self.pass_input = build_part("pass_input", spec.pass_input, runtime) if getattr(spec, "pass_input", None) is not None else None
+        self.copies = int(getattr(spec, "copies", 0))       # the residual stream in this many copies; 0: one plain stream
+        if self.copies and self.pass_input is not None:
+            raise ValueError("a pass input does not go with a residual stream in several copies")
         self.schedule = tuple(spec.schedule)
         for e in self.schedule:
             if not 0 <= e.layer < len(self.layers):
@@ -106,7 +110,7 @@ class DecoderModel:
         if self.caches is None:
             raise RuntimeError("the model has no cache attached")
         tokens = ctx.num_tokens
-        stream = ResidualStream(self.rt, tokens, self.hidden)
+        stream = CopiedStream(self.rt, tokens, self.hidden, self.copies) if self.copies else ResidualStream(self.rt, tokens, self.hidden)
         self.embedding.forward(ctx, stream.residual)
         for state in self._states():        # a request that starts in this step finds its state slots at zero
             ops.zero_fresh_state(state, ctx.state_slot, ctx.q_start, ctx.q_len, ctx.positions)
