@@ -544,8 +544,32 @@ def compare_configs_netusun(name: str, layers: int):
     return ours, llama
 
 
+# Layer sizes for `--compare dopudra`: layers cycle constant-decay memory, constant-decay memory, parallel (attention behind a
+# convolution with a distance table, beside a memory with channel decays), each with the feed-forward without a gate; four copies of
+# the residual stream. Attention of the Llama decoder's head count, grouping and head size; memories of the size of the Migelix
+# design's; the two matrices of the feed-forward hold as many weights as the gated unit's three.
+def compare_configs_dopudra(name: str, layers: int):
+    """(Dopudra config.json, Llama config.json) of one size."""
+    size = MIGELIX_SIZES[name]
+    _migelix, llama = compare_configs_migelix(size, layers)
+    memory = {"heads": size["delta_heads"], "dim": size["delta_dim"], "vdim": size["delta_dim"]}
+    left = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5, "conv": 4,
+            "bias_max": 256, "buckets": 32, "q_temp": {"coef": 0.1, "every": 512}}
+    lightning = dict(memory, decay=[1.0 - 2.0 ** (-2.0 - 8.0 * h / memory["heads"]) for h in range(memory["heads"])])
+    parallel = {"left": left, "right": dict(memory, tau=16.0, decay_rank=16), "left_scale": 1.0, "right_scale": 1.0}
+    mlp = {"kind": "dense", "ff": size["ff"] * 3 // 2}
+    entries = [{"type": "parallel", "mixer": parallel, "mlp": mlp} if i % 3 == 2 else {"type": "lightning", "mixer": lightning, "mlp": mlp}
+               for i in range(layers)]
+    ours = {"architecture": "Dopudra", "width": size["width"], "vocab": size["vocab"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "streams": 4, "max_positions": 8192, "layers": entries}
+    llama["tie_word_embeddings"] = False        # a head of its own, as Dopudra has
+    return ours, llama
+
+
 def _compared(design: str, size_name: str, layers: int):
     """The two configurations of ``--compare design`` at one size."""
+    if design == "dopudra":
+        return compare_configs_dopudra(size_name, layers)
     if design == "netusun":
         return compare_configs_netusun(size_name, layers)
     if design == "migelix":
@@ -611,9 +635,10 @@ def _measure_design(config: dict, batch: int, context: int, prompt_len: int, ste
 
 
 def run_compare(args) -> dict:
-    """``--compare nidilix | migelix | tutizen | netusun``: prefill and decode throughput of that design at a few layer sizes
+    """``--compare nidilix | migelix | tutizen | netusun | dopudra``: prefill and decode throughput of that design at a few layer sizes
     beside the Llama decoder at equal size, with the device time per class of kernel; Netusun also beside Tutizen, the design
-    whose layers are closest to its own (the same mixture, a norm on a sublayer's output). Not the headline workload."""
+    whose layers are closest to its own (the same mixture, a norm on a sublayer's output), and Dopudra beside Migelix (attention
+    beside a matrix memory, decayed memories). Not the headline workload."""
     layers = args.layers or 6
     sizes = [s for s in args.compare_sizes.split(",") if s]
     result = {"mode": "compare", "design": args.compare, "beside": "llama", "layers": layers, "dtype": "bf16", "data": "synthetic", "sizes": {}}
@@ -625,6 +650,9 @@ def run_compare(args) -> dict:
         if args.compare == "netusun":
             closest = compare_configs_tutizen(TUTIZEN_SIZES[name], layers)[0]
             result["sizes"][name]["tutizen"] = _measure_design(closest, args.batch, args.context, 2048, args.steps, args.warmup)
+        if args.compare == "dopudra":
+            closest = compare_configs_migelix(MIGELIX_SIZES[name], layers)[0]
+            result["sizes"][name]["migelix"] = _measure_design(closest, args.batch, args.context, 2048, args.steps, args.warmup)
     return result
 
 
@@ -724,7 +752,7 @@ def main(argv=None) -> int:
     p.add_argument("--no-breakdown", action="store_true", help="skip the per-class times of one decode step and the prefill")
     p.add_argument("--profile", choices=["decode", "prefill"], default=None,
                    help="run a few eager steps of one kind for a profiler instead of measuring")
-    p.add_argument("--compare", choices=["nidilix", "migelix", "tutizen", "netusun"], default=None,
+    p.add_argument("--compare", choices=["nidilix", "migelix", "tutizen", "netusun", "dopudra"], default=None,
                    help="instead of the headline workload: this design's prefill and decode beside the Llama decoder at equal size")
     p.add_argument("--compare-sizes", default="w1024,w2048", help="comma-separated names of the sizes to compare")
     args = p.parse_args(argv)

@@ -59,7 +59,7 @@ chunk_decay_kernel(const ChunkArgs p) {
     if (nt <= 0 || c >= HD) return;
     float* at = p.cum + static_cast<size_t>(p.q_start[seq] + first) * HD + c;
     const float b = p.bias[c];
-    float sum = 0.f;
+    double sum = 0.0;       // rounded once per token: differences of these sums are the exponents of whole decays
     for (int t0 = 0; t0 < nt; t0 += 8) {
         float l[8];
 #pragma unroll
@@ -70,7 +70,7 @@ chunk_decay_kernel(const ChunkArgs p) {
         for (int u = 0; u < 8; ++u)
             if (t0 + u < nt) {
                 sum += l[u];
-                at[static_cast<size_t>(t0 + u) * HD] = sum;
+                at[static_cast<size_t>(t0 + u) * HD] = static_cast<float>(sum);
             }
     }
 }
