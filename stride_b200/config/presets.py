@@ -1,4 +1,4 @@
-"""Named shapes, as config.json dictionaries (Llama 3, and two of the Nidilix design): the tiny shapes used
+"""Named shapes, as config.json dictionaries (Llama 3, two of the Nidilix design, a tiny one of the Netusun and of the Dopudra design): the tiny shapes used
 for correctness runs (tiny-d has the head size and widths that the tensor-core
 kernels take) and the 8B / 3B / 70B shapes used for measurements. The
 reference keeps such presets in crates/stride-model/src/presets.rs:73-91."""
@@ -59,7 +59,21 @@ def _netusun_tiny() -> dict:
             "loop": {"start": 0, "stop": 2, "times": 2}}
 
 
+def _dopudra_tiny() -> dict:
+    """Three layers on two copies of the residual stream: a memory with a constant decay, attention beside a memory with channel
+    decays, another constant one; two with a feed-forward."""
+    left = {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "scale": 32 ** -0.5, "conv": 4, "bias_max": 64, "buckets": 16,
+            "q_temp": {"coef": 0.2, "every": 32}}
+    right = {"heads": 2, "dim": 32, "vdim": 64, "tau": 12.0, "decay_rank": 8}
+    layers = [{"type": "lightning", "mixer": {"heads": 2, "dim": 32, "vdim": 64, "decay": [0.75, 0.99]}, "mlp": None},
+              {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.1, "right_scale": 0.8}, "mlp": {"kind": "dense", "ff": 320}},
+              {"type": "lightning", "mixer": {"heads": 4, "dim": 16, "vdim": 16, "decay": [0.5, 0.9, 0.98, 0.999]}, "mlp": {"kind": "dense", "ff": 192}}]
+    return {"architecture": "Dopudra", "width": 128, "vocab": 384, "streams": 2, "max_positions": 512, "norm": {"eps": 1e-5},
+            "embedding": {"scale": 0.8}, "layers": layers}
+
+
 PRESETS = {
+    "dopudra-tiny": _dopudra_tiny(),
     "netusun-tiny": _netusun_tiny(),
     "nidilix-tiny": _nidilix(128, 512, "rarb", {"width": 160, "blocks": 5, "conv": 3},
                              {"heads": 4, "dim": 16, "rot_dim": 16, "vdim": 24, "kv_rank": 48, "rot": {"base": 10000.0, "dims": 16},

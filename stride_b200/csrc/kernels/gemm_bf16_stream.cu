@@ -75,6 +75,7 @@ struct RowNorm {
     float* residual;                   // producer (MODE 3): [tokens, n] float32, updated in place
     const float* norm_weight;          // producer: [n]
     float* out_partials;               // producer: [gridDim.x][16]
+    int act;                           // MODE 0: 1 stores relu(product)^2, formed in float32
 };
 
 // NT: token tiles of eight, MT: row tiles of 16 per CTA. MODE 0: bfloat16 output, 1: float32 output, 3: RowNorm
@@ -412,6 +413,10 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                 static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(__fmul_rn(r_new, w_pre[MODE == 3 ? it : 0]));
                 sq_s[token][local] = r_new * r_new;
             } else {
+                if (MODE == 0 && norm.act == 1) {
+                    sum = fmaxf(sum, 0.f);
+                    sum *= sum;
+                }
                 static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(sum);
             }
         }
@@ -561,6 +566,20 @@ extern "C" int stride_gemm_stream_bf16(const void* x, const void* w, void* out, 
                           : stream_gemm::launch_stream<1, 0>(xp, wp, out, tokens, n_out, k, stream, status);
     return out_is_f32 ? stream_gemm::launch_stream<2, 1>(xp, wp, out, tokens, n_out, k, stream, status)
                       : stream_gemm::launch_stream<2, 0>(xp, wp, out, tokens, n_out, k, stream, status);
+}
+
+// The same with relu(.)^2 on the product, formed from the float32 sums: out [tokens, n_out] bf16.
+extern "C" int stride_gemm_stream_relu2(const void* x, const void* w, void* out, int tokens, int n_out, int k, int* status,
+                                        cudaStream_t stream) {
+    if (tokens < 0 || n_out <= 0 || k <= 0) return STRIDE_BAD_ARGUMENT;
+    if (tokens > 16 || k % 8 || (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) % 16) return STRIDE_UNSUPPORTED;
+    if (tokens == 0) return 0;
+    auto xp = static_cast<const __nv_bfloat16*>(x);
+    auto wp = static_cast<const __nv_bfloat16*>(w);
+    stream_gemm::RowNorm norm{};
+    norm.act = 1;
+    if (tokens <= 8) return stream_gemm::launch_stream<1, 0>(xp, wp, out, tokens, n_out, k, stream, status, stream_gemm::QkvEpilogue{}, norm);
+    return stream_gemm::launch_stream<2, 0>(xp, wp, out, tokens, n_out, k, stream, status, stream_gemm::QkvEpilogue{}, norm);
 }
 
 // The projection of queries, keys and values for at most 16 tokens with rotation and cache write in its

@@ -150,8 +150,8 @@ shift_mix_kernel(const T* __restrict__ x, const float* __restrict__ mu, float* _
 // o [tokens, H, DV] float32 -> out [tokens, H * DV] (compute type): o / sqrt(mean(o^2) + eps) * weight * gate.
 // weight [.. ] float32 read at h * w_head_stride + j (0: one weight for all heads). gate_kind 0: sigmoid of float32
 // gate[t * ld_gate + h * DV + j]; 1: silu of a compute-type gate at the same place; 2: sigmoid of a compute-type gate.
-// One warp a (token, head).
-template <typename T>
+// One warp a (token, head); V columns a lane and turn (4 where rows and pointers allow 16-byte accesses).
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, int w_head_stride, const void* __restrict__ gate,
                       int ld_gate, int gate_kind, T* __restrict__ out, int tokens, int H, int DV, float eps) {
@@ -162,20 +162,86 @@ head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ wei
     if (pair >= static_cast<long long>(tokens) * H) return;
     const int t = static_cast<int>(pair / H), h = static_cast<int>(pair % H);
     const float* row = o + (static_cast<size_t>(t) * H + h) * DV;
+    const size_t g0 = static_cast<size_t>(t) * ld_gate + h * DV;
+    struct alignas(V * sizeof(T)) Pack { T v[V]; };
     float ss = 0.f;
-    for (int j = lane; j < DV; j += 32) ss = fmaf(row[j], row[j], ss);
+    for (int j = lane * V; j < DV; j += 32 * V) {
+        alignas(16) float x[V];
+        if constexpr (V == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+        else x[0] = row[j];
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+    }
     ss = warp_sum(ss);
     const float inv = 1.f / sqrtf(ss / static_cast<float>(DV) + eps);
-    for (int j = lane; j < DV; j += 32) {
-        const size_t at = static_cast<size_t>(t) * ld_gate + h * DV + j;
-        const float g = gate_kind == 0   ? sigmoid_f(static_cast<const float*>(gate)[at])
-                        : gate_kind == 1 ? silu_f(to_f32(static_cast<const T*>(gate)[at]))
-                                         : sigmoid_f(to_f32(static_cast<const T*>(gate)[at]));
-        out[(static_cast<size_t>(t) * H + h) * DV + j] = from_f32<T>(row[j] * inv * weight[h * w_head_stride + j] * g);
+    for (int j = lane * V; j < DV; j += 32 * V) {
+        alignas(16) float x[V];
+        alignas(16) float w[V];
+        Pack g, y;
+        if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+            *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(weight + h * w_head_stride + j);
+        } else {
+            x[0] = row[j];
+            w[0] = weight[h * w_head_stride + j];
+        }
+        if (gate_kind) g = *reinterpret_cast<const Pack*>(static_cast<const T*>(gate) + g0 + j);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float z = gate_kind ? to_f32(g.v[e]) : static_cast<const float*>(gate)[g0 + j + e];
+            y.v[e] = from_f32<T>(x[e] * inv * w[e] * (gate_kind == 1 ? silu_f(z) : sigmoid_f(z)));
+        }
+        *reinterpret_cast<Pack*>(out + (static_cast<size_t>(t) * H + h) * DV + j) = y;
     }
 }
 
-// The same for the delta rule, whose pieces carry a memory across by a full matrix: piece_t [z, H, D, D] holds it, piece_s
+// The same with a CTA a (token, head), for heads so wide that a warp would walk them for long (one norm over all heads of a
+// token counts as one head). V columns a thread and turn.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict__ weight, int w_head_stride, const void* __restrict__ gate,
+                           int ld_gate, int gate_kind, T* __restrict__ out, int H, int DV, float eps) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x / H, h = blockIdx.x % H;
+    const float* row = o + (static_cast<size_t>(t) * H + h) * DV;
+    const size_t g0 = static_cast<size_t>(t) * ld_gate + h * DV;
+    float ss = 0.f;
+    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
+        alignas(16) float x[V];
+        if constexpr (V == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+        else x[0] = row[j];
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / static_cast<float>(DV) + eps);
+    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
+        alignas(16) float x[V];
+        alignas(16) float w[V];
+        alignas(16) T g[V];
+        alignas(16) T y[V];
+        if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
+            *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(weight + h * w_head_stride + j);
+        } else {
+            x[0] = row[j];
+            w[0] = weight[h * w_head_stride + j];
+        }
+        struct alignas(V * sizeof(T)) Pack { T v[V]; };
+        if (gate_kind) *reinterpret_cast<Pack*>(g) = *reinterpret_cast<const Pack*>(static_cast<const T*>(gate) + g0 + j);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float z = gate_kind ? to_f32(g[e]) : static_cast<const float*>(gate)[g0 + j + e];
+            y[e] = from_f32<T>(x[e] * inv * w[e] * (gate_kind == 1 ? silu_f(z) : sigmoid_f(z)));
+        }
+        *reinterpret_cast<Pack*>(out + (static_cast<size_t>(t) * H + h) * DV + j) = *reinterpret_cast<Pack*>(y);
+    }
+}
+
+constexpr int kWideHead = 512;
+
+// Between the two passes over pieces of the delta rule, whose pieces carry a memory across by a full matrix: piece_t [z, H, D, D] holds it, piece_s
 // [z, H, D, DV] what the piece adds from a zero memory; S_next = T S + B. A CTA owns 16 columns of S of one head of one
 // request and walks the pieces in order; T comes through shared memory in slabs of 16 columns. The memory at a piece's
 // start takes the place of the piece's own sum, the memory after the last piece goes into the state.
@@ -251,52 +317,6 @@ delta_pieces_combine_kernel(float* __restrict__ piece_s, const float* __restrict
         if (c0 + col < DV) S_g[static_cast<size_t>(row) * DV + c0 + col] = S_s[row][col];
     }
 }
-
-// The same with a CTA a (token, head), for heads so wide that a warp would walk them for long (one norm over all heads of a
-// token counts as one head). V columns a thread and turn.
-template <typename T, int V>
-__global__ void __launch_bounds__(256)
-head_norm_gate_wide_kernel(const float* __restrict__ o, const float* __restrict__ weight, int w_head_stride, const void* __restrict__ gate,
-                           int ld_gate, int gate_kind, T* __restrict__ out, int H, int DV, float eps) {
-    __shared__ float scratch[32];
-    pdl_trigger();
-    pdl_wait();
-    const int t = blockIdx.x / H, h = blockIdx.x % H;
-    const float* row = o + (static_cast<size_t>(t) * H + h) * DV;
-    const size_t g0 = static_cast<size_t>(t) * ld_gate + h * DV;
-    float ss = 0.f;
-    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
-        alignas(16) float x[V];
-        if constexpr (V == 4) *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
-        else x[0] = row[j];
-#pragma unroll
-        for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
-    }
-    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / static_cast<float>(DV) + eps);
-    for (int j = threadIdx.x * V; j < DV; j += blockDim.x * V) {
-        alignas(16) float x[V];
-        alignas(16) float w[V];
-        alignas(16) T g[V];
-        alignas(16) T y[V];
-        if constexpr (V == 4) {
-            *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(row + j);
-            *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(weight + h * w_head_stride + j);
-        } else {
-            x[0] = row[j];
-            w[0] = weight[h * w_head_stride + j];
-        }
-        struct alignas(V * sizeof(T)) Pack { T v[V]; };
-        if (gate_kind) *reinterpret_cast<Pack*>(g) = *reinterpret_cast<const Pack*>(static_cast<const T*>(gate) + g0 + j);
-#pragma unroll
-        for (int e = 0; e < V; ++e) {
-            const float z = gate_kind ? to_f32(g[e]) : static_cast<const float*>(gate)[g0 + j + e];
-            y[e] = from_f32<T>(x[e] * inv * w[e] * (gate_kind == 1 ? silu_f(z) : sigmoid_f(z)));
-        }
-        *reinterpret_cast<Pack*>(out + (static_cast<size_t>(t) * H + h) * DV + j) = *reinterpret_cast<Pack*>(y);
-    }
-}
-
-constexpr int kWideHead = 512;
 
 }  // namespace stride
 
@@ -462,10 +482,12 @@ int stride_head_norm_gate(const float* o, const float* weight, int w_head_stride
                           int tokens, int H, int DV, float eps, int dtype, cudaStream_t stream) {
     if (tokens < 0 || H <= 0 || DV <= 0 || gate_kind < 0 || gate_kind > 2) return STRIDE_BAD_ARGUMENT;
     if (tokens == 0) return 0;
+    if (dtype != STRIDE_DTYPE_F32 && dtype != STRIDE_DTYPE_BF16) return STRIDE_BAD_ARGUMENT;
     const long long pairs = static_cast<long long>(tokens) * H;
-    if (DV >= kWideHead && pairs < 0x7fffffff && (dtype == STRIDE_DTYPE_F32 || dtype == STRIDE_DTYPE_BF16)) {
-        auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-        const bool vec = DV % 4 == 0 && ld_gate % 4 == 0 && aligned(o) && aligned(weight) && aligned(gate) && aligned(out) && w_head_stride % 4 == 0;
+    if (pairs >= 0x7fffffff) return STRIDE_UNSUPPORTED;
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool vec = DV % 4 == 0 && ld_gate % 4 == 0 && aligned(o) && aligned(weight) && aligned(gate) && aligned(out) && w_head_stride % 4 == 0;
+    if (DV >= kWideHead) {
         const dim3 cta(DV / (vec ? 4 : 1) >= 256 ? 256 : 128), each(static_cast<unsigned>(pairs));
         if (dtype == STRIDE_DTYPE_F32)
             stride::launch(vec ? head_norm_gate_wide_kernel<float, 4> : head_norm_gate_wide_kernel<float, 1>, each, cta, 0, stream, o, weight,
@@ -477,13 +499,11 @@ int stride_head_norm_gate(const float* o, const float* weight, int w_head_stride
     }
     const dim3 grid(static_cast<unsigned>((pairs + 7) / 8)), block(256);
     if (dtype == STRIDE_DTYPE_F32)
-        stride::launch(head_norm_gate_kernel<float>, grid, block, 0, stream, o, weight, w_head_stride, gate, ld_gate, gate_kind,
-                       static_cast<float*>(out), tokens, H, DV, eps);
-    else if (dtype == STRIDE_DTYPE_BF16)
-        stride::launch(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, stream, o, weight, w_head_stride, gate, ld_gate, gate_kind,
-                       static_cast<__nv_bfloat16*>(out), tokens, H, DV, eps);
+        stride::launch(vec ? head_norm_gate_kernel<float, 4> : head_norm_gate_kernel<float, 1>, grid, block, 0, stream, o, weight, w_head_stride,
+                       gate, ld_gate, gate_kind, static_cast<float*>(out), tokens, H, DV, eps);
     else
-        return STRIDE_BAD_ARGUMENT;
+        stride::launch(vec ? head_norm_gate_kernel<__nv_bfloat16, 4> : head_norm_gate_kernel<__nv_bfloat16, 1>, grid, block, 0, stream, o, weight,
+                       w_head_stride, gate, ld_gate, gate_kind, static_cast<__nv_bfloat16*>(out), tokens, H, DV, eps);
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -15,7 +15,8 @@
 //                    A thread owns a channel and reads all it needs before it writes.
 //   conv_row_norm    the same with one norm over all query channels of a token and one over all its key channels (weights of
 //                    those widths) instead of a norm a head, and a factor on the queries that grows with the token's position p:
-//                    1 + coef ln(floor((p + 1) / every) + 1) (every 0: none). One CTA a token.
+//                    1 + coef ln(floor((p + 1) / every) + 1) (every 0: none). One CTA a token. A request that brings one
+//                    token has its tail moved on the spot (nobody else reads it); conv_tail does the others afterwards.
 // One warp a (token, head); float32 arithmetic; sums in an order that depends on the head's width only. Heads of whole
 // 16-byte packs on 16-byte boundaries take the packed form: a lane holds whole packs of its head (8 bfloat16 or 4 float32
 // channels), a warp serves one head of up to 32 packs or two heads of up to 16, and every row of a tap is one 16-byte read.
@@ -223,17 +224,18 @@ conv_head_norm_vec_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out
 }
 
 // One CTA a token. A thread works on packs of V channels (16 bytes of the compute type, or one channel where sizes or pointers
-// are not multiples of a pack) and keeps their convolved values in shared memory until the two sums of squares are known.
-template <typename T, int V>
-__global__ void __launch_bounds__(256)
+// are not multiples of a pack) and keeps their convolved values in shared memory until the two sums of squares are known. AHEAD taps'
+// reads are in flight together: several for a few tokens, where latency decides; one for many, where registers do.
+template <typename T, int V, int AHEAD>
+__global__ void __launch_bounds__(AHEAD == 1 ? 256 : 512)
 conv_row_norm_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out, int ld_out, const float* __restrict__ conv_w, int taps,
-                     const float* __restrict__ state, long long state_stride, long long tail_off,
-                     const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ q_start, const int32_t* __restrict__ state_slot,
-                     const int32_t* __restrict__ positions, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                     float* __restrict__ state, long long state_stride, long long tail_off,
+                     const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ q_start, const int32_t* __restrict__ q_len,
+                     const int32_t* __restrict__ state_slot, const int32_t* __restrict__ positions, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                      float temp_coef, int temp_every, const int32_t* __restrict__ slot_mapping, T* __restrict__ k_pages,
                      T* __restrict__ v_pages, int nq, int nkv, int hd, int vd, int page_size) {
     extern __shared__ __align__(16) float y_row[];      // C floats
-    __shared__ float part[2][8];
+    __shared__ float part[2][16];
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -241,7 +243,8 @@ conv_row_norm_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out, int
     if (seq < 0) return;
     const int q_dim = nq * hd, k_dim = nkv * hd, C = q_dim + k_dim + nkv * vd;
     const int start = q_start[seq], local = t - start;
-    const float* tail = state ? state + static_cast<size_t>(state_slot[seq]) * state_stride + tail_off : nullptr;
+    float* tail = state ? state + static_cast<size_t>(state_slot[seq]) * state_stride + tail_off : nullptr;
+    const bool single = tail && q_len[seq] == 1;
     auto load = [](const auto* p, float* v) {
         if constexpr (V == 1) v[0] = to_f32(*p);
         else ConvPack<std::remove_cv_t<std::remove_reference_t<decltype(*p)>>>::load(p, v);
@@ -259,14 +262,26 @@ conv_row_norm_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out, int
         if (conv_w && taps > 1) {
 #pragma unroll
             for (int e = 0; e < V; ++e) y[e] = 0.f;
-            for (int j = 0; j < taps; ++j) {
-                const int src = local - (taps - 1) + j;
-                float u[V], w[V];
-                if (src >= 0) load(raw + static_cast<size_t>(start + src) * ld + c, u);
-                else load_floats(tail + static_cast<size_t>(taps - 1 + src) * C + c, u);
-                load_floats(conv_w + static_cast<size_t>(j) * C + c, w);
+            for (int j0 = 0; j0 < taps; j0 += AHEAD) {
+                float u[AHEAD][V], w[AHEAD][V];
 #pragma unroll
-                for (int e = 0; e < V; ++e) y[e] = fmaf(w[e], u[e], y[e]);
+                for (int a = 0; a < AHEAD; ++a)
+                    if (j0 + a < taps) {
+                        const int src = local - (taps - 1) + j0 + a;
+                        if (src >= 0) load(raw + static_cast<size_t>(start + src) * ld + c, u[a]);
+                        else load_floats(tail + static_cast<size_t>(taps - 1 + src) * C + c, u[a]);
+                        load_floats(conv_w + static_cast<size_t>(j0 + a) * C + c, w[a]);
+                    }
+#pragma unroll
+                for (int a = 0; a < AHEAD; ++a)
+                    if (j0 + a < taps) {
+#pragma unroll
+                        for (int e = 0; e < V; ++e) y[e] = fmaf(w[a][e], u[a][e], y[e]);
+                        if (single && j0 + a > 0) {         // row m of the tail becomes what was row m + 1; the new value is the last row
+#pragma unroll
+                            for (int e = 0; e < V; ++e) tail[static_cast<size_t>(j0 + a - 1) * C + c + e] = u[a][e];
+                        }
+                    }
             }
         } else {
             load(raw + static_cast<size_t>(t) * ld + c, y);
@@ -337,12 +352,12 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 conv_tail_kernel(const T* __restrict__ raw, int ld, float* __restrict__ state, long long state_stride, long long tail_off,
                  const int32_t* __restrict__ q_start, const int32_t* __restrict__ q_len, const int32_t* __restrict__ state_slot, int C,
-                 int taps) {
+                 int taps, int min_len) {
     pdl_trigger();
     pdl_wait();
     const int seq = blockIdx.x;
     const int len = q_len[seq];
-    if (len <= 0) return;
+    if (len < min_len) return;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= C) return;
     const int keep = taps - 1, start = q_start[seq];
@@ -403,15 +418,15 @@ int stride_conv_head_norm(const void* raw, int ld, void* out, int ld_out, const 
     return STRIDE_LAUNCH_STATUS();
 }
 
-int stride_conv_row_norm(const void* raw, int ld, void* out, int ld_out, const float* conv_w, int taps, const float* state,
+int stride_conv_row_norm(const void* raw, int ld, void* out, int ld_out, const float* conv_w, int taps, float* state,
                          long long state_stride, long long tail_off, const int32_t* seq_of_token, const int32_t* q_start,
-                         const int32_t* state_slot, const int32_t* positions, const float* wq, const float* wk, float eps, float temp_coef,
+                         const int32_t* q_len, const int32_t* state_slot, const int32_t* positions, const float* wq, const float* wk, float eps, float temp_coef,
                          int temp_every, const int32_t* slot_mapping, void* k_pages, void* v_pages, int tokens, int nq, int nkv, int hd,
                          int vd, int page_size, int dtype, cudaStream_t stream) {
     const long long C = static_cast<long long>(nq + nkv) * hd + static_cast<long long>(nkv) * vd;
     if (tokens < 0 || nq <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || ld < C || ld_out < C || taps < 1 || temp_every < 0)
         return STRIDE_BAD_ARGUMENT;
-    if (taps > 1 && (!conv_w || !state || !q_start || !state_slot || state_stride < tail_off + (taps - 1) * C)) return STRIDE_BAD_ARGUMENT;
+    if (taps > 1 && (!conv_w || !state || !q_start || !q_len || !state_slot || state_stride < tail_off + (taps - 1) * C)) return STRIDE_BAD_ARGUMENT;
     if ((slot_mapping != nullptr && (k_pages == nullptr || v_pages == nullptr)) || (temp_every > 0 && !positions)) return STRIDE_BAD_ARGUMENT;
     const long long bytes = C * 4;
     if (taps > kConvMaxTaps || bytes > 200 * 1024) return STRIDE_UNSUPPORTED;
@@ -421,6 +436,7 @@ int stride_conv_row_norm(const void* raw, int ld, void* out, int ld_out, const f
     const bool vec = hd % pack == 0 && vd % pack == 0 && ld % pack == 0 && ld_out % pack == 0 && aligned(raw) && aligned(out) &&
                      aligned(k_pages) && aligned(v_pages) && aligned(wq) && aligned(wk) && aligned(state) && aligned(conv_w) &&
                      state_stride % 4 == 0 && tail_off % 4 == 0;
+    const bool few = tokens <= 64 || dtype == STRIDE_DTYPE_F32;        // (float32: one order of the sums for every number of tokens)
     auto run = [&](auto kernel, auto* typed_raw) {
         using T = std::remove_cv_t<std::remove_pointer_t<decltype(typed_raw)>>;
         if (bytes > 48 * 1024) {
@@ -428,22 +444,24 @@ int stride_conv_row_norm(const void* raw, int ld, void* out, int ld_out, const f
             if (e != cudaSuccess) return static_cast<int>(e);
         }
         const long long items = vec ? C / pack : C;
-        const int threads = items >= 256 ? 256 : static_cast<int>((items + 31) / 32 * 32);
+        const int limit = few ? 512 : 256, threads = items >= limit ? limit : static_cast<int>((items + 31) / 32 * 32);
         stride::launch(kernel, dim3(tokens), dim3(threads), static_cast<size_t>(bytes), stream, typed_raw, ld, static_cast<T*>(out), ld_out,
-                       conv_w, taps, state, state_stride, tail_off, seq_of_token, q_start, state_slot, positions, wq, wk, eps, temp_coef,
+                       conv_w, taps, state, state_stride, tail_off, seq_of_token, q_start, q_len, state_slot, positions, wq, wk, eps, temp_coef,
                        temp_every, slot_mapping, static_cast<T*>(k_pages), static_cast<T*>(v_pages), nq, nkv, hd, vd, page_size);
         return STRIDE_LAUNCH_STATUS();
     };
     if (dtype == STRIDE_DTYPE_F32)
-        return run(vec ? conv_row_norm_kernel<float, 4> : conv_row_norm_kernel<float, 1>, static_cast<const float*>(raw));
+        return run(vec ? conv_row_norm_kernel<float, 4, 4> : conv_row_norm_kernel<float, 1, 4>, static_cast<const float*>(raw));
     if (dtype == STRIDE_DTYPE_BF16)
-        return run(vec ? conv_row_norm_kernel<__nv_bfloat16, 8> : conv_row_norm_kernel<__nv_bfloat16, 1>, static_cast<const __nv_bfloat16*>(raw));
+        return run(few ? (vec ? conv_row_norm_kernel<__nv_bfloat16, 8, 4> : conv_row_norm_kernel<__nv_bfloat16, 1, 4>)
+                       : (vec ? conv_row_norm_kernel<__nv_bfloat16, 8, 1> : conv_row_norm_kernel<__nv_bfloat16, 1, 1>),
+                   static_cast<const __nv_bfloat16*>(raw));
     return STRIDE_BAD_ARGUMENT;
 }
 
 int stride_conv_tail(const void* raw, int ld, float* state, long long state_stride, long long tail_off, const int32_t* q_start,
-                     const int32_t* q_len, const int32_t* state_slot, int num_seqs, int C, int taps, int dtype, cudaStream_t stream) {
-    if (num_seqs < 0 || C <= 0 || ld < C || taps < 1 || !state || state_stride < tail_off + static_cast<long long>(taps - 1) * C)
+                     const int32_t* q_len, const int32_t* state_slot, int num_seqs, int C, int taps, int min_len, int dtype, cudaStream_t stream) {
+    if (num_seqs < 0 || C <= 0 || ld < C || taps < 1 || min_len < 1 || !state || state_stride < tail_off + static_cast<long long>(taps - 1) * C)
         return STRIDE_BAD_ARGUMENT;
     if (taps > kConvMaxTaps || num_seqs > 0x7fffffff / 2) return STRIDE_UNSUPPORTED;
     if (num_seqs == 0 || taps == 1) return 0;
@@ -451,10 +469,10 @@ int stride_conv_tail(const void* raw, int ld, float* state, long long state_stri
     if (grid.y > 65535) return STRIDE_UNSUPPORTED;
     if (dtype == STRIDE_DTYPE_F32)
         stride::launch(conv_tail_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(raw), ld, state, state_stride, tail_off,
-                       q_start, q_len, state_slot, C, taps);
+                       q_start, q_len, state_slot, C, taps, min_len);
     else if (dtype == STRIDE_DTYPE_BF16)
         stride::launch(conv_tail_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, static_cast<const __nv_bfloat16*>(raw), ld, state,
-                       state_stride, tail_off, q_start, q_len, state_slot, C, taps);
+                       state_stride, tail_off, q_start, q_len, state_slot, C, taps, min_len);
     else
         return STRIDE_BAD_ARGUMENT;
     return STRIDE_LAUNCH_STATUS();

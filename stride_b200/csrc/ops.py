@@ -33,7 +33,7 @@ _SIGNATURES = {
                                             c_int, c_void_p]),
     "stride_add_rmsnorm": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p]),
     "stride_add_residual": ("elementwise", [c_void_p, c_void_p, c_longlong, c_int, c_void_p]),
-    "stride_zero_fresh_state": ("elementwise", [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
+    "stride_zero_fresh_states": ("elementwise", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
     "stride_rope_kv_write": ("elementwise", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_silu_mul": ("elementwise", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
@@ -56,6 +56,7 @@ _SIGNATURES = {
     "stride_gemm_rows_add_norm": ("gemm_bf16_rows", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int,
                                                      c_int, c_int, c_void_p, c_void_p, c_void_p]),
     "stride_gemm_stream_bf16": ("gemm_bf16_stream", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
+    "stride_gemm_stream_relu2": ("gemm_bf16_stream", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]),
     "stride_gemm_stream_qkv_rope": ("gemm_bf16_stream", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                          c_void_p, c_int, c_float, c_void_p, c_void_p]),
@@ -143,13 +144,15 @@ _SIGNATURES = {
                                              c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                              c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_conv_tail": ("short_conv", [c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                        c_int, c_void_p]),
+                                        c_int, c_int, c_void_p]),
     "stride_conv_row_norm": ("short_conv", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
-                                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p, c_void_p,
-                                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+                                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p,
+                                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_copies_step": ("stream_copies", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
                                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_decay_scan": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                           c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_decay_step": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
                                            c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_decay_chunks": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
                                              c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -190,7 +193,7 @@ def _fn(name: str, what: str | None = None):
 # What a launcher counts as when the time of a step is split up. Matrix products say more (their shape) at the call.
 _CLASS_OF = {
     "stride_embed_gather": "embedding", "stride_add_rmsnorm": "norm", "stride_add_residual": "residual sum",
-    "stride_scale_rows": "norm", "stride_zero_fresh_state": "state slots", "stride_rope_kv_write": "rotation + cache write",
+    "stride_scale_rows": "norm", "stride_zero_fresh_states": "state slots", "stride_rope_kv_write": "rotation + cache write",
     "stride_silu_mul": "silu * up", "stride_paged_attention_generic": "attention (exact kernel)",
     "stride_paged_decode_attention_tma": "attention (decode)", "stride_paged_decode_attention_rules": "attention (decode)", "stride_paged_decode_attention_gated": "attention (decode)", "stride_paged_prefill_attention": "attention (prefill, mma.sync)",
     "stride_paged_prefill_attention_tc": "attention (prefill, tcgen05)", "stride_sample_rows": "sampling", "stride_sample_ranked": "sampling",
@@ -213,6 +216,7 @@ _CLASS_OF = {
     "stride_conv_tail": "convolution + head norms + cache write", "stride_mlstm_scan": "matrix LSTM: recurrence",
     "stride_conv_row_norm": "convolution + row norms + cache write", "stride_copies_step": "residual copies + norm",
     "stride_decay_scan": "fading memory: recurrence", "stride_decay_chunks": "fading memory: recurrence",
+    "stride_decay_step": "fading memory: recurrence",
     "stride_paged_decode_attention_biased": "attention (decode)",
 }
 
@@ -355,15 +359,21 @@ def add_residual(residual, delta) -> None:
                                       _code(delta.dtype), _stream()), "add_residual")
 
 
-def zero_fresh_state(state, state_slot, q_start, q_len, positions) -> None:
-    """Clears ``state[slot]`` for every sequence of the step whose first token sits at position 0 (``state``:
-    [num_slots, ...] of a 4-byte element type; the index arrays are the step's, at their layout's capacity)."""
-    if state.element_size() != 4:
-        raise KernelError("state rows must have a 4-byte element type")
-    row_bytes = (state.numel() // state.shape[0]) * 4
-    _check(_fn("stride_zero_fresh_state")(_dev(state, "state"), row_bytes, state.shape[0], _dev(state_slot, "state_slot", torch.int32),
-                                          _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
-                                          _dev(positions, "positions", torch.int32), q_len.shape[0], _stream()), "zero_fresh_state")
+def zero_fresh_states(states, state_slot, q_start, q_len, positions) -> None:
+    """Clears row ``slot`` of every tensor of ``states`` ([num_slots, ...] of a 4-byte element type) for every sequence of the step
+    whose first token sits at position 0 (the index arrays are the step's, at their layout's capacity)."""
+    if not states:
+        return
+    slots = states[0].shape[0]
+    if any(s.element_size() != 4 or s.shape[0] != slots for s in states):
+        raise KernelError("state rows must have a 4-byte element type, and all states the same number of slots")
+    n = len(states)
+    pointers = (c_void_p * n)(*[_dev(s, "state") for s in states])
+    row_bytes = (c_longlong * n)(*[s.numel() // slots * 4 for s in states])
+    _check(_fn("stride_zero_fresh_states")(ctypes.cast(pointers, c_void_p), ctypes.cast(row_bytes, c_void_p), n, slots,
+                                           _dev(state_slot, "state_slot", torch.int32), _dev(q_start, "q_start", torch.int32),
+                                           _dev(q_len, "q_len", torch.int32), _dev(positions, "positions", torch.int32), q_len.shape[0],
+                                           _stream()), "zero_fresh_states")
 
 
 def rope_kv_write(qkv, bias, positions, slot_mapping, cos, sin, k_pages, v_pages, nq: int, nkv: int, hd: int,
@@ -612,18 +622,24 @@ def _decay_args(proj, q_off, k_off, v_off, logit, bias, H, D, DV, o):
 
 
 def decay_scan(proj, q_off: int, k_off: int, v_off: int, logit, bias, fade, q_scale: float, inv_tau: float, o, state, q_start, q_len,
-               state_slot, num_seqs: int, H: int, D: int, DV: int) -> None:
+               state_slot, num_seqs: int, H: int, D: int, DV: int, single: bool = False) -> None:
     """A matrix memory that fades, over every request of the step in token order. ``proj`` [tokens, ld] holds q, k ([H, D]) and v
     ([H, DV]) from the given columns on. Channel decays (``fade`` None): ``S = diag(sigmoid(logit + bias)^inv_tau) S + k v^T``,
     ``o = q_scale S^T q`` (``logit`` float32 [tokens, H * D], ``bias`` float32 [H * D]). Constant decay (``fade`` float32 [H], the
-    decay minus one): ``S = (1 + fade) S + silu(k) silu(v)^T``, ``o = S^T silu(q)``. ``o`` [tokens, H * DV] float32; S in ``state``."""
+    decay minus one): ``S = (1 + fade) S + silu(k) silu(v)^T``, ``o = S^T silu(q)``. ``o`` [tokens, H * DV] float32; S in ``state``.
+    ``single``: every request brings one token at most; one pass over S where the sizes allow it (its sums take another order)."""
     if state.shape[1] < H * D * DV:
         raise KernelError("decay_scan: the state rows are too short")
-    _check(_fn("stride_decay_scan")(
+    args = (
         *_decay_args(proj, q_off, k_off, v_off, logit, bias, H, D, DV, o), _opt(logit, "logit", torch.float32),
         _opt(bias, "bias", torch.float32), _opt(fade, "fade", torch.float32), float(q_scale), float(inv_tau), _dev(o, "o", torch.float32),
         *_state_rows(state), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
-        _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype), _stream()), "decay_scan")
+        _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype), _stream())
+    if single:
+        code = _fn("stride_decay_step")(*args)
+        if code != -2:
+            return _check(code, "decay_step")
+    _check(_fn("stride_decay_scan")(*args), "decay_scan")
 
 
 def decay_chunks_scratch_floats(num_seqs: int, max_q_len: int, H: int, D: int, DV: int) -> int:
@@ -699,11 +715,12 @@ def conv_head_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start
         _code(raw.dtype), _stream()), "conv_head_norm")
 
 
-def conv_row_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start, state_slot, positions, wq, wk, eps: float, temp_coef: float,
-                  temp_every: int, slot_mapping, k_pages, v_pages, nq: int, nkv: int, hd: int, vd: int, page_size: int) -> None:
+def conv_row_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start, q_len, state_slot, positions, wq, wk, eps: float,
+                  temp_coef: float, temp_every: int, slot_mapping, k_pages, v_pages, nq: int, nkv: int, hd: int, vd: int, page_size: int) -> None:
     """``conv_head_norm`` with one RMS norm over a token's whole query projection (weight ``wq`` [nq * hd]) and one over its whole
     key projection (``wk`` [nkv * hd]) in place of a norm a head, and queries multiplied by
-    ``1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)`` at position p (``temp_every`` 0: not)."""
+    ``1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)`` at position p (``temp_every`` 0: not). The tails of requests that bring one
+    token move on here; for the others ``conv_tail`` with ``min_len`` 2 does it afterwards."""
     taps = 1 if conv_w is None else conv_w.shape[0]
     if out.dtype != raw.dtype or out.shape[0] != raw.shape[0]:
         raise KernelError("conv_row_norm: raw and out must agree in rows and element type")
@@ -712,18 +729,19 @@ def conv_row_norm(raw, out, conv_w, state, tail_off: int, seq_of_token, q_start,
     _check(_fn("stride_conv_row_norm")(
         _dev(raw, "raw"), raw.shape[1], _dev(out, "out"), out.shape[1], _opt(conv_w, "conv_w", torch.float32), taps,
         *(_state_rows(state) if state is not None else (None, 0)), int(tail_off),
-        _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32), _dev(state_slot, "state_slot", torch.int32),
-        _dev(positions, "positions", torch.int32), _opt(wq, "wq", torch.float32), _opt(wk, "wk", torch.float32), float(eps), float(temp_coef),
+        _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
+        _dev(state_slot, "state_slot", torch.int32), _dev(positions, "positions", torch.int32), _opt(wq, "wq", torch.float32), _opt(wk, "wk", torch.float32), float(eps), float(temp_coef),
         int(temp_every), _opt(slot_mapping, "slot_mapping", torch.int32), _opt(k_pages, "k_pages", raw.dtype),
         _opt(v_pages, "v_pages", raw.dtype), raw.shape[0], nq, nkv, hd, vd, page_size, _code(raw.dtype), _stream()), "conv_row_norm")
 
 
-def conv_tail(raw, state, tail_off: int, q_start, q_len, state_slot, num_seqs: int, channels: int, taps: int) -> None:
-    """Moves every request's convolution tail on by the step's rows of ``raw`` (its first ``channels`` columns)."""
+def conv_tail(raw, state, tail_off: int, q_start, q_len, state_slot, num_seqs: int, channels: int, taps: int, min_len: int = 1) -> None:
+    """Moves the convolution tail of every request that brings at least ``min_len`` tokens on by the step's rows of ``raw`` (its first
+    ``channels`` columns)."""
     _check(_fn("stride_conv_tail")(
         _dev(raw, "raw"), raw.shape[1], *_state_rows(state), int(tail_off),
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32),
-        int(num_seqs), int(channels), int(taps), _code(raw.dtype), _stream()), "conv_tail")
+        int(num_seqs), int(channels), int(taps), int(min_len), _code(raw.dtype), _stream()), "conv_tail")
 
 
 def rms_norm_cols(x, col_off: int, width: int, weight, out, eps: float) -> None:
@@ -1391,6 +1409,22 @@ def linear_stream(x, weight, out) -> bool:
         return False
     _check(code, "gemm_stream_bf16")
     return True
+
+
+def linear_relu2(x, weight, out) -> None:
+    """``out = relu(x @ weight.T)^2``: in the epilogue of the weight-streaming product for a few bfloat16 rows, else the product and
+    a kernel of its own."""
+    m, k = x.shape
+    n = weight.shape[0]
+    if x.dtype == torch.bfloat16 and 0 < m <= TC_GEMM_MAX_TOKENS and STREAM_GEMM and -(-n // 128) < TC_GEMM_MIN_TILES and \
+            weight.shape[1] == k and out.shape == (m, n):
+        code = _fn("stride_gemm_stream_relu2", f"product {n}x{k} (weight streaming, relu^2)")(
+            _dev(x, "x", torch.bfloat16), _dev(weight, "weight", torch.bfloat16), _dev(out, "out", torch.bfloat16), m, n, k,
+            _status_ptr(x.device), _stream())
+        if code != -2:
+            return _check(code, "gemm_stream_relu2")
+    linear(x, weight, out)
+    relu_squared(out)
 
 
 def linear_qkv_rope(x, weight, qkv, bias, positions, slot_mapping, cos, sin, k_pages, v_pages, nq: int, nkv: int, hd: int,

@@ -372,18 +372,16 @@ class PagedAttention(Mixer):
         slots = ctx.slot_mapping[cache.group][:tokens] if cache.writes else None
         state = cache.state if self.taps > 1 else None
         if self.row_norm:
-            ops.conv_row_norm(raw, qkv, self.conv_w, state, 0, ctx.seq_of_token[:tokens], ctx.q_start, ctx.state_slot, ctx.positions[:tokens],
-                              self.wq_norm, self.wk_norm, self.norm_eps, self.q_coef, self.q_every, slots,
+            ops.conv_row_norm(raw, qkv, self.conv_w, state, 0, ctx.seq_of_token[:tokens], ctx.q_start, ctx.q_len, ctx.state_slot,
+                              ctx.positions[:tokens], self.wq_norm, self.wk_norm, self.norm_eps, self.q_coef, self.q_every, slots,
                               cache.k_pages if cache.writes else None, cache.v_pages if cache.writes else None, self.nq, self.nkv, self.hd,
                               self.vd, cache.page_size)
-            self._move_tails(raw, state, ctx)
+            if state is not None and ctx.decode_tail_seq:       # single tokens have moved theirs
+                ops.conv_tail(raw, state, 0, ctx.q_start, ctx.q_len, ctx.state_slot, ctx.decode_tail_seq, self.qkv_dim, self.taps, min_len=2)
             return
         ops.conv_head_norm(raw, qkv, self.conv_w, state, 0, ctx.seq_of_token[:tokens], ctx.q_start, ctx.state_slot, self.wq_norm, self.wk_norm,
                            self.norm_eps, slots, cache.k_pages if cache.writes else None, cache.v_pages if cache.writes else None, self.nq,
                            self.nkv, self.hd, self.vd, cache.page_size)
-        self._move_tails(raw, state, ctx)
-
-    def _move_tails(self, raw, state, ctx):
         if state is not None:
             ops.conv_tail(raw, state, 0, ctx.q_start, ctx.q_len, ctx.state_slot, sequence_slots(ctx), self.qkv_dim, self.taps)
 

@@ -102,18 +102,23 @@ class DecayMemoryMixer(Mixer):
 
     def _recur(self, proj, logit, o, ctx, state) -> None:
         columns, sizes = (0, self.k_off, self.v_off), (self.H, self.D, self.DV)
-        first = 0
-        portions = ctx.decode_tail_seq          # requests that may bring more than one token
-        if proj.dtype == torch.bfloat16 and portions and 0 < ops.DECAY_CHUNKS_MIN_TOKENS <= ctx.max_q_len and \
-                portions * -(-ctx.max_q_len // ops.DECAY_CHUNK) <= 65535:
+        half = proj.dtype == torch.bfloat16         # float32 models keep the one chain, whose sums do not depend on the cutting
+        portions, slots = ctx.decode_tail_seq, sequence_slots(ctx)       # the requests before the trailing single tokens; all of them
+
+        def chain(first, past, single):
+            if past > first:
+                ops.decay_scan(proj, *columns, logit, self.decay_bias, self.fade, self.q_scale, self.inv_tau, o, state, ctx.q_start[first:],
+                               ctx.q_len[first:], ctx.state_slot[first:], past - first, *sizes, single=single)
+
+        if not half:
+            return chain(0, slots, False)
+        if portions and 0 < ops.DECAY_CHUNKS_MIN_TOKENS <= ctx.max_q_len and portions * -(-ctx.max_q_len // ops.DECAY_CHUNK) <= 65535:
             scratch = self.rt.scratch("memory_chunks", ops.decay_chunks_scratch_floats(portions, ctx.max_q_len, *sizes))
             ops.decay_chunks(proj, *columns, logit, self.decay_bias, self.powers, self.q_scale, self.inv_tau, o, state, ctx.q_start, ctx.q_len,
                              ctx.state_slot, portions, *sizes, ctx.max_q_len, scratch)
-            first = portions
-        rest = sequence_slots(ctx) - first
-        if rest > 0:
-            ops.decay_scan(proj, *columns, logit, self.decay_bias, self.fade, self.q_scale, self.inv_tau, o, state, ctx.q_start[first:],
-                           ctx.q_len[first:], ctx.state_slot[first:], rest, *sizes)
+        else:
+            chain(0, portions, False)
+        chain(portions, slots, True)
 
 
 class LightningMixer(DecayMemoryMixer):

@@ -29,8 +29,7 @@ class PlainMLP(FeedForward):
 
     def forward(self, x, ctx, lazy_output: bool = False):
         act = self.rt.buffer("ffn_act", x.shape[0], self.inter)
-        ops.linear(x, self.w_up, act)
-        ops.relu_squared(act)
+        ops.linear_relu2(x, self.w_up, act)
         if lazy_output:
             return Projection(act, self.w_down)
         out = self.rt.buffer("ffn_out", x.shape[0], self.hidden)

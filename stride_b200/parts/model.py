@@ -112,8 +112,8 @@ class DecoderModel:
         tokens = ctx.num_tokens
         stream = CopiedStream(self.rt, tokens, self.hidden, self.copies) if self.copies else ResidualStream(self.rt, tokens, self.hidden)
         self.embedding.forward(ctx, stream.residual)
-        for state in self._states():        # a request that starts in this step finds its state slots at zero
-            ops.zero_fresh_state(state, ctx.state_slot, ctx.q_start, ctx.q_len, ctx.positions)
+        # a request that starts in this step finds its state slots at zero
+        ops.zero_fresh_states(self._states(), ctx.state_slot, ctx.q_start, ctx.q_len, ctx.positions)
         first = None
         if self.pass_input is not None:         # the embedding's output in the compute dtype, for every pass to come
             first = self.rt.buffer("embedding_out", tokens, self.hidden)

@@ -252,6 +252,38 @@ def test_memory_with_channel_decays(gpu, dtype, H, D, DV, form):
     assert torch.equal(state_dev[:, H * D * DV:].cpu(), state[:, H * D * DV:]) and torch.equal(state_dev[3].cpu(), state[3])
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("constant", [True, False])
+@pytest.mark.parametrize("H,D,DV", [(3, 12, 20), (2, 64, 128), (1, 200, 24), (2, 128, 132), (4, 32, 32), (1, 256, 260), (3, 10, 14)])
+def test_a_single_token_of_every_request(gpu, dtype, constant, H, D, DV):
+    """The one-pass form: three requests with a past, a slot without a request, state rows inside wider ones. (A width that is no
+    multiple of four runs the chain.)"""
+    from stride_b200.csrc import ops
+    g = torch.Generator().manual_seed(H * D + DV)
+    new = [1, 1, 1]
+    proj, k_off, v_off, state = memory_inputs(H, D, DV, new, dtype, g)
+    wide = torch.full((4, 8 + -(-state.shape[1] // 4) * 4 + 4), float("nan"), device="cuda")
+    view = wide[:, 8:8 + state.shape[1]]
+    view.copy_(state)
+    logit, bias = torch.randn(4, H * D, generator=g) * 3.0, torch.randn(H * D, generator=g)
+    decay = torch.rand(H, generator=g, dtype=torch.float64)
+    o = torch.full((4, H * DV), float("nan"), device="cuda")
+    order = [3, 1, 2]
+    ops.decay_scan(proj.cuda(), 0, k_off, v_off, None if constant else logit.cuda(), None if constant else bias.cuda(),
+                   (decay - 1).float().cuda() if constant else None, D ** -0.5, 0.3, o, view, dev([0, 1, 2, 0]), dev([1, 1, 1, 0]), dev(order + [0]), 4,
+                   H, D, DV, single=True)
+    alpha = (torch.sigmoid(logit.double() + bias.double()) ** 0.3).view(-1, H, D)
+    for t, slot in enumerate(order):
+        rate = (lambda _t, a: float(decay[a])) if constant else (lambda _t, a: alpha[t, a][:, None])
+        S0 = state[slot, :H * D * DV].double().view(H, D, DV)
+        want, S = plain_memory(proj[t:t + 1].double(), k_off, v_off, S0, rate, H, D, DV, plain.silu if constant else (lambda x: x),
+                               1.0 if constant else D ** -0.5)
+        close(o[t], want.reshape(-1), 1e-5)
+        close(view[slot, :H * D * DV], S.reshape(-1), 1e-5)
+    assert torch.equal(view[:, H * D * DV:].cpu(), state[:, H * D * DV:]) and torch.equal(view[0].cpu(), state[0])
+    assert torch.isnan(wide[:, :8]).all() and torch.isnan(wide[:, 8 + state.shape[1]:]).all()
+
+
 @pytest.mark.parametrize("dtype,tol", [("float32", 3e-6), ("bfloat16", 8e-3)])
 @pytest.mark.parametrize("width,kind", [(20, "sigmoid_compute"), (520, "sigmoid_compute"), (514, "silu"), (2048, "sigmoid_compute"), (700, "sigmoid")])
 def test_norm_over_all_heads_with_a_gate(gpu, dtype, tol, width, kind):
@@ -316,10 +348,10 @@ def test_convolution_row_norms_query_factor_and_tails(gpu, dtype, tol, nq, nkv, 
     k_pages = torch.full((pages, nkv, page, hd), 7.0, dtype=STORED[dtype], device="cuda")
     v_pages = torch.full((pages, nkv, page, vd), 7.0, dtype=STORED[dtype], device="cuda")
     out = torch.zeros(tokens, C + 8, dtype=STORED[dtype], device="cuda")
-    ops.conv_row_norm(raw.cuda(), out, conv_w.t().contiguous().cuda() if taps else None, state if keep else None, 4, seq_of, q_start, state_slot,
+    ops.conv_row_norm(raw.cuda(), out, conv_w.t().contiguous().cuda() if taps else None, state if keep else None, 4, seq_of, q_start, q_len, state_slot,
                       positions, wq.cuda(), wk.cuda(), 1e-5, coef, every, slot_map.cuda(), k_pages, v_pages, nq, nkv, hd, vd, page)
     if keep:
-        ops.conv_tail(raw.cuda(), state, 4, q_start, q_len, state_slot, 4, C, taps)
+        ops.conv_tail(raw.cuda(), state, 4, q_start, q_len, state_slot, 4, C, taps, min_len=2)
     at = 0
     for h, p, n, slot in zip(histories, past, new, slots_of_state):
         y = plain.short_convolution(h.double(), conv_w.double()) if taps else h.double()
@@ -490,10 +522,15 @@ def test_long_portions_beside_single_tokens(gpu, tmp_models, dtype):
     replay(folder, dtype, steps, want, 16, 4, "beside", min_ok=1.0 if dtype == "float32" else 0.97)
 
 
-def test_float32_logits_do_not_depend_on_the_cutting(gpu, tmp_models):
-    """Bitwise: every sum of the 32-bit path has an order that depends on the token's position only."""
+@pytest.mark.parametrize("name", ["A", "wide"])
+def test_float32_logits_do_not_depend_on_the_cutting(gpu, tmp_models, name):
+    """Bitwise: every sum of the 32-bit path has an order that depends on the token's position only (the wide model's rows take
+    several turns of a CTA's threads)."""
     from stride_b200.engine.trace import TraceSession
-    folder, requests, _want = model_case(tmp_models, "bitwise", cases.CASE_A, cases.case_state("A", 13), "float32", 13, [141, 18, 27])
+    wide = cases.config(1100, 50, [(cases.lightning(4, 32, 144), None), (cases.parallel(cases.attention(12, 3, 64), cases.memory(2, 16, 24)), None)])
+    cfg, state = (wide, cases.seeded_state(wide, 13)) if name == "wide" else (cases.CASE_A, cases.case_state("A", 13))
+    folder, _state = write(tmp_models, "bitwise_" + name, cfg, state, "float32")
+    requests = {f"r{i}": seeded_tokens(n, cfg["vocab"], 650 + i) for i, n in enumerate([141, 18, 27])}
     results = []
     for steps in (modes.whole(requests), modes.changing_portions(requests), modes.mixed(requests, live_limit=3, seed=2)):
         session = TraceSession(folder, "float32", max_tokens=modes.peak_tokens(steps), block_size=8, max_requests=3)
