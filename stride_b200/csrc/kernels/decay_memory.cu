@@ -62,7 +62,7 @@ chunk_decay_kernel(const ChunkArgs p) {
     if (nt <= 0 || c >= HD) return;
     float* at = p.cum + static_cast<size_t>(p.q_start[seq] + first) * HD + c;
     const float b = p.bias[c];
-    double sum = 0.0;       // rounded once per token: differences of these sums are the exponents of whole decays
+    float sum = 0.f, lost = 0.f;        // Kahan's sum: differences of these sums are the exponents of whole decays
     for (int t0 = 0; t0 < nt; t0 += 8) {
         float l[8];
 #pragma unroll
@@ -72,8 +72,10 @@ chunk_decay_kernel(const ChunkArgs p) {
 #pragma unroll
         for (int u = 0; u < 8; ++u)
             if (t0 + u < nt) {
-                sum += l[u];
-                at[static_cast<size_t>(t0 + u) * HD] = static_cast<float>(sum);
+                const float y = __fadd_rn(l[u], -lost), next = __fadd_rn(sum, y);
+                lost = __fadd_rn(__fadd_rn(next, -sum), -y);
+                sum = next;
+                at[static_cast<size_t>(t0 + u) * HD] = sum;
             }
     }
 }

@@ -277,11 +277,16 @@ conv_row_norm_kernel(const T* __restrict__ raw, int ld, T* __restrict__ out, int
                     if (j0 + a < taps) {
 #pragma unroll
                         for (int e = 0; e < V; ++e) y[e] = fmaf(w[a][e], u[a][e], y[e]);
-                        if (single && j0 + a > 0) {         // row m of the tail becomes what was row m + 1; the new value is the last row
-#pragma unroll
-                            for (int e = 0; e < V; ++e) tail[static_cast<size_t>(j0 + a - 1) * C + c + e] = u[a][e];
-                        }
                     }
+            }
+            if (single) {           // row m of the tail becomes what was row m + 1; the new value is the last row
+                for (int m = 0; m < taps - 1; ++m) {
+                    float u[V];
+                    if (m + 1 < taps - 1) load_floats(tail + static_cast<size_t>(m + 1) * C + c, u);
+                    else load(raw + static_cast<size_t>(t) * ld + c, u);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) tail[static_cast<size_t>(m) * C + c + e] = u[e];
+                }
             }
         } else {
             load(raw + static_cast<size_t>(t) * ld + c, y);
