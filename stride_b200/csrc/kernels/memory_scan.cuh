@@ -1,4 +1,4 @@
-// The scan shared by the mixers whose memory is a matrix per head (linear_recurrence.cu, decay_memory.cu): a head's S [D, DV]
+// The scan shared by the mixers whose memory is a matrix per head (linear_recurrence.cu, decay_memory.cu, state_space.cu): a head's S [D, DV]
 // in registers, one token after the other, any of the rules below; and the pass between pieces of a long portion.
 #pragma once
 
@@ -11,6 +11,7 @@ enum MemoryRule {
     kBonusMemory = 1,       // o = (S + diag(bonus) k v^T)^T a ; S <- diag(exp(-exp(w + w0))) S + k v^T
     kChannelDecay = 2,      // S <- diag(sigmoid(w + w0)^(1 / tau)) S + k v^T ; o = q_scale S^T a
     kConstantDecay = 3,     // S <- (1 + fade) S + silu(k) silu(v)^T ; o = S^T silu(a)
+    kTokenDecay = 4,        // d = softplus(beta + dt_bias), S <- exp(-exp(a_log) d) S + d k v^T ; o = S^T a + skip v (a number a head and token)
 };
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
@@ -31,7 +32,7 @@ struct ScanArgs {
     const float* w;         // [tokens, H * D]: the decay minus one (delta), its double logarithm before w0 (bonus rule), or the
                             // logit before w0 whose sigmoid to the power 1 / tau is the decay (channel decays)
     const void* v;          // values [tokens, ldv], head h at column h * DV
-    const float* beta;      // [tokens, H] (delta) or null
+    const float* beta;      // [tokens, H] (delta); [tokens, ld_beta]: step sizes before bias and softplus (token decay); or null
     const float* w0;        // [H * D] added to w before exp(-exp(.)) (bonus rule) or the sigmoid (channel decays), or null
     const float* bonus;     // [H * D] (bonus rule) or null
     const float* fade;      // [H] (constant decay): the head's decay minus one
@@ -43,6 +44,10 @@ struct ScanArgs {
     const int32_t* q_len;
     const int32_t* state_slot;
     int lda, ldv, H, group, D, DV, in_bf16;
+    const float* dt_bias;   // [H] each (token decay)
+    const float* a_log;
+    const float* skip;
+    int ld_beta;
     // the convolution's tail (delta rule; taps 0: none): the last taps - 1 rows of proj's first C columns
     const void* proj;
     int ld_proj, C, taps, proj_bf16;
@@ -113,6 +118,8 @@ scan_kernel(const ScanArgs p) {
             s_w0[i] = i < D ? p.w0[h * D + i] : 0.f;
         }
     const float fade = RULE == kConstantDecay ? p.fade[h] : 0.f;
+    const float rate = RULE == kTokenDecay ? expf(p.a_log[h]) : 0.f, dt_bias = RULE == kTokenDecay ? p.dt_bias[h] : 0.f;
+    const float skip = RULE == kTokenDecay ? p.skip[h] : 0.f;
 
     float fa[ROW_ITEMS], fk[ROW_ITEMS], fw[ROW_ITEMS], fv[V_ITEMS], fb = 0.f;
     auto fetch = [&](int c0) {          // the chunk from token c0 on, into registers (zeros past the request's end)
@@ -125,7 +132,7 @@ scan_kernel(const ScanArgs p) {
                 const size_t row = static_cast<size_t>(start + c0 + tt);
                 fa[n] = load_any(p.a, row * p.lda + hk * D + i, p.in_bf16);
                 fk[n] = load_any(p.k, row * p.lda + hk * D + i, p.in_bf16);
-                if (RULE != kConstantDecay) fw[n] = p.w[row * H * D + h * D + i];
+                if (RULE != kConstantDecay && RULE != kTokenDecay) fw[n] = p.w[row * H * D + h * D + i];
             }
         }
 #pragma unroll
@@ -138,6 +145,8 @@ scan_kernel(const ScanArgs p) {
         }
         if (RULE == 0 && threadIdx.x < CHUNK)
             fb = c0 + threadIdx.x < len ? p.beta[static_cast<size_t>(start + c0 + threadIdx.x) * H + h] : 0.f;
+        if (RULE == kTokenDecay && threadIdx.x < CHUNK)
+            fb = c0 + threadIdx.x < len ? p.beta[static_cast<size_t>(start + c0 + threadIdx.x) * p.ld_beta + h] : 0.f;
     };
     auto stash = [&](int buf) {
 #pragma unroll
@@ -149,7 +158,7 @@ scan_kernel(const ScanArgs p) {
             if (RULE == kChannelDecay) w = i < D ? expm1f(log_sigmoid_f(w + s_w0[i]) * p.inv_tau) : 0.f;
             s_a[buf][tt][i] = RULE == kConstantDecay ? silu_f(fa[n]) : RULE == kChannelDecay ? fa[n] * p.q_scale : fa[n];
             s_k[buf][tt][i] = RULE == kConstantDecay ? silu_f(fk[n]) : fk[n];
-            if (RULE != kConstantDecay) s_w[buf][tt][i] = w;
+            if (RULE != kConstantDecay && RULE != kTokenDecay) s_w[buf][tt][i] = w;
         }
 #pragma unroll
         for (int n = 0; n < V_ITEMS; ++n) {
@@ -157,6 +166,11 @@ scan_kernel(const ScanArgs p) {
             if (idx < CHUNK * CTA_COLS) s_v[buf][idx / CTA_COLS][idx % CTA_COLS] = RULE == kConstantDecay ? silu_f(fv[n]) : fv[n];
         }
         if (RULE == 0 && threadIdx.x < CHUNK) s_beta[buf][threadIdx.x] = fb;
+        if (RULE == kTokenDecay && threadIdx.x < CHUNK) {
+            const float d = softplus_f(fb + dt_bias);
+            s_beta[buf][threadIdx.x] = d;
+            s_w[buf][threadIdx.x][0] = expm1f(-rate * d);
+        }
     };
 
     fetch(first);
@@ -220,21 +234,25 @@ scan_kernel(const ScanArgs p) {
                 }
 #pragma unroll
                 for (int c = 0; c < NC; ++c) out[c] = (acc[c][0] + acc[c][1]) + (acc[c][2] + acc[c][3]);
-            } else if (RULE == kChannelDecay || RULE == kConstantDecay) {
+            } else if (RULE == kChannelDecay || RULE == kConstantDecay || RULE == kTokenDecay) {
+                const float plain = RULE == kTokenDecay ? s_w[buf][tt][0] : fade;
+                float in[NC];           // what the memory takes of a value
+#pragma unroll
+                for (int c = 0; c < NC; ++c) in[c] = RULE == kTokenDecay ? s_beta[buf][tt] * vj[c] : vj[c];
                 float acc[NC][4];
 #pragma unroll
                 for (int c = 0; c < NC; ++c) acc[c][0] = acc[c][1] = acc[c][2] = acc[c][3] = 0.f;
 #pragma unroll
                 for (int g = 0; g < R / 4; ++g) {
                     const float4 k = k4[LANES * g], q = a4[LANES * g];
-                    float4 w = make_float4(fade, fade, fade, fade);
+                    float4 w = make_float4(plain, plain, plain, plain);
                     if (RULE == kChannelDecay) w = w4[LANES * g];
                     const float wv[4] = {w.x, w.y, w.z, w.w}, kv4[4] = {k.x, k.y, k.z, k.w}, qv[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
                     for (int c = 0; c < NC; ++c)
 #pragma unroll
                         for (int e = 0; e < 4; ++e) {
-                            S[c][4 * g + e] = fmaf(kv4[e], vj[c], fmaf(wv[e], S[c][4 * g + e], S[c][4 * g + e]));
+                            S[c][4 * g + e] = fmaf(kv4[e], in[c], fmaf(wv[e], S[c][4 * g + e], S[c][4 * g + e]));
                             acc[c][e] = fmaf(qv[e], S[c][4 * g + e], acc[c][e]);
                         }
                 }
@@ -270,6 +288,10 @@ scan_kernel(const ScanArgs p) {
             for (int o = 1; o < LANES; o <<= 1)
 #pragma unroll
                 for (int c = 0; c < NC; ++c) out[c] += __shfl_xor_sync(0xffffffffu, out[c], o);
+            if (RULE == kTokenDecay) {
+#pragma unroll
+                for (int c = 0; c < NC; ++c) out[c] = fmaf(skip, vj[c], out[c]);
+            }
             if (il == 0 && mode != 1) {
 #pragma unroll
                 for (int c = 0; c < NC; ++c)

@@ -10,15 +10,17 @@
 //                 it: 1 makes s the softmax of z over all experts, 2 makes a group's score its largest c, 4 leaves the
 //                 weights at s * route_scale (no division by their sum);
 //   moe_plan      one CTA counts the rows of every expert, lays the (token, choice) pairs out expert by expert and
-//                 writes where each pair went: `offsets` [experts + 1], `perm_token` [rows] and `row_of` [tokens, top];
+//                 writes where each pair went: `offsets` [experts + 1], `perm_token` [rows] and `row_of` [tokens, top], and
+//                 on request every row's weight;
 //   grouped_gemm  C[p, :] = act(A[src(p), :] W[e(p)]^T) for the rows p of every expert e, the tiles of all experts in
 //                 one launch (the CTA finds its expert from `offsets` on the device, so nothing goes back to the
 //                 host and the step can be replayed from a graph); float32 FMA with a fixed k order for float32
 //                 operands, tensor-core tiles (mma_tile.cuh) for bfloat16;
 //                 act 1 squares the positive part; act 2 reads W's rows as (gate, up) pairs, row 2i beside row 2i + 1,
 //                 and writes g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), N / 2 wide;
-//                 act 3 reads the same pairs and writes g sigmoid(g) u;
-//   moe_combine   out[t] = sum_k weight[t, k] * Y[row_of[t, k]] (+ a shared expert's output, optionally times the
+//                 act 3 reads the same pairs and writes g sigmoid(g) u; with `row_weight` the sums of row p are multiplied by
+//                 row_weight[p] first (the product of a row that was multiplied by it);
+//   moe_combine   out[t] = sum_k weight[t, k] * Y[row_of[t, k]] (no weights: the plain sum) (+ a shared expert's output, optionally times the
 //                 sigmoid of a per-token logit), in the order of k.
 // A row's result depends only on that row: not on the batch, nor on where the plan put it.
 #include "common.cuh"
@@ -280,7 +282,8 @@ moe_select_sigmoid_kernel(const float* __restrict__ logits, int ld, const float*
 // ids: [tokens, top] (-1: a padded token). rank_tmp: [tokens * top] scratch.
 __global__ void __launch_bounds__(256)
 moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
-                int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, int top) {
+                int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, const float* __restrict__ weights,
+                float* __restrict__ row_weight, int top) {
     pdl_trigger();
     pdl_wait();
     __shared__ int counts[kMaxExperts];
@@ -308,6 +311,7 @@ moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t
             const int row = starts[e] + rank_tmp[i];
             row_of[i] = row;
             perm_token[row] = i / top;
+            if (row_weight) row_weight[row] = weights[i];
         } else {
             row_of[i] = -1;
         }
@@ -332,7 +336,7 @@ template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256)
 grouped_gemm_kernel(const TA* __restrict__ A, int lda, const int32_t* __restrict__ row_map, const TW* __restrict__ W,
                     const int32_t* __restrict__ offsets, int experts, TC* __restrict__ C, int ldc, int N, int K, int act, float limit,
-                    float alpha) {
+                    float alpha, const float* __restrict__ row_weight) {
     pdl_trigger();
     pdl_wait();
     __shared__ float As[GK][GM + 4];
@@ -385,6 +389,11 @@ grouped_gemm_kernel(const TA* __restrict__ A, int lda, const int32_t* __restrict
     for (int i = 0; i < 4; ++i) {
         const int m = m0 + ty * 4 + i;
         if (m >= m_end) continue;
+        if (row_weight) {
+            const float f = row_weight[m];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] *= f;
+        }
         if (act >= 2) {                     // columns come in (gate, up) pairs
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
@@ -412,7 +421,7 @@ template <typename TC>
 __global__ void __launch_bounds__(128)
 grouped_gemm_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32_t* __restrict__ row_map,
                        const __nv_bfloat16* __restrict__ W, const int32_t* __restrict__ offsets, int experts, TC* __restrict__ C, int ldc,
-                       int N, int K, int act, float limit, float alpha) {
+                       int N, int K, int act, float limit, float alpha, const float* __restrict__ row_weight) {
     pdl_trigger();
     pdl_wait();
     __shared__ TileSmem sm;
@@ -436,6 +445,20 @@ grouped_gemm_tc_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32
     __syncthreads();
     float acc[2][4][4];
     mma_tile_64x64(sm, W + static_cast<size_t>(e) * N * K, K, 1, n0, N, K, acc);
+    if (row_weight) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int x = 0; x < 4; x += 2) {        // elements x and x + 1 of a fragment lie in one row
+                const int m = m0 + tile_row(i, x);
+                const float f = m < m_end ? row_weight[m] : 0.f;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    acc[i][j][x] *= f;
+                    acc[i][j][x + 1] *= f;
+                }
+            }
+    }
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -471,7 +494,7 @@ moe_combine_kernel(const float* __restrict__ Y, const int32_t* __restrict__ row_
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const int row = row_of[static_cast<size_t>(t) * top + k];
-            if (row >= 0) acc = fmaf(weights[static_cast<size_t>(t) * top + k], Y[static_cast<size_t>(row) * hidden + c], acc);
+            if (row >= 0) acc = fmaf(weights ? weights[static_cast<size_t>(t) * top + k] : 1.f, Y[static_cast<size_t>(row) * hidden + c], acc);
         }
         if (shared) acc = fmaf(share, to_f32(shared[static_cast<size_t>(t) * hidden + c]), acc);
         out[static_cast<size_t>(t) * hidden + c] = from_f32<T>(acc);
@@ -557,17 +580,19 @@ int stride_moe_select_sigmoid(const float* logits, int ld, const float* correcti
 }
 
 int stride_moe_plan(const int32_t* ids, int tokens, int top, int experts, int32_t* offsets, int32_t* perm_token, int32_t* row_of,
-                    int32_t* rank_tmp, cudaStream_t stream) {
-    if (tokens < 0 || top <= 0 || experts <= 0) return STRIDE_BAD_ARGUMENT;
+                    int32_t* rank_tmp, const float* weights, float* row_weight, cudaStream_t stream) {
+    if (tokens < 0 || top <= 0 || experts <= 0 || (row_weight && !weights)) return STRIDE_BAD_ARGUMENT;
     if (experts > kMaxExperts) return STRIDE_UNSUPPORTED;
-    stride::launch(moe_plan_kernel, dim3(1), dim3(256), 0, stream, ids, tokens * top, experts, offsets, perm_token, row_of, rank_tmp, top);
+    stride::launch(moe_plan_kernel, dim3(1), dim3(256), 0, stream, ids, tokens * top, experts, offsets, perm_token, row_of, rank_tmp, weights,
+                   row_weight, top);
     return STRIDE_LAUNCH_STATUS();
 }
 
 // kind: 0 = everything float32 (FMA); 1 = bfloat16 A and W, bfloat16 C; 2 = bfloat16 A and W, float32 C (both on the
 // tensor cores); 3 = as 2 on the FMA kernel.
 int stride_grouped_gemm(const void* A, int lda, const int32_t* row_map, const void* W, const int32_t* offsets, int experts, void* C,
-                        int ldc, int max_rows, int N, int K, int act, float limit, float alpha, int kind, cudaStream_t stream) {
+                        int ldc, int max_rows, int N, int K, int act, float limit, float alpha, const float* row_weight, int kind,
+                        cudaStream_t stream) {
     if (max_rows < 0 || experts <= 0 || N <= 0 || K <= 0 || lda < K || act < 0 || act > 3 || ldc < (act >= 2 ? N / 2 : N) || (act >= 2 && N % 2))
         return STRIDE_BAD_ARGUMENT;
     if (max_rows == 0) return 0;
@@ -577,17 +602,17 @@ int stride_grouped_gemm(const void* A, int lda, const int32_t* row_map, const vo
     static_assert(GM == TM && GN == TN, "both forms of the grouped product use tiles of one size");
     if (kind == 1)
         stride::launch(grouped_gemm_tc_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, static_cast<const __nv_bfloat16*>(A), lda, row_map,
-                       static_cast<const __nv_bfloat16*>(W), offsets, experts, static_cast<__nv_bfloat16*>(C), ldc, N, K, act, limit, alpha);
+                       static_cast<const __nv_bfloat16*>(W), offsets, experts, static_cast<__nv_bfloat16*>(C), ldc, N, K, act, limit, alpha, row_weight);
     else if (kind == 2)
         stride::launch(grouped_gemm_tc_kernel<float>, grid, dim3(128), 0, stream, static_cast<const __nv_bfloat16*>(A), lda, row_map,
-                       static_cast<const __nv_bfloat16*>(W), offsets, experts, static_cast<float*>(C), ldc, N, K, act, limit, alpha);
+                       static_cast<const __nv_bfloat16*>(W), offsets, experts, static_cast<float*>(C), ldc, N, K, act, limit, alpha, row_weight);
     else if (kind == 3)     // bfloat16 operands on the FMA kernel (kept for comparison)
         stride::launch(grouped_gemm_kernel<__nv_bfloat16, __nv_bfloat16, float>, grid, dim3(256), 0, stream,
                        static_cast<const __nv_bfloat16*>(A), lda, row_map, static_cast<const __nv_bfloat16*>(W), offsets, experts,
-                       static_cast<float*>(C), ldc, N, K, act, limit, alpha);
+                       static_cast<float*>(C), ldc, N, K, act, limit, alpha, row_weight);
     else if (kind == 0)
         stride::launch(grouped_gemm_kernel<float, float, float>, grid, dim3(256), 0, stream, static_cast<const float*>(A), lda, row_map,
-                       static_cast<const float*>(W), offsets, experts, static_cast<float*>(C), ldc, N, K, act, limit, alpha);
+                       static_cast<const float*>(W), offsets, experts, static_cast<float*>(C), ldc, N, K, act, limit, alpha, row_weight);
     else
         return STRIDE_BAD_ARGUMENT;
     return STRIDE_LAUNCH_STATUS();

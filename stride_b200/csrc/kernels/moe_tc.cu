@@ -13,7 +13,8 @@
 //
 // act 0: none; 1: the square of the positive part; 2: the rows of W come as (gate, up) pairs, row 2i beside row
 // 2i + 1, and the tile leaves g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), N / 2 wide;
-// 3: the same pairs, and the tile leaves g sigmoid(g) u.
+// 3: the same pairs, and the tile leaves g sigmoid(g) u. With `row_weight` the sums of row p are multiplied by row_weight[p]
+// before the activation.
 //
 // gather_rows lays the rows of the step's tokens out expert by expert first (xs[p] = x[perm[p]]), so that the first
 // product's A operand is one matrix a tensor map can describe; the second product's input is in that order already.
@@ -50,7 +51,7 @@ template <int BLOCK_N, int STAGES, typename OutT>
 __global__ void __launch_bounds__(kGroupThreads, 2)
 grouped_gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         const int32_t* __restrict__ offsets, int experts, OutT* __restrict__ C, int ldc, int N, int K, int act,
-                        float limit, float alpha, int vec_ok, int* __restrict__ status) {
+                        float limit, float alpha, const float* __restrict__ row_weight, int vec_ok, int* __restrict__ status) {
     constexpr int A_BYTES = kGroupM * kGroupK * 2;
     constexpr int W_BYTES = BLOCK_N * kGroupK * 2;
     constexpr int STAGE_BYTES = A_BYTES + W_BYTES;
@@ -135,12 +136,17 @@ grouped_gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
         if (ok) {
             const int width = act >= 2 ? N / 2 : N;
             OutT* crow = C + static_cast<size_t>(m) * ldc;
+            const float row_f = row_weight && m < m_end ? row_weight[m] : 1.f;
 #pragma unroll 1
             for (int c0 = 0; c0 < BLOCK_N; c0 += 32) {
                 if (n0 + c0 >= N) break;                       // uniform over the warp
                 float v[32];
                 tmem_ld32(tmem_base + (static_cast<uint32_t>(quad * 32) << 16) + c0, v);
                 if (m >= m_end) continue;
+                if (row_weight) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] *= row_f;
+                }
                 if (act >= 2) {
                     const int col = (n0 + c0) / 2;
                     float r[16];
@@ -203,7 +209,7 @@ gather_rows_kernel(const uint4* __restrict__ x, int ldx16, const int32_t* __rest
 
 template <typename OutT>
 int launch_grouped(const CUtensorMap* map_a, const CUtensorMap* map_w, const int32_t* offsets, int experts, OutT* C, int ldc, int max_rows,
-                   int N, int K, int act, float limit, float alpha, int vec_ok, int* status, cudaStream_t stream) {
+                   int N, int K, int act, float limit, float alpha, const float* row_weight, int vec_ok, int* status, cudaStream_t stream) {
     constexpr int BLOCK_N = 128, STAGES = 3;
     constexpr int smem = STAGES * (kGroupM * kGroupK * 2 + BLOCK_N * kGroupK * 2) + 1024;
     static bool configured[64] = {};
@@ -218,8 +224,8 @@ int launch_grouped(const CUtensorMap* map_a, const CUtensorMap* map_w, const int
     const int max_tiles = (max_rows + kGroupM - 1) / kGroupM + experts;       // no expert has more than one ragged tile
     if (max_tiles > 65535) return STRIDE_UNSUPPORTED;
     const dim3 grid((N + BLOCK_N - 1) / BLOCK_N, max_tiles);
-    stride::launch(kernel, grid, dim3(kGroupThreads), smem, stream, *map_a, *map_w, offsets, experts, C, ldc, N, K, act, limit, alpha, vec_ok,
-                   status);
+    stride::launch(kernel, grid, dim3(kGroupThreads), smem, stream, *map_a, *map_w, offsets, experts, C, ldc, N, K, act, limit, alpha,
+                   row_weight, vec_ok, status);
     return STRIDE_LAUNCH_STATUS();
 }
 
@@ -234,7 +240,7 @@ extern "C" {
 // C: [max_rows, N] (N / 2 with act 2 and 3), bf16 or float32. Returns -2 for what it does not take (K or lda not a multiple of
 // 8, unaligned operands); the caller then uses the other grouped product.
 int stride_grouped_gemm_tc5(const void* A, int lda, const void* W, const int32_t* offsets, int experts, void* C, int ldc, int max_rows, int N,
-                            int K, int act, float limit, float alpha, int out_is_f32, int* status, cudaStream_t stream) {
+                            int K, int act, float limit, float alpha, const float* row_weight, int out_is_f32, int* status, cudaStream_t stream) {
     if (max_rows < 0 || experts <= 0 || N <= 0 || K <= 0 || lda < K || act < 0 || act > 3 || ldc < (act >= 2 ? N / 2 : N) || (act >= 2 && N % 2))
         return STRIDE_BAD_ARGUMENT;
     if (status == nullptr) return STRIDE_BAD_ARGUMENT;
@@ -248,10 +254,10 @@ int stride_grouped_gemm_tc5(const void* A, int lda, const void* W, const int32_t
     const int elem = out_is_f32 ? 4 : 2;
     const int vec_ok = (reinterpret_cast<uintptr_t>(C) % 16 == 0 && (static_cast<long long>(ldc) * elem) % 16 == 0) ? 1 : 0;
     if (out_is_f32)
-        return tc::launch_grouped<float>(map_a, map_w, offsets, experts, static_cast<float*>(C), ldc, max_rows, N, K, act, limit, alpha, vec_ok,
-                                         status, stream);
+        return tc::launch_grouped<float>(map_a, map_w, offsets, experts, static_cast<float*>(C), ldc, max_rows, N, K, act, limit, alpha,
+                                         row_weight, vec_ok, status, stream);
     return tc::launch_grouped<__nv_bfloat16>(map_a, map_w, offsets, experts, static_cast<__nv_bfloat16*>(C), ldc, max_rows, N, K, act, limit,
-                                             alpha, vec_ok, status, stream);
+                                             alpha, row_weight, vec_ok, status, stream);
 }
 
 // xs[p] = x[perm[p]] for the rows p that the plan filled; rows of `row_bytes` (a multiple of 16), x with row stride ldx_bytes.

@@ -10,6 +10,11 @@
 //                   added, each query and key head (width hd) and each value head (width vd) is divided by its own root
 //                   mean square (no weight; either norm can be switched off), written back in place, and keys and values
 //                   go to the token's place in the pages ([page, kv_head, slot, width]) when a slot mapping is given.
+//   qkv_rotate_norm the same for projections whose queries and keys turn first: bias; the first `rot` entries of a query or
+//                   key head turn by the position's angles (entry i with entry i + rot / 2); the head is divided by its root
+//                   mean square; queries go back in place, keys and values into the pages. Values can be kept aside
+//                   (float32, per token) by one layer and blended into the values of later ones:
+//                   v <- (1 - share) v + share first. Heads may lie in columns wider than they are (zeros behind).
 //   rms_norm_cols   out[t] = x / sqrt(mean(x^2) + eps) * w for a column block x of a wider buffer (a latent between two
 //                   products): one warp a row, float32 statistics.
 // The order of every sum depends only on the row's width, never on the batch.
@@ -330,6 +335,141 @@ qkv_unit_norm_vec_kernel(T* __restrict__ qkv, int row_stride, const float* __res
     }
 }
 
+// One head a group of LANES lanes (16: two heads a warp, for heads of at most 16 packs). A head's entries pass through shared
+// memory between bias and rotation, since an entry's partner lies in another lane. hd / vd: columns of a head in the row and in
+// the pages; qd / vdim: its entries (the rest are zeros). V entries a pack: 16 bytes of the compute type where sizes and
+// pointers allow, else single entries. The order of a head's sum depends on qd, LANES and V only.
+struct RotateNormArgs {
+    void* qkv;
+    int row_stride;
+    const float* bias;
+    const int32_t* positions;
+    const float* cos_t;         // [positions, rot / 2]
+    const float* sin_t;
+    int rot;
+    const int32_t* slot_mapping;
+    void* k_pages;
+    void* v_pages;
+    int nq, nkv, hd, vd, qd, vdim, page_size;
+    float eps;
+    float* first;               // [tokens, nkv * vdim]: written when share is null, read otherwise; null: values stay as they are
+    const float* share;
+};
+
+template <typename T, int LANES, int V>
+__global__ void __launch_bounds__(kNormWarps * 32)
+qkv_rotate_norm_kernel(const RotateNormArgs p) {
+    __shared__ __align__(16) float stage[kNormWarps * (32 / LANES)][kMaxHead];
+    pdl_trigger();
+    pdl_wait();
+    constexpr int kPerWarp = 32 / LANES;
+    constexpr int kPacks = LANES == 32 ? kMaxHead / (32 * V) : 1;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & (LANES - 1), sub = (threadIdx.x & 31) / LANES;
+    const int t = blockIdx.x;
+    const int head = (blockIdx.y * kNormWarps + warp) * kPerWarp + sub;     // query heads, then key heads, then value heads
+    const bool live = head < p.nq + 2 * p.nkv;        // a group without a head still takes part in barriers and shuffles
+    const bool is_value = head >= p.nq + p.nkv;
+    const int width = live ? (is_value ? p.vdim : p.qd) : 0, cols = is_value ? p.vd : p.hd;
+    const int column = is_value ? (p.nq + p.nkv) * p.hd + (head - p.nq - p.nkv) * p.vd : head * p.hd;
+    T* x = static_cast<T*>(p.qkv) + static_cast<size_t>(t) * p.row_stride + (live ? column : 0);
+    float* mine = stage[warp * kPerWarp + sub];
+    auto load = [](const auto* from, float* v) {
+        if constexpr (V == 1) v[0] = to_f32(*from);
+        else Pack<T>::load(from, v);
+    };
+    auto load_floats = [](const float* from, float* v) {
+        if constexpr (V == 1) v[0] = *from;
+        else {
+#pragma unroll
+            for (int j = 0; j < V; j += 4) Pack<float>::load(from + j, v + j);
+        }
+    };
+    float v[kPacks][V];
+#pragma unroll
+    for (int i = 0; i < kPacks; ++i) {
+        const int d = (lane + LANES * i) * V;
+        if (d < width) {
+            load(x + d, v[i]);
+            if (p.bias) {
+                float b[V];
+                load_floats(p.bias + column + d, b);
+#pragma unroll
+                for (int j = 0; j < V; ++j) v[i][j] = __fadd_rn(v[i][j], b[j]);
+            }
+            if (!is_value) {
+#pragma unroll
+                for (int j = 0; j < V; ++j) mine[d + j] = v[i][j];
+            }
+        }
+    }
+    __syncwarp();
+    float sq = 0.f;
+    if (!is_value) {
+        const int half = p.rot / 2, at = half ? p.positions[t] : 0;
+#pragma unroll
+        for (int i = 0; i < kPacks; ++i) {
+            const int d = (lane + LANES * i) * V;
+            if (d < width) {
+                if (d < p.rot) {
+                    const float* c_row = p.cos_t + static_cast<size_t>(at) * half;
+                    const float* s_row = p.sin_t + static_cast<size_t>(at) * half;
+#pragma unroll
+                    for (int j = 0; j < V; ++j) {
+                        const int e = d + j;
+                        if (e >= p.rot) break;
+                        const bool low = e < half;
+                        const int pair = low ? e : e - half;
+                        const float c = c_row[pair], s = s_row[pair], other = mine[low ? e + half : pair];
+                        v[i][j] = low ? __fmul_rn(v[i][j], c) - __fmul_rn(other, s) : __fmul_rn(v[i][j], c) + __fmul_rn(other, s);
+                    }
+                }
+#pragma unroll
+                for (int j = 0; j < V; ++j) sq = fmaf(v[i][j], v[i][j], sq);
+            }
+        }
+    }
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if (!live) return;
+    const float inv = is_value ? 1.f : rsqrtf(sq / static_cast<float>(p.qd) + p.eps);
+    const int kvh = is_value ? head - p.nq - p.nkv : head - p.nq;
+    T* dst = x;                 // queries stay where they are; keys and values only go to the pages
+    if (head >= p.nq) {
+        const int slot = p.slot_mapping ? p.slot_mapping[t] : -1;
+        dst = slot < 0 ? nullptr
+                       : static_cast<T*>(is_value ? p.v_pages : p.k_pages) +
+                             ((static_cast<size_t>(slot / p.page_size) * p.nkv + kvh) * p.page_size + slot % p.page_size) * cols;
+    }
+    float* first = is_value && p.first ? p.first + (static_cast<size_t>(t) * p.nkv + kvh) * p.vdim : nullptr;
+    const float share = first && p.share ? *p.share : 0.f;
+#pragma unroll
+    for (int i = 0; i < kPacks; ++i) {
+        const int d = (lane + LANES * i) * V;
+        if (d >= cols) continue;
+        if (d >= width) {       // the columns behind a head's entries
+#pragma unroll
+            for (int j = 0; j < V; ++j) v[i][j] = 0.f;
+        } else if (is_value) {
+            if (first && p.share) {
+#pragma unroll
+                for (int j = 0; j < V; ++j)
+                    if (d + j < width) v[i][j] = __fadd_rn(__fmul_rn(1.f - share, v[i][j]), __fmul_rn(share, first[d + j]));
+            } else if (first) {
+#pragma unroll
+                for (int j = 0; j < V; ++j)
+                    if (d + j < width) first[d + j] = v[i][j];
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < V; ++j) v[i][j] = __fmul_rn(v[i][j], inv);
+        }
+        if (dst) {
+            if constexpr (V == 1) dst[d] = from_f32<T>(v[i][0]);
+            else Pack<T>::store(dst + d, v[i]);
+        }
+    }
+}
+
 // x: [rows, ld] from column 0 on (the caller offsets the pointer); out: [rows, ld_out]. One warp a row.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -381,6 +521,39 @@ int stride_norm_add(float* residual, const void* delta, const float* bias, const
     } else {
         return STRIDE_BAD_ARGUMENT;
     }
+    return STRIDE_LAUNCH_STATUS();
+}
+
+int stride_qkv_rotate_norm(void* qkv, int row_stride, const float* bias, const int32_t* positions, const float* cos_t, const float* sin_t,
+                           int rot, const int32_t* slot_mapping, void* k_pages, void* v_pages, int tokens, int nq, int nkv, int hd, int vd,
+                           int qd, int vdim, int page_size, float eps, float* first, const float* share, int dtype, cudaStream_t stream) {
+    if (tokens < 0 || nq < 0 || nkv < 0 || qd <= 0 || vdim <= 0 || hd < qd || vd < vdim || page_size <= 0 || rot < 0 || rot > qd || rot % 2 ||
+        row_stride < (nq + nkv) * hd + nkv * vd)
+        return STRIDE_BAD_ARGUMENT;
+    if (slot_mapping != nullptr && (k_pages == nullptr || v_pages == nullptr)) return STRIDE_BAD_ARGUMENT;
+    if ((rot > 0 && (!positions || !cos_t || !sin_t)) || (share && !first)) return STRIDE_BAD_ARGUMENT;
+    if (hd > kMaxHead || vd > kMaxHead) return STRIDE_UNSUPPORTED;
+    if (tokens == 0 || nq + nkv == 0) return 0;
+    const RotateNormArgs p = {qkv, row_stride, bias, positions, cos_t, sin_t, rot, slot_mapping, k_pages, v_pages, nq, nkv, hd, vd, qd, vdim, page_size,
+                              eps, first, share};
+    auto aligned = [](const void* q) { return reinterpret_cast<uintptr_t>(q) % 16 == 0; };
+    const int pack = dtype == STRIDE_DTYPE_F32 ? 4 : 8;
+    // packs never straddle a head's end, nor the middle of what turns
+    const bool vec = hd % pack == 0 && vd % pack == 0 && qd % pack == 0 && vdim % pack == 0 && row_stride % pack == 0 && aligned(qkv) &&
+                     aligned(bias) && aligned(k_pages) && aligned(v_pages);
+    const bool halves = vec && hd <= 16 * pack && vd <= 16 * pack;       // two heads a warp
+    const int groups = halves ? (nq + 2 * nkv + 1) / 2 : nq + 2 * nkv;
+    const dim3 grid(tokens, (groups + kNormWarps - 1) / kNormWarps), block(kNormWarps * 32);
+    if (dtype == STRIDE_DTYPE_F32)
+        stride::launch(halves ? qkv_rotate_norm_kernel<float, 16, 4> : vec ? qkv_rotate_norm_kernel<float, 32, 4> : qkv_rotate_norm_kernel<float, 32, 1>,
+                       grid, block, 0, stream, p);
+    else if (dtype == STRIDE_DTYPE_BF16)
+        stride::launch(halves ? qkv_rotate_norm_kernel<__nv_bfloat16, 16, 8>
+                       : vec  ? qkv_rotate_norm_kernel<__nv_bfloat16, 32, 8>
+                              : qkv_rotate_norm_kernel<__nv_bfloat16, 32, 1>,
+                       grid, block, 0, stream, p);
+    else
+        return STRIDE_BAD_ARGUMENT;
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -118,11 +118,11 @@ _SIGNATURES = {
     "stride_rglru_scan_pieces": ("rglru", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_moe_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
-    "stride_moe_plan": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "stride_moe_plan": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "stride_grouped_gemm": ("moe", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                    c_float, c_int, c_void_p]),
+                                    c_float, c_void_p, c_int, c_void_p]),
     "stride_grouped_gemm_tc5": ("moe_tc", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                           c_float, c_int, c_void_p, c_void_p]),
+                                           c_float, c_void_p, c_int, c_void_p, c_void_p]),
     "stride_gather_rows": ("moe_tc", [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p]),
     "stride_moe_combine": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_relu_squared": ("moe", [c_void_p, c_longlong, c_int, c_void_p]),
@@ -133,6 +133,8 @@ _SIGNATURES = {
                                       c_void_p, c_int, c_void_p]),
     "stride_qkv_unit_norm": ("unit_norm", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                            c_float, c_int, c_int, c_int, c_void_p]),
+    "stride_qkv_rotate_norm": ("unit_norm", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p]),
     "stride_moe_select_sigmoid": ("moe", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                           c_void_p]),
     "stride_moe_select_groups": ("moe", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -150,6 +152,20 @@ _SIGNATURES = {
                                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_copies_step": ("stream_copies", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
                                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_ssm_conv": ("state_space", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p,
+                                        c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "stride_ssm_tail": ("state_space", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                                        c_int, c_void_p]),
+    "stride_ssm_scan": ("state_space", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                        c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_ssm_step": ("state_space", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                        c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                        c_int, c_int, c_void_p]),
+    "stride_ssm_chunks": ("state_space", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                          c_longlong, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                          c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
+    "stride_gated_group_norm": ("state_space", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int,
+                                                c_void_p]),
     "stride_decay_scan": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
                                            c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_decay_step": ("decay_memory", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
@@ -203,6 +219,7 @@ _CLASS_OF = {
     "stride_side_gate": "token side input", "stride_side_norm_add": "token side input", "stride_cast_rows": "token side input",
     "stride_moe_select": "router", "stride_moe_select_sigmoid": "router", "stride_moe_select_groups": "router", "stride_head_gate": "gates and caps",
     "stride_add_sinusoid": "embedding", "stride_norm_add": "norm", "stride_qkv_unit_norm": "head norms + cache write",
+    "stride_qkv_rotate_norm": "rotation + head norms + cache write",
     "stride_rglru_conv": "recurrent block: convolution",
     "stride_rglru_gates": "recurrent block: gates", "stride_rglru_scan": "recurrent block: recurrence", "stride_rglru_scan_pieces": "recurrent block: recurrence", "stride_moe_route": "router",
     "stride_moe_plan": "router", "stride_grouped_gemm": "expert products", "stride_moe_combine": "expert sum",
@@ -217,6 +234,9 @@ _CLASS_OF = {
     "stride_conv_row_norm": "convolution + row norms + cache write", "stride_copies_step": "residual copies + norm",
     "stride_decay_scan": "fading memory: recurrence", "stride_decay_chunks": "fading memory: recurrence",
     "stride_decay_step": "fading memory: recurrence",
+    "stride_ssm_conv": "state space: convolution", "stride_ssm_tail": "state space: convolution", "stride_ssm_scan": "state space: recurrence",
+    "stride_ssm_step": "state space: recurrence", "stride_ssm_chunks": "state space: recurrence",
+    "stride_gated_group_norm": "gate + norm of parts",
     "stride_paged_decode_attention_biased": "attention (decode)",
 }
 
@@ -572,6 +592,27 @@ def shift_mix(x, mu, state, prev_off: int, seq_of_token, q_start, q_len, state_s
         _dev(state_slot, "state_slot", torch.int32), _dev(out, "out"), tokens, width, mixes, _code(x.dtype), _stream()), "shift_mix")
 
 
+def qkv_rotate_norm(qkv, bias, positions, cos, sin, rot: int, slot_mapping, k_pages, v_pages, nq: int, nkv: int, hd: int, vd: int, qd: int,
+                    vdim: int, page_size: int, eps: float, first=None, share=None) -> None:
+    """In a fused projection [q heads | k heads | v heads] (heads of ``qd`` / ``vdim`` entries in columns of ``hd`` / ``vd``): the bias; the
+    first ``rot`` entries of query and key heads turn by ``cos`` / ``sin`` (float32 [positions, rot / 2], entry i with i + rot / 2) and
+    the heads are divided by their root mean square. Queries go back in place, keys and values into the pages. ``first`` (float32
+    [tokens, nkv * vdim]) without ``share``: receives the values; with ``share`` (float32, one number): values become
+    ``(1 - share) v + share first``."""
+    tokens = qkv.shape[0]
+    if rot and (cos.shape[1] != rot // 2 or sin.shape != cos.shape):
+        raise KernelError("qkv_rotate_norm: the tables must have one column per turned pair")
+    if first is not None and first.shape != (tokens, nkv * vdim):
+        raise KernelError("qkv_rotate_norm: the values kept aside must be [tokens, nkv * vdim]")
+    if k_pages is not None and (k_pages.shape[-1] != hd or v_pages.shape[-1] != vd):
+        raise KernelError("qkv_rotate_norm: the pages have the wrong width")
+    _check(_fn("stride_qkv_rotate_norm")(
+        _dev(qkv, "qkv"), qkv.shape[1], _opt(bias, "bias", torch.float32), _dev(positions, "positions", torch.int32),
+        _dev(cos, "cos", torch.float32), _dev(sin, "sin", torch.float32), int(rot), _opt(slot_mapping, "slot_mapping", torch.int32),
+        _opt(k_pages, "k_pages", qkv.dtype), _opt(v_pages, "v_pages", qkv.dtype), tokens, nq, nkv, hd, vd, qd, vdim, page_size, float(eps),
+        _opt(first, "first", torch.float32), _opt(share, "share", torch.float32), _code(qkv.dtype), _stream()), "qkv_rotate_norm")
+
+
 def head_norm_gate(o, weight, per_head_weight: bool, gate, gate_kind: str, out, H: int, DV: int, eps: float, gate_off: int = 0) -> None:
     """``out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * weight * gate`` per head. ``weight`` [DV] for all heads or
     [H * DV]; ``gate`` [tokens, >= gate_off + H * DV], read from column ``gate_off`` on: ``sigmoid`` of float32 values or
@@ -660,6 +701,132 @@ def decay_chunks(proj, q_off: int, k_off: int, v_off: int, logit, bias, powers, 
         _dev(o, "o", torch.float32), *_state_rows(state), _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
         _dev(state_slot, "state_slot", torch.int32), int(num_seqs), H, D, DV, _code(proj.dtype), -(-max_q_len // DECAY_CHUNK),
         _dev(scratch, "scratch", torch.float32), _stream()), "decay_chunks")
+
+
+# ----------------------------------------------------------------------- selective state space
+# Portions of at least this many tokens run chunk by chunk in bfloat16 models (0: none do).
+SSM_CHUNKS_MIN_TOKENS = int(_os.environ.get("STRIDE_B200_SSM_CHUNKS_MIN", "48"))
+SSM_CHUNK = 128
+
+
+class SsmShape:
+    """Sizes of the memory, its step sizes' and skip's vectors (float32 [H]) and the convolution (``w`` float32 [taps, channels], ``b``
+    float32 [channels], channels = H P + 2 G N in the order x, B, C)."""
+
+    def __init__(self, H: int, G: int, N: int, P: int, taps: int, dt_bias, a_log, skip, w, b):
+        self.H, self.G, self.N, self.P, self.taps = H, G, N, P, taps
+        self.dt_bias, self.a_log, self.skip, self.w, self.b = dt_bias, a_log, skip, w, b
+        self.channels = H * P + 2 * G * N
+        self.ring_off = -(-H * N * P // 4) * 4         # a request's state row: S of every head, then the ring of the convolution's inputs
+
+    def state_floats(self) -> int:
+        return self.ring_off + (self.taps * self.channels if self.taps > 1 else 0)
+
+    def vectors(self) -> tuple:
+        f32 = torch.float32
+        return _dev(self.dt_bias, "dt_bias", f32), _dev(self.a_log, "a_log", f32), _dev(self.skip, "skip", f32)
+
+    def check(self, state, what: str) -> None:
+        if state.shape[1] < self.state_floats():
+            raise KernelError(f"{what}: the state rows are too short")
+        if self.w.shape != (self.taps, self.channels) or self.b.shape != (self.channels,):
+            raise KernelError(f"{what}: the convolution's weights must be [taps, channels], its bias [channels]")
+
+
+def _ssm_input(proj, off: int, channels: int) -> tuple:
+    """(pointer, columns of a row, is bfloat16) of the convolved columns of a projection."""
+    if proj.dtype not in DTYPE_CODE or proj.shape[1] < off + channels:
+        raise KernelError("the projection must be float32 or bfloat16 and hold every convolved channel")
+    return _dev(proj, "proj") + off * proj.element_size(), proj.shape[1], _code(proj.dtype)
+
+
+def ssm_conv(s: SsmShape, proj, off: int, state, seq_of_token, q_start, positions, state_slot, out) -> None:
+    """``out[t] = silu(b + sum_j w[j] u_(t - taps + 1 + j))`` per channel for every row of ``out``; ``u``: the columns of ``proj`` from
+    ``off`` on, before a request's first row of the step the ring in its state row."""
+    s.check(state, "ssm_conv")
+    tokens = out.shape[0]
+    if proj.shape[0] < tokens or out.shape[1] < s.channels or seq_of_token.numel() < tokens:
+        raise KernelError("ssm_conv: shapes do not agree")
+    pointer, stride = _state_rows(state)
+    _check(_fn("stride_ssm_conv")(
+        *_ssm_input(proj, off, s.channels), s.channels, s.taps, _dev(s.w, "w", torch.float32), _dev(s.b, "b", torch.float32),
+        pointer + 4 * s.ring_off, stride, _dev(seq_of_token, "seq_of_token", torch.int32), _dev(q_start, "q_start", torch.int32),
+        _dev(positions, "positions", torch.int32), _dev(state_slot, "state_slot", torch.int32), _dev(out, "out"), out.shape[1], tokens,
+        _code(out.dtype), _stream()), "ssm_conv")
+
+
+def ssm_tail(s: SsmShape, proj, off: int, state, q_start, q_len, positions, state_slot, num_seqs: int) -> None:
+    """The rings of the first ``num_seqs`` requests take up the last inputs of their tokens of this step."""
+    s.check(state, "ssm_tail")
+    if s.taps == 1:
+        return
+    pointer, stride = _state_rows(state)
+    _check(_fn("stride_ssm_tail")(
+        *_ssm_input(proj, off, s.channels), s.channels, s.taps, pointer + 4 * s.ring_off, stride, _dev(q_start, "q_start", torch.int32),
+        _dev(q_len, "q_len", torch.int32), _dev(positions, "positions", torch.int32), _dev(state_slot, "state_slot", torch.int32),
+        int(num_seqs), _stream()), "ssm_tail")
+
+
+def _ssm_args(s: SsmShape, u, raw, raw_off: int, y) -> tuple:
+    if u.shape[1] < s.channels or y.shape[1] != s.H * s.P or raw.dtype != torch.float32 or raw.shape[1] < raw_off + s.H:
+        raise KernelError("state space memory: shapes do not agree, or the step sizes are not float32")
+    p, item = _dev(u, "u"), u.element_size()
+    return (p, p + s.H * s.P * item, p + (s.H * s.P + s.G * s.N) * item, u.shape[1], _dev(raw, "raw") + 4 * raw_off, raw.shape[1],
+            *s.vectors(), _dev(y, "y", torch.float32))
+
+
+def ssm_scan(s: SsmShape, u, raw, raw_off: int, y, state, q_start, q_len, state_slot, num_seqs: int) -> None:
+    """Per head ``d = softplus(raw + dt_bias); S = exp(-exp(a_log) d) S + d B x^T; y = S^T C + skip x``, in token order. ``u`` [tokens, >=
+    channels]: x, B, C behind the convolution; ``raw`` float32, read from column ``raw_off`` on; ``y`` float32 [tokens, H * P]."""
+    s.check(state, "ssm_scan")
+    _check(_fn("stride_ssm_scan")(*_ssm_args(s, u, raw, raw_off, y), *_state_rows(state), _dev(q_start, "q_start", torch.int32),
+                                  _dev(q_len, "q_len", torch.int32), _dev(state_slot, "state_slot", torch.int32), int(num_seqs), s.H, s.G, s.N,
+                                  s.P, _code(u.dtype), _stream()), "ssm_scan")
+
+
+def ssm_step_supported(s: SsmShape, state) -> bool:
+    return s.P % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0 and s.N <= 256 and s.taps <= 16
+
+
+def ssm_step(s: SsmShape, proj, off: int, raw, raw_off: int, y, state, q_start, q_len, positions, state_slot, num_seqs: int) -> None:
+    """Convolution, recurrence and the ring's new row for requests that bring one token each."""
+    s.check(state, "ssm_step")
+    if y.shape[1] != s.H * s.P or raw.dtype != torch.float32 or raw.shape[1] < raw_off + s.H:
+        raise KernelError("ssm_step: shapes do not agree, or the step sizes are not float32")
+    _check(_fn("stride_ssm_step")(
+        *_ssm_input(proj, off, s.channels), _dev(raw, "raw") + 4 * raw_off, raw.shape[1], _dev(s.w, "w", torch.float32),
+        _dev(s.b, "b", torch.float32), *s.vectors(), _dev(y, "y", torch.float32), *_state_rows(state), s.ring_off,
+        _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(positions, "positions", torch.int32),
+        _dev(state_slot, "state_slot", torch.int32), int(num_seqs), s.H, s.G, s.N, s.P, s.taps, _stream()), "ssm_step")
+
+
+def ssm_chunks_scratch_floats(s: SsmShape, num_seqs: int, max_q_len: int) -> int:
+    return num_seqs * -(-max_q_len // SSM_CHUNK) * s.H * (s.N * s.P + 1)
+
+
+def ssm_chunks(s: SsmShape, u, raw, raw_off: int, y, state, proj, off: int, q_start, q_len, positions, state_slot, num_seqs: int,
+               max_q_len: int, scratch) -> None:
+    """``ssm_scan`` and ``ssm_tail`` in one (bfloat16 ``u``), the chunks of every portion side by side, sums in another order.
+    ``scratch``: ``ssm_chunks_scratch_floats``."""
+    s.check(state, "ssm_chunks")
+    if u.dtype != torch.bfloat16 or scratch.numel() < ssm_chunks_scratch_floats(s, num_seqs, max_q_len):
+        raise KernelError("ssm_chunks: bfloat16 inputs and a large enough scratch are needed")
+    pu, ld_u, u_bf16 = _ssm_input(proj, off, s.channels)
+    _check(_fn("stride_ssm_chunks")(
+        *_ssm_args(s, u, raw, raw_off, y), *_state_rows(state), s.ring_off, pu, ld_u, u_bf16, s.taps, _dev(q_start, "q_start", torch.int32),
+        _dev(q_len, "q_len", torch.int32), _dev(positions, "positions", torch.int32), _dev(state_slot, "state_slot", torch.int32), int(num_seqs),
+        s.H, s.G, s.N, s.P, -(-max_q_len // SSM_CHUNK), _dev(scratch, "scratch", torch.float32), _stream()), "ssm_chunks")
+
+
+def gated_group_norm(y, z, z_off: int, weight, out, parts: int, eps: float) -> None:
+    """``out = weight u / sqrt(mean(u^2) + eps)`` with ``u = y silu(z)``, the mean over each of ``parts`` equal parts of a row. ``z``: float32
+    or ``out``'s type, read from column ``z_off`` on."""
+    tokens, width = out.shape
+    if y.shape != out.shape or z.shape[0] < tokens or z.shape[1] < z_off + width or weight.numel() != width or width % parts:
+        raise KernelError("gated_group_norm: shapes do not agree")
+    _check(_fn("stride_gated_group_norm")(_dev(y, "y", torch.float32), _dev(z, "z") + z_off * z.element_size(), z.shape[1], _code(z.dtype),
+                                          _dev(weight, "weight", torch.float32), _dev(out, "out"), tokens, width, int(parts), float(eps),
+                                          _code(out.dtype), _stream()), "gated_group_norm")
 
 
 # ------------------------------------------------------------ a residual stream in several copies
@@ -989,18 +1156,20 @@ def moe_select_groups(logits, correction, seq_of_token, ids, weights, experts: i
                                            int(keep), float(route_scale), rule, _stream()), "moe_select_groups")
 
 
-def moe_plan(ids, experts: int, offsets, perm_token, row_of, rank_tmp) -> None:
+def moe_plan(ids, experts: int, offsets, perm_token, row_of, rank_tmp, weights=None, row_weight=None) -> None:
+    """``row_weight`` (float32, one per row; with ``weights`` [tokens, top]) receives every row's weight."""
     tokens, top = ids.shape
     _check(_fn("stride_moe_plan")(_dev(ids, "ids", torch.int32), tokens, top, experts, _dev(offsets, "offsets", torch.int32),
                                   _dev(perm_token, "perm_token", torch.int32), _dev(row_of, "row_of", torch.int32),
-                                  _dev(rank_tmp, "rank_tmp", torch.int32), _stream()), "moe_plan")
+                                  _dev(rank_tmp, "rank_tmp", torch.int32), _opt(weights, "weights", torch.float32),
+                                  _opt(row_weight, "row_weight", torch.float32), _stream()), "moe_plan")
 
 
-def grouped_gemm(a, row_map, w, offsets, c, max_rows: int, act: int = 0, limit: float = 0.0, alpha: float = 1.0) -> None:
+def grouped_gemm(a, row_map, w, offsets, c, max_rows: int, act: int = 0, limit: float = 0.0, alpha: float = 1.0, row_weight=None) -> None:
     """For every expert e and row p in ``offsets[e] .. offsets[e+1]``: ``c[p] = act(a[row_map[p]] @ w[e].T)`` (``row_map`` None:
     row p itself). ``w`` [experts, n, k]; ``act`` 1 squares the positive part; ``act`` 2 takes rows 2i and 2i + 1 of ``w[e]`` as
     gate and up of unit i and leaves ``g' sigmoid(alpha g') (u' + 1)`` (clamped at ``limit``) in ``c`` [rows, n / 2]; ``act`` 3
-    takes the same pairs and leaves ``g sigmoid(g) u``."""
+    takes the same pairs and leaves ``g sigmoid(g) u``. ``row_weight`` (float32, one per row) multiplies a row's sums before the activation."""
     experts, n, k = w.shape
     if a.dtype == torch.float32:
         kind = 0
@@ -1010,7 +1179,7 @@ def grouped_gemm(a, row_map, w, offsets, c, max_rows: int, act: int = 0, limit: 
         kind = 2
     _check(_fn("stride_grouped_gemm")(_dev(a, "a"), a.shape[1], _opt(row_map, "row_map", torch.int32), _dev(w, "w", a.dtype),
                                       _dev(offsets, "offsets", torch.int32), experts, _dev(c, "c"), c.shape[1], int(max_rows), n, k, int(act),
-                                      float(limit), float(alpha), kind, _stream()), "grouped_gemm")
+                                      float(limit), float(alpha), _opt(row_weight, "row_weight", torch.float32), kind, _stream()), "grouped_gemm")
 
 
 # Steps with at least this many (token, choice) rows run the experts' products on the tcgen05 kernel (128-row tiles
@@ -1036,7 +1205,7 @@ def gather_rows(x, perm, offsets, experts: int, xs, max_rows: int) -> bool:
     return True
 
 
-def grouped_gemm_tc(a, w, offsets, c, max_rows: int, act: int = 0, limit: float = 0.0, alpha: float = 1.0) -> bool:
+def grouped_gemm_tc(a, w, offsets, c, max_rows: int, act: int = 0, limit: float = 0.0, alpha: float = 1.0, row_weight=None) -> bool:
     """``grouped_gemm`` without a row map (row p of ``a`` belongs to the expert whose range holds p) on the tcgen05 kernel,
     bfloat16 operands, ``c`` bfloat16 or float32. False when it does not take the sizes (nothing was done)."""
     experts, n, k = w.shape
@@ -1044,7 +1213,7 @@ def grouped_gemm_tc(a, w, offsets, c, max_rows: int, act: int = 0, limit: float 
         return False
     code = _fn("stride_grouped_gemm_tc5")(_dev(a, "a"), a.stride(0), _dev(w, "w"), _dev(offsets, "offsets", torch.int32), experts, _dev(c, "c"),
                                           c.shape[1], int(max_rows), n, k, int(act), float(limit), float(alpha),
-                                          1 if c.dtype == torch.float32 else 0, _status_ptr(a.device), _stream())
+                                          _opt(row_weight, "row_weight", torch.float32), 1 if c.dtype == torch.float32 else 0, _status_ptr(a.device), _stream())
     if code == -2:
         return False
     _check(code, "grouped_gemm_tc5")
@@ -1052,13 +1221,13 @@ def grouped_gemm_tc(a, w, offsets, c, max_rows: int, act: int = 0, limit: float 
 
 
 def moe_combine(y, row_of, weights, shared, out, shared_gate=None) -> None:
-    """``shared_gate``: a float32 column (one logit per token, possibly a column of a wider buffer); the shared expert's
+    """``weights`` None: the plain sum of a token's rows. ``shared_gate``: a float32 column (one logit per token, possibly a column of a wider buffer); the shared expert's
     output is then multiplied by its sigmoid."""
     tokens, hidden = out.shape
     gate_ptr, gate_stride = (None, 0) if shared_gate is None else (shared_gate.data_ptr(), shared_gate.stride(0))
     if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.shape[0] != tokens):
         raise KernelError("moe_combine: the shared expert's gate must be one float32 logit per token")
-    _check(_fn("stride_moe_combine")(_dev(y, "y", torch.float32), _dev(row_of, "row_of", torch.int32), _dev(weights, "weights", torch.float32),
+    _check(_fn("stride_moe_combine")(_dev(y, "y", torch.float32), _dev(row_of, "row_of", torch.int32), _opt(weights, "weights", torch.float32),
                                      _opt(shared, "shared", out.dtype), gate_ptr, gate_stride, _dev(out, "out"), tokens, hidden,
                                      row_of.shape[1], _code(out.dtype), _stream()), "moe_combine")
 

@@ -21,6 +21,13 @@ Spec params, all optional:
 * ``value_dim``: the width of a value head where it is not the keys' (keys and values then lie in pages of their own width).
 * ``qk_norm`` / ``v_norm`` ``unit``: every query and key head / every value head is divided by its root mean square
   (``norm_eps`` inside the root, no weight) after the bias and before any rotation; keys and values are kept so.
+* ``qk_norm`` ``unit_rotated``: the same unit norm on queries and keys behind the rotation (of the first entries of a head, halves
+  paired). One kernel adds the biases, turns, norms, mixes values (below) and writes the pages.
+* ``value_mix`` ``first`` | ``later``, with ``qk_norm`` ``unit_rotated``: a tensor ``vmix`` of one number. The layer called ``first`` leaves
+  its values of the step's tokens in a float32 buffer of the runtime; a ``later`` one uses (and keeps in its pages)
+  ``(1 - vmix) v + vmix v_first``. ``first`` does not read its own number.
+* ``padded_heads``, with ``qk_norm`` ``unit_rotated``: in bfloat16, heads of a size that the tensor-core attention kernels lack are laid out
+  with zeros up to the next one they have, where that at most doubles what a token keeps.
 * ``distance_slopes`` c: head h of H takes ``2^(-c (h + 1) / H) * (i - j)`` off the score of query i and key j (Press et
   al., "Train Short, Test Long: Attention with Linear Biases Enables Input Length Extrapolation", with c = 8).
 * ``output_bias``: a bias ``o.b`` on the output projection. The mixer hands it out as ``output_bias`` and the layer's
@@ -115,6 +122,9 @@ class PagedAttention(Mixer):
         self.short_names = p.get("names") == "short"
         self.vd = int(p.get("value_dim", self.hd))
         self.unit_qk, self.unit_v = p.get("qk_norm") == "unit", p.get("v_norm") == "unit"
+        self.unit_rotated, self.value_mix, self.v_share = p.get("qk_norm") == "unit_rotated", p.get("value_mix"), None
+        if self.value_mix not in (None, "first", "later") or (self.value_mix and not self.unit_rotated):
+            raise ValueError("values are mixed with those of a first layer, behind unit norms on rotated queries and keys")
         self.norm_eps = float(p.get("norm_eps", 0.0))
         self.head_gate = p.get("output_gate") == "head"
         self.has_output_bias, self.borrows = bool(p.get("output_bias", False)), bool(p.get("borrowed_kv", False))
@@ -131,8 +141,19 @@ class PagedAttention(Mixer):
                                or not self.short_names or self.taps > 16):
             raise ValueError("a convolution, weighted head norms or norms over whole projections go with no rotation, no biases, no unit norms, no borrowed pages, "
                              "no per-head gate, short tensor names and at most 16 taps")
-        self.own_prepare = self.unit_qk or self.unit_v or self.vd != self.hd or self.borrows or self.conv_path
-        if self.own_prepare and not self.plain_position and (self.vd != self.hd or self.borrows):
+        self.own_prepare = self.unit_qk or self.unit_v or self.vd != self.hd or self.borrows or self.conv_path or self.unit_rotated
+        if self.unit_rotated and (self.conv_path or self.unit_v or self.values_are_keys or self.borrows or self.plain_position or self.head_gate
+                                  or p.get("output_gate")):
+            raise ValueError("unit norms behind the rotation go with a rotation and with none of convolution, value norms, gates, borrowed "
+                             "pages and values taken from keys")
+        # the sizes of a head in memory: the stated ones, or padded with zeros to a size of the tensor-core kernels
+        self.head_q, self.head_v = self.hd, self.vd
+        if p.get("padded_heads") and self.unit_rotated and runtime.dtype == torch.bfloat16:
+            size = next((n for n in (64, 128) if n >= max(self.hd, self.vd)), 0)
+            if size and 2 * size <= 2 * (self.hd + self.vd) and ops.fast_attention_supported(runtime.dtype, self.nq, self.nkv, size):
+                self.hd = self.vd = size
+                self.q_dim, self.kv_dim = self.nq * size, self.nkv * size
+        if self.own_prepare and not self.unit_rotated and not self.plain_position and (self.vd != self.hd or self.borrows):
             raise ValueError("a rotation with borrowed pages or a value width of its own is not supported")
         self.fused_gate = self.head_gate and self.own_prepare and self.plain_position
         slope_c = p.get("distance_slopes")
@@ -143,7 +164,7 @@ class PagedAttention(Mixer):
         # gate columns are padded so that every row of the fused buffer starts on a 16-byte boundary
         self.gate_cols = -(-self.nq // 8) * 8 if self.fused_gate else 0
         self.qkv_dim = self.q_dim + self.kv_cols + self.gate_cols
-        permutation = getattr(self.position, "head_permutation", lambda: None)()
+        permutation = None if self.unit_rotated else getattr(self.position, "head_permutation", lambda: None)()
         self.perm = None if permutation is None else torch.tensor(permutation, dtype=torch.long)
         self.w_qkv = self.w_o = self.bias = self.w_gate = self.sinks = self.conv_w = self.wq_norm = self.wk_norm = None
         if self.zero_sinks:
@@ -164,17 +185,20 @@ class PagedAttention(Mixer):
 
     def declare(self):
         w, b = self._names()
-        d = {w["q"]: TensorDecl((self.q_dim, self.hidden)), w["o"]: TensorDecl((self.hidden, self.o_in))}
+        q_dim, kv_dim, v_dim = self.nq * self.head_q, self.nkv * self.head_q, self.nkv * self.head_v      # as stored
+        d = {w["q"]: TensorDecl((q_dim, self.hidden)), w["o"]: TensorDecl((self.hidden, self.nq * self.head_v))}
         if not self.borrows:
-            d[w["k"]] = TensorDecl((self.kv_dim, self.hidden))
+            d[w["k"]] = TensorDecl((kv_dim, self.hidden))
             if not self.values_are_keys:
-                d[w["v"]] = TensorDecl((self.v_dim, self.hidden))
+                d[w["v"]] = TensorDecl((v_dim, self.hidden))
         if self.spec.bias:
-            d[b["q"]] = TensorDecl((self.q_dim,), "vector")
+            d[b["q"]] = TensorDecl((q_dim,), "vector")
             if not self.borrows:
-                d[b["k"]] = TensorDecl((self.kv_dim,), "vector")
+                d[b["k"]] = TensorDecl((kv_dim,), "vector")
                 if not self.values_are_keys:
-                    d[b["v"]] = TensorDecl((self.v_dim,), "vector")
+                    d[b["v"]] = TensorDecl((v_dim,), "vector")
+        if self.value_mix:
+            d[self.spec.prefix + "vmix"] = TensorDecl((), "vector")
         if self.has_output_bias:
             d[b["o"]] = TensorDecl((self.hidden,), "vector")
         if self.gated:
@@ -201,6 +225,28 @@ class PagedAttention(Mixer):
         heads = t.shape[dim] // self.hd
         index = (torch.arange(heads)[:, None] * self.hd + perm[None, :]).reshape(-1).to(t.device)
         return t.index_select(dim, index).contiguous()
+
+    def _sizes(self, name):
+        """(heads, size as stored, size in memory) of a projection's heads."""
+        return {"q": (self.nq, self.head_q, self.hd), "k": (self.nkv, self.head_q, self.hd), "v": (self.nkv, self.head_v, self.vd),
+                "o": (self.nq, self.head_v, self.vd)}[name]
+
+    def _padded(self, t, name, dim: int = 0):
+        """``t`` with the heads along ``dim`` at their size in memory, zeros behind the stored entries."""
+        heads, stored, size = self._sizes(name)
+        if stored == size:
+            return t
+        shape = list(t.shape)
+        out = torch.zeros((*shape[:dim], heads, size, *shape[dim + 1:]), dtype=t.dtype, device=t.device)
+        out.narrow(dim + 1, 0, stored).copy_(t.reshape(*shape[:dim], heads, stored, *shape[dim + 1:]))
+        return out.reshape(*shape[:dim], heads * size, *shape[dim + 1:])
+
+    def _unpadded(self, t, name, dim: int = 0):
+        heads, stored, size = self._sizes(name)
+        if stored == size:
+            return t
+        shape = list(t.shape)
+        return t.reshape(*shape[:dim], heads, size, *shape[dim + 1:]).narrow(dim + 1, 0, stored).reshape(*shape[:dim], heads * stored, *shape[dim + 1:])
 
     def bind(self, weights):
         w, b = self._names()
@@ -229,13 +275,15 @@ class PagedAttention(Mixer):
         if self.perm is not None:
             raise ValueError("head norms are not combined with a rotation that reorders the heads' entries")
         order = ["q"] + ([] if self.borrows else ["k", "v"])
-        rows = [weights[w[n]] for n in order] + ([weights[w["g"]]] if self.fused_gate else [])
+        rows = [self._padded(weights[w[n]], n) for n in order] + ([weights[w["g"]]] if self.fused_gate else [])
         if self.gate_cols > self.nq:
             rows.append(torch.zeros((self.gate_cols - self.nq, self.hidden), dtype=rows[0].dtype, device=rows[0].device))
         self.w_qkv = torch.cat(rows, dim=0).contiguous()
-        self.w_o = weights[w["o"]]
+        self.w_o = self._padded(weights[w["o"]], "o", 1)
         if self.spec.bias:
-            self.bias = torch.cat([weights[b[n]] for n in order]).contiguous()
+            self.bias = torch.cat([self._padded(weights[b[n]], n) for n in order]).contiguous()
+        if self.value_mix:
+            self.v_share = weights[self.spec.prefix + "vmix"]
         if self.gated and not self.fused_gate:
             self.w_gate = weights[w["g"]]
         if self.has_sinks:
@@ -262,11 +310,11 @@ class PagedAttention(Mixer):
 
     def _named_own(self):
         w, b = self._names()
-        out, at = {w["o"]: self.w_o}, 0
+        out, at = {w["o"]: self._unpadded(self.w_o, "o", 1)}, 0
         for n, rows in [("q", self.q_dim)] + ([] if self.borrows else [("k", self.kv_dim), ("v", self.v_dim)]):
-            out[w[n]] = self.w_qkv[at:at + rows]
+            out[w[n]] = self._unpadded(self.w_qkv[at:at + rows], n)
             if self.bias is not None:
-                out[b[n]] = self.bias[at:at + rows]
+                out[b[n]] = self._unpadded(self.bias[at:at + rows], n)
             at += rows
         if self.gated:
             out[w["g"]] = self.w_qkv[at:at + self.nq] if self.fused_gate else self.w_gate
@@ -275,6 +323,8 @@ class PagedAttention(Mixer):
         if self.has_output_bias:
             out[b["o"]] = self.output_bias
         p = self.spec.prefix
+        if self.value_mix:
+            out[p + "vmix"] = self.v_share
         if self.taps:
             q, k = self.q_dim, self.q_dim + self.kv_dim
             stored = self.conv_w.t()
@@ -386,8 +436,15 @@ class PagedAttention(Mixer):
             ops.conv_tail(raw, state, 0, ctx.q_start, ctx.q_len, ctx.state_slot, sequence_slots(ctx), self.qkv_dim, self.taps)
 
     def _norm_and_store(self, qkv, ctx, cache, tokens):
-        """Bias, head norms and the pages: in one kernel when there is no rotation, else the norms here and rotation and
-        pages through the position part."""
+        """Bias, head norms and the pages: in one kernel when there is no rotation or the norms come behind it, else the norms
+        here and rotation and pages through the position part."""
+        if self.unit_rotated:
+            cos, sin = self.position.plain_tables()
+            first = self.rt.buffer("first_values", tokens, self.nkv * self.head_v, torch.float32) if self.value_mix else None
+            ops.qkv_rotate_norm(qkv, self.bias, ctx.positions[:tokens], cos, sin, self.position.rotated,
+                                ctx.slot_mapping[cache.group][:tokens] if cache.writes else None, cache.k_pages, cache.v_pages, self.nq, self.nkv,
+                                self.hd, self.vd, self.head_q, self.head_v, cache.page_size, self.norm_eps, first, self.v_share if self.value_mix == "later" else None)
+            return
         writes = cache.writes and not self.borrows
         nkv = 0 if self.borrows else self.nkv
         if self.plain_position:

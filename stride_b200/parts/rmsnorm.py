@@ -6,7 +6,7 @@ Spec params: ``tensor`` names the weight (default: the prefix + ``weight``); ``w
 ``shape`` ``scalar``: the checkpoint keeps one number for all coordinates (a tensor without dimensions), which is spread
 over the width when it is bound, so every kernel sees a vector; ``scale_tensor`` names a second vector [width] (a learned scale
 on what a sublayer adds to the stream) that multiplies the norm's output element by element: the two are one float32 factor
-from load on.
+from load on; ``factor`` f multiplies the norm's output by a number (a scale on the logits, say, where the head follows).
 
 Besides the pre-norm use (``apply``) the norm can sit on a sublayer's output: ``add_normed`` adds ``mult * norm(delta)``
 to the residual stream."""
@@ -28,6 +28,7 @@ class RMSNorm(Norm):
         self.offset = float(p.get("weight_offset", 0.0))
         self.scalar = p.get("shape") == "scalar"
         self._scale_name = p.get("scale_tensor")
+        self.factor = float(p.get("factor", 1.0))
         self.stored = self.stored_scale = None
 
     def declare(self):
@@ -43,6 +44,8 @@ class RMSNorm(Norm):
         if self._scale_name:
             self.stored_scale = weights[self._scale_name]
             self.weight = (self.weight * self.stored_scale).contiguous()
+        if self.factor != 1.0:
+            self.weight = self.weight * self.factor
 
     def named_tensors(self):
         out = {self._name: self.stored}

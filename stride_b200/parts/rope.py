@@ -33,8 +33,8 @@ from ..csrc import ops
 from .base import PositionEncoding, register_part
 
 
-def rope_inverse_frequencies(head_dim: int, theta: float, scaling) -> torch.Tensor:
-    inv_freq = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=torch.float32) / head_dim))
+def rope_inverse_frequencies(head_dim: int, theta: float, scaling, dtype=torch.float32) -> torch.Tensor:
+    inv_freq = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=dtype) / max(head_dim, 1)))
     if scaling is not None and scaling.rope_type == "llama3":
         original = scaling.original_max_position_embeddings
         wavelength = 2 * math.pi / inv_freq
@@ -42,7 +42,7 @@ def rope_inverse_frequencies(head_dim: int, theta: float, scaling) -> torch.Tens
         high_wavelength = original / scaling.high_freq_factor
         scaled = inv_freq / scaling.factor
         smooth = ((original / wavelength - scaling.low_freq_factor) /
-                  (scaling.high_freq_factor - scaling.low_freq_factor)).clamp(0.0, 1.0)
+                  ((scaling.high_freq_factor - scaling.low_freq_factor) or 1.0)).clamp(0.0, 1.0)
         blended = (1 - smooth) * scaled + smooth * inv_freq
         inv_freq = torch.where(wavelength > low_wavelength, scaled, inv_freq)
         inv_freq = torch.where((wavelength <= low_wavelength) & (wavelength >= high_wavelength), blended, inv_freq)
@@ -66,9 +66,9 @@ def yarn_frequencies(dims: int, theta: float, scaling):
 class RotaryEncoding(PositionEncoding):
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
-        if spec.head_dim % 2:
-            raise ValueError(f"rotary encoding needs an even head_dim, got {spec.head_dim}")
         p = dict(spec.params)
+        if spec.head_dim % 2 and "rotated" not in p:
+            raise ValueError(f"rotary encoding needs an even head_dim, got {spec.head_dim}")
         self.rotated = int(p.get("rotated", spec.head_dim))
         self.pairing = p.get("pairing", "halves")
         if self.rotated % 2 or not 0 <= self.rotated <= spec.head_dim or self.pairing not in ("halves", "neighbours"):
@@ -93,16 +93,34 @@ class RotaryEncoding(PositionEncoding):
         fill = half - r // 2
         return first + rest[:fill] + second + rest[fill:]
 
+    def plain_tables(self):
+        """(cos, sin), each float32 [max_positions, rotated / 2], for a kernel that itself pairs entry i with entry
+        i + rotated / 2 and leaves the rest of a head alone. Angles are formed in float64 and rounded once."""
+        if self.pairing != "halves":
+            raise ValueError(f"the pairing {self.pairing!r} has no tables of this form")
+        return self.rt.shared(("rope-plain", self.spec), self._build_plain)
+
+    def _build_plain(self):
+        f, magnitude = self._frequencies()
+        angles = torch.outer(torch.arange(self.max_positions, dtype=torch.float64), f)
+        return tuple((t * magnitude).float().contiguous().to(self.rt.device) for t in (angles.cos(), angles.sin()))
+
+    def _frequencies(self):
+        """float64 frequencies [rotated / 2] and the factor on cos and sin."""
+        r, sc = self.rotated, self.spec.scaling
+        if sc is not None and sc.rope_type == "yarn":
+            return yarn_frequencies(r, self.spec.theta, sc)
+        if sc is not None and sc.rope_type == "llama3":
+            return rope_inverse_frequencies(r, self.spec.theta, sc, torch.float64), 1.0
+        if sc is not None:
+            raise ValueError(f"rope scaling {sc.rope_type!r} is not available for a partial or neighbour-paired rotation")
+        return float(self.spec.theta) ** (-torch.arange(0, r, 2, dtype=torch.float64) / max(r, 1)), 1.0
+
     def _build_general(self):
         """Tables in the kernels' layout [max_positions, head_dim / 2] for a partial rotation, YaRN or both: angles in
         float64, rounded once; pairs that pass unchanged get cos 1 and sin 0."""
-        hd, r, sc = self.spec.head_dim, self.rotated, self.spec.scaling
-        if sc is not None and sc.rope_type == "yarn":
-            f, magnitude = yarn_frequencies(r, self.spec.theta, sc)
-        elif sc is not None:
-            raise ValueError(f"rope scaling {sc.rope_type!r} is not available for a partial or neighbour-paired rotation")
-        else:
-            f, magnitude = float(self.spec.theta) ** (-torch.arange(0, r, 2, dtype=torch.float64) / max(r, 1)), 1.0
+        hd, r = self.spec.head_dim, self.rotated
+        f, magnitude = self._frequencies()
         angles = torch.outer(torch.arange(self.max_positions, dtype=torch.float64), f)
         cos = torch.ones((self.max_positions, hd // 2), dtype=torch.float32)
         sin = torch.zeros((self.max_positions, hd // 2), dtype=torch.float32)

@@ -28,6 +28,11 @@ Another family of the same part, chosen by the spec:
 * param ``router`` ``softmax_groups``: scores are the softmax of z over all experts; a group counts as its largest
   score; the ``top`` largest scores inside the ``keep`` best groups win; the weights are those scores times
   ``route_scale``, not divided by their sum. No ``correction`` tensor.
+* param ``router`` ``sigmoid_scores``: scores are ``sigmoid(z)``; the ``top`` largest win, and the weights are those scores as they
+  are. No ``correction`` tensor.
+* param ``weigh`` ``inputs`` (gated experts only): a token's weight multiplies what the expert is given, not what it gives, so the
+  output is ``sum_k expert_k(w_k h)``. Both of the expert's first products are linear in their input, so the number is applied to
+  their float32 sums, in the epilogue in front of the activation.
 * param ``shared_gate``: the shared expert's output is multiplied by ``sigmoid(W_sg h)``, one number per token (tensor
   ``shared.sg`` [1, hidden]); its row rides in the router's product.
 """
@@ -59,8 +64,11 @@ class RoutedExperts(FeedForward):
         self.router_kind = p.get("router", "softmax_top")
         self.groups, self.keep, self.route_scale = int(p.get("groups", 1)), int(p.get("keep", 1)), float(p.get("route_scale", 1.0))
         self.shared_gate = bool(p.get("shared_gate", False))
-        if self.router_kind not in ("softmax_top", "sigmoid_groups", "softmax_groups"):
-            raise ValueError(f"router {self.router_kind!r} is not known (softmax_top, sigmoid_groups and softmax_groups are)")
+        self.weigh_inputs = p.get("weigh", "outputs") == "inputs"
+        if self.router_kind not in ("softmax_top", "sigmoid_groups", "softmax_groups", "sigmoid_scores"):
+            raise ValueError(f"router {self.router_kind!r} is not known (softmax_top, sigmoid_groups, softmax_groups and sigmoid_scores are)")
+        if self.weigh_inputs and not self.gated:
+            raise ValueError("weights on the experts' inputs go with gated experts")
         if self.router_kind != "softmax_top" and (self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups
                                                      or self.top > self.keep * (self.experts // self.groups)):
             raise ValueError(f"{self.experts} experts in {self.groups} groups of which {self.keep} stay cannot give {self.top} choices")
@@ -154,9 +162,9 @@ class RoutedExperts(FeedForward):
         if self.router_kind == "sigmoid_groups":
             ops.moe_select_sigmoid(logits, self.correction, ctx.seq_of_token[:tokens], ids, weights, self.experts, self.groups, self.keep,
                                    self.route_scale)
-        elif self.router_kind == "softmax_groups":
+        elif self.router_kind in ("softmax_groups", "sigmoid_scores"):
             ops.moe_select_groups(logits, None, ctx.seq_of_token[:tokens], ids, weights, self.experts, self.groups, self.keep,
-                                  self.route_scale, softmax=True, group_max=True, keep_scores=True)
+                                  self.route_scale, softmax=self.router_kind == "softmax_groups", group_max=True, keep_scores=True)
         else:
             ops.moe_select(logits if not self.shared_gate else logits[:, :self.experts].contiguous(), self.bias,
                            ctx.seq_of_token[:tokens], ids, weights)
@@ -164,12 +172,13 @@ class RoutedExperts(FeedForward):
         perm = self.rt.buffer("moe_perm", tokens, top, i32).view(-1)
         rank = self.rt.buffer("moe_rank", tokens, top, i32).view(-1)
         offsets = self.rt.scratch(f"moe_offsets_{self.experts}", self.experts + 1, i32)
-        ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank)
+        row_weight = self.rt.buffer("moe_row_weight", tokens, top, torch.float32).view(-1) if self.weigh_inputs else None
+        ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank, weights if self.weigh_inputs else None, row_weight)
         hidden_rows = self.rt.buffer("moe_hidden", tokens, top * self.ff).view(pairs, self.ff)
         y = self.rt.buffer("moe_y", tokens, top * self.hidden, torch.float32).view(pairs, self.hidden)
         act = (2 if self.clamped else 3) if self.gated else 1
-        if not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act):
-            ops.grouped_gemm(x, perm, self.w_up, offsets, hidden_rows, pairs, act=act, limit=self.limit, alpha=self.alpha)
+        if not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight):
+            ops.grouped_gemm(x, perm, self.w_up, offsets, hidden_rows, pairs, act=act, limit=self.limit, alpha=self.alpha, row_weight=row_weight)
             ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
         shared = None
         if self.shared_ff:
@@ -190,11 +199,11 @@ class RoutedExperts(FeedForward):
             shared = self.rt.buffer("moe_shared_out", tokens, self.hidden)
             ops.linear(mid, self.shared_down, shared)
         out = self.rt.buffer("ffn_out", tokens, self.hidden)
-        ops.moe_combine(y, row_of, weights, shared, out, logits[:, self.experts] if self.shared_gate else None)
+        ops.moe_combine(y, row_of, None if self.weigh_inputs else weights, shared, out, logits[:, self.experts] if self.shared_gate else None)
         return out
 
 
-    def _products_tc(self, x, perm, offsets, hidden_rows, y, tokens, pairs, act) -> bool:
+    def _products_tc(self, x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight) -> bool:
         """Both products of all experts on the tcgen05 kernel, for steps of many rows: the tokens' rows are laid out
         expert by expert first, so that every expert's rows are one block of a matrix. False: nothing was done."""
         if not ops.grouped_tc_wanted(x.dtype, pairs):
@@ -202,7 +211,7 @@ class RoutedExperts(FeedForward):
         rows = self.rt.buffer("moe_rows", tokens, self.top * self.hidden).view(pairs, self.hidden)
         if not ops.gather_rows(x, perm, offsets, self.experts, rows, pairs):
             return False
-        if not ops.grouped_gemm_tc(rows, self.w_up, offsets, hidden_rows, pairs, act, self.limit, self.alpha):
+        if not ops.grouped_gemm_tc(rows, self.w_up, offsets, hidden_rows, pairs, act, self.limit, self.alpha, row_weight):
             return False
         if not ops.grouped_gemm_tc(hidden_rows, self.w_down, offsets, y, pairs, 0):
             ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
