@@ -566,8 +566,32 @@ def compare_configs_dopudra(name: str, layers: int):
     return ours, llama
 
 
+# Layer sizes for `--compare negotar`: layers cycle state space, attention (with value mixing), each with the mixture. Attention of
+# the Llama decoder's head count, grouping and head size; the state space memory has twice the width as inner channels, in heads of
+# 64 with a state of 128 and eight groups; a token uses as many feed-forward weights as in the Llama decoder's.
+NEGOTAR_SIZES = {"w1024": dict(experts=16, top=3, expert_ff=896, heads=32), "w2048": dict(experts=32, top=4, expert_ff=1344, heads=64)}
+
+
+def compare_configs_negotar(name: str, layers: int):
+    """(Negotar config.json, Llama config.json) of one size."""
+    size, own = TUTIZEN_SIZES[name], NEGOTAR_SIZES[name]
+    _tutizen, llama = compare_configs_tutizen(size, layers)
+    attention = {"heads": size["heads"], "kv_heads": size["kv"], "dim": size["dim"], "vdim": size["dim"], "scale": size["dim"] ** -0.5,
+                 "softcap": 50.0, "v_mix": True,
+                 "rot": {"base": 500000.0, "dims": size["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    memory = {"heads": own["heads"], "vdim": 64, "groups": 8, "state": 128, "conv": 4, "norm_groups": 8}
+    mlp = {"kind": "moe", "expert": {"ff": own["expert_ff"]}, "router": {"experts": own["experts"], "top": own["top"]}}
+    entries = [{"type": "attention", "mixer": attention, "mlp": mlp} if i % 2 else {"type": "mamba2", "mixer": memory, "mlp": mlp}
+               for i in range(layers)]
+    ours = {"architecture": "Negotar", "width": size["width"], "vocab": size["vocab"], "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": entries}
+    llama["tie_word_embeddings"] = True         # as Negotar shares its head with the embedding
+    return ours, llama
+
+
 def _compared(design: str, size_name: str, layers: int):
     """The two configurations of ``--compare design`` at one size."""
+    if design == "negotar":
+        return compare_configs_negotar(size_name, layers)
     if design == "dopudra":
         return compare_configs_dopudra(size_name, layers)
     if design == "netusun":
@@ -635,10 +659,11 @@ def _measure_design(config: dict, batch: int, context: int, prompt_len: int, ste
 
 
 def run_compare(args) -> dict:
-    """``--compare nidilix | migelix | tutizen | netusun | dopudra``: prefill and decode throughput of that design at a few layer sizes
+    """``--compare nidilix | migelix | tutizen | netusun | dopudra | negotar``: prefill and decode throughput of that design at a few layer sizes
     beside the Llama decoder at equal size, with the device time per class of kernel; Netusun also beside Tutizen, the design
     whose layers are closest to its own (the same mixture, a norm on a sublayer's output), and Dopudra beside Migelix (attention
-    beside a matrix memory, decayed memories). Not the headline workload."""
+    beside a matrix memory, decayed memories), Negotar beside Tutizen (unit norms on heads, a sigmoid router, a norm on a sublayer's
+    output) and Dopudra (memories that fade). Not the headline workload."""
     layers = args.layers or 6
     sizes = [s for s in args.compare_sizes.split(",") if s]
     result = {"mode": "compare", "design": args.compare, "beside": "llama", "layers": layers, "dtype": "bf16", "data": "synthetic", "sizes": {}}
@@ -647,9 +672,12 @@ def run_compare(args) -> dict:
         result["sizes"][name] = {
             args.compare: _measure_design(ours, args.batch, args.context, 2048, args.steps, args.warmup),
             "llama": _measure_design(llama, args.batch, args.context, 2048, args.steps, args.warmup)}
-        if args.compare == "netusun":
+        if args.compare in ("netusun", "negotar"):
             closest = compare_configs_tutizen(TUTIZEN_SIZES[name], layers)[0]
             result["sizes"][name]["tutizen"] = _measure_design(closest, args.batch, args.context, 2048, args.steps, args.warmup)
+        if args.compare == "negotar":
+            closest = compare_configs_dopudra(name, layers)[0]
+            result["sizes"][name]["dopudra"] = _measure_design(closest, args.batch, args.context, 2048, args.steps, args.warmup)
         if args.compare == "dopudra":
             closest = compare_configs_migelix(MIGELIX_SIZES[name], layers)[0]
             result["sizes"][name]["migelix"] = _measure_design(closest, args.batch, args.context, 2048, args.steps, args.warmup)
@@ -752,7 +780,7 @@ def main(argv=None) -> int:
     p.add_argument("--no-breakdown", action="store_true", help="skip the per-class times of one decode step and the prefill")
     p.add_argument("--profile", choices=["decode", "prefill"], default=None,
                    help="run a few eager steps of one kind for a profiler instead of measuring")
-    p.add_argument("--compare", choices=["nidilix", "migelix", "tutizen", "netusun", "dopudra"], default=None,
+    p.add_argument("--compare", choices=["nidilix", "migelix", "tutizen", "netusun", "dopudra", "negotar"], default=None,
                    help="instead of the headline workload: this design's prefill and decode beside the Llama decoder at equal size")
     p.add_argument("--compare-sizes", default="w1024,w2048", help="comma-separated names of the sizes to compare")
     args = p.parse_args(argv)

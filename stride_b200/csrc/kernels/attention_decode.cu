@@ -240,7 +240,7 @@ paged_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
 #pragma unroll
                 for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) s[nt][e] = tanh_approx(s[nt][e] * cap_in);
+                    for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * cap_in);
             }
             if (slopes != nullptr) {    // a penalty on the key's distance; a row of the tile is a head of the group
 #pragma unroll

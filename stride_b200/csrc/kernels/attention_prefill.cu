@@ -145,7 +145,7 @@ paged_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfl
 #pragma unroll
             for (int nt = 0; nt < kKTile / 8; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[nt][e] = tanh_approx(s[nt][e] * cap_in);
+                for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * cap_in);
         }
         if (slopes != nullptr) {    // a penalty on the key's distance, in the units of the raw scores
             const float slope_raw = slopes[head] * 1.4426950408889634f / scale_log2e;

@@ -338,7 +338,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             for (int i = 0; i < 64; ++i) sv[i] = __uint_as_float(sr[i]);
             if (cap_in > 0.f) {     // capped scores: c tanh(scale s / c); scale_log2e then holds c log2(e)
 #pragma unroll
-                for (int i = 0; i < 64; ++i) sv[i] = tanh_approx(sv[i] * cap_in);
+                for (int i = 0; i < 64; ++i) sv[i] = tanh_quick(sv[i] * cap_in);
             }
             if (slopes != nullptr) {
                 const float d0 = static_cast<float>(k0 - pos_r);
