@@ -179,7 +179,7 @@ class NegotarConfig:
                                 scaling=scaling, params=(("angles", "float64"), ("rotated", int(rot["dims"]))))
         params = [("names", "short"), ("value_dim", m["vdim"]), ("qk_norm", "unit_rotated"), ("norm_eps", self.norm_eps), ("padded_heads", True)]
         if m.get("softcap") is not None:
-            params.append(("softcap", float(m["softcap"])))
+            params += [("softcap", float(m["softcap"])), ("precise_cap", True)]
         if mixing is not None:
             params.append(("value_mix", mixing))
         return MixerSpec(kind="attention", hidden=self.width, num_heads=m["heads"], num_kv_heads=m["kv_heads"], head_dim=m["dim"],

@@ -240,7 +240,12 @@ paged_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __gri
 #pragma unroll
                 for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * cap_in);
+                    for (int e = 0; e < 4; ++e) s[nt][e] = tanh_approx(s[nt][e] * cap_in);
+            } else if (cap_in < 0.f) {      // the same, tanh in 32-bit accuracy
+#pragma unroll
+                for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * -cap_in);
             }
             if (slopes != nullptr) {    // a penalty on the key's distance; a row of the tile is a head of the group
 #pragma unroll
@@ -504,12 +509,12 @@ int launch_decode(const __nv_bfloat16* q, int q_stride, __nv_bfloat16* out, cons
     if (tma)
         stride::launch(paged_decode_split_kernel<HD, true>, grid, dim3(128), smem, stream, *map_k, *map_v, q, q_stride, k_pages, v_pages,
                        block_table, table_width, seq_of_token, positions, part_o, part_ml, tickets, out, nq, nkv, page_size,
-                       (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes,
+                       (softcap != 0.f ? fabsf(softcap) : scale) * 1.4426950408889634f, window, softcap != 0.f ? scale / softcap : 0.f, sinks, slopes,
                        rel, rel_len, split_keys, num_splits, status, gate_col);
     else
         stride::launch(paged_decode_split_kernel<HD, false>, grid, dim3(128), smem, stream, no_map, no_map, q, q_stride, k_pages, v_pages,
                        block_table, table_width, seq_of_token, positions, part_o, part_ml, tickets, out, nq, nkv, page_size,
-                       (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes,
+                       (softcap != 0.f ? fabsf(softcap) : scale) * 1.4426950408889634f, window, softcap != 0.f ? scale / softcap : 0.f, sinks, slopes,
                        rel, rel_len, split_keys, num_splits, status, gate_col);
     return STRIDE_LAUNCH_STATUS();
 }
@@ -616,7 +621,7 @@ int stride_paged_decode_attention_biased(const void* q, int q_stride, void* out,
                                         int nkv, int hd, int page_size, float scale, int window, float softcap, const float* sinks,
                                         const float* slopes, const float* rel, int rel_len, int gate_col, int max_context, int* status, cudaStream_t stream) {
     if (rel && rel_len <= 0) return STRIDE_BAD_ARGUMENT;
-    if (softcap < 0.f || gate_col < -1 || (gate_col >= 0 && gate_col + nq > q_stride)) return STRIDE_BAD_ARGUMENT;
+    if (gate_col < -1 || (gate_col >= 0 && gate_col + nq > q_stride)) return STRIDE_BAD_ARGUMENT;
     if (tokens < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || max_context <= 0)
         return STRIDE_BAD_ARGUMENT;
     if (nq % nkv) return STRIDE_BAD_ARGUMENT;

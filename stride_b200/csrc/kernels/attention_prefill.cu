@@ -145,7 +145,12 @@ paged_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bfl
 #pragma unroll
             for (int nt = 0; nt < kKTile / 8; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * cap_in);
+                for (int e = 0; e < 4; ++e) s[nt][e] = tanh_approx(s[nt][e] * cap_in);
+        } else if (cap_in < 0.f) {      // the same, tanh in 32-bit accuracy
+#pragma unroll
+            for (int nt = 0; nt < kKTile / 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = tanh_quick(s[nt][e] * -cap_in);
         }
         if (slopes != nullptr) {    // a penalty on the key's distance, in the units of the raw scores
             const float slope_raw = slopes[head] * 1.4426950408889634f / scale_log2e;
@@ -271,8 +276,8 @@ int launch_prefill(const __nv_bfloat16* q, int q_stride, __nv_bfloat16* out, con
     dim3 grid(max_tiles, nq);
     stride::launch(paged_prefill_kernel<HD>, dim3(grid), dim3(128), smem, stream, q, q_stride, out, k_pages, v_pages, block_table, table_width, q_start,
                                                           q_len, ctx_len, num_seqs, nq, nkv, page_size,
-                                                          (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window,
-                                                          softcap > 0.f ? scale / softcap : 0.f, sinks, slopes, rel, rel_len);
+                                                          (softcap != 0.f ? fabsf(softcap) : scale) * 1.4426950408889634f, window,
+                                                          softcap != 0.f ? scale / softcap : 0.f, sinks, slopes, rel, rel_len);
     return STRIDE_LAUNCH_STATUS();
 }
 
@@ -283,7 +288,7 @@ using namespace stride;
 // Attention for the first `num_seqs` requests of the step, which own the first
 // `tokens` rows of the flat batch. q: [tokens, q_stride]; out: [tokens, nq * hd].
 // Returns -2 for sizes it does not run (head sizes other than 64 and 128); the
-// caller then uses the generic kernel. softcap c > 0 caps the scaled scores at c tanh(s / c) (with the hardware's tanh);
+// caller then uses the generic kernel. softcap c > 0 caps the scaled scores at c tanh(s / c) (with the hardware's tanh; softcap -c: the same with a tanh of 32-bit accuracy);
 // sinks (float32 [nq] or null) adds exp(sink) of the head to the softmax's denominator; slopes (float32 [nq] or null)
 // takes slope_h times the key's distance off every score of head h; rel (float32 [nq, rel_len] or null) adds
 // rel[h, min(distance, rel_len - 1)] to every score of head h.
@@ -292,7 +297,7 @@ extern "C" int stride_paged_prefill_attention(const void* q, int q_stride, void*
                                               const int32_t* q_len, const int32_t* ctx_len, int num_seqs, int tokens, int nq,
                                               int nkv, int hd, int page_size, float scale, int window, float softcap,
                                               const float* sinks, const float* slopes, const float* rel, int rel_len, cudaStream_t stream) {
-    if (tokens < 0 || num_seqs < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || softcap < 0.f ||
+    if (tokens < 0 || num_seqs < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || table_width <= 0 || window < 0 ||
         (rel && rel_len <= 0))
         return STRIDE_BAD_ARGUMENT;
     if (nq % nkv) return STRIDE_BAD_ARGUMENT;

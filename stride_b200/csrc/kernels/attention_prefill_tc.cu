@@ -338,7 +338,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             for (int i = 0; i < 64; ++i) sv[i] = __uint_as_float(sr[i]);
             if (cap_in > 0.f) {     // capped scores: c tanh(scale s / c); scale_log2e then holds c log2(e)
 #pragma unroll
-                for (int i = 0; i < 64; ++i) sv[i] = tanh_quick(sv[i] * cap_in);
+                for (int i = 0; i < 64; ++i) sv[i] = tanh_approx(sv[i] * cap_in);
+            } else if (!REL && cap_in < 0.f) {      // the same, tanh in 32-bit accuracy (not beside a table of distances)
+#pragma unroll
+                for (int i = 0; i < 64; ++i) sv[i] = tanh_quick(sv[i] * -cap_in);
             }
             if (slopes != nullptr) {
                 const float d0 = static_cast<float>(k0 - pos_r);
@@ -495,7 +498,7 @@ int launch_attn(const CUtensorMap* map_q, const CUtensorMap* map_k, const CUtens
                                        : (tma ? attn_prefill_tc_kernel<HD, HEADS, true, false> : attn_prefill_tc_kernel<HD, HEADS, false, false>);
     stride::launch(kernel, grid, block, smem, stream, *map_q, tma ? *map_k : *map_q, tma ? *map_v : *map_q, k_pages, v_pages, out,
                    block_table, table_width, q_start, q_len, ctx_len, num_seqs, nq, nkv, page_shift,
-                   (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, softcap > 0.f ? scale / softcap : 0.f, sinks, slopes, rel,
+                   (softcap != 0.f ? fabsf(softcap) : scale) * 1.4426950408889634f, window, softcap != 0.f ? scale / softcap : 0.f, sinks, slopes, rel,
                    rel_len, status);
     return STRIDE_LAUNCH_STATUS();
 }
@@ -527,7 +530,8 @@ static bool kv_tma() {
 // the flat batch. q: [tokens, q_stride] bf16 (head h at columns h*hd); out: [tokens, nq*hd];
 // pages: [num_pages, nkv, page_size, hd]. Returns -2 for what it does not take (head sizes other
 // than 64 and 128, page sizes that are no power of two from 4 to 64, unaligned strides); the caller
-// then uses the mma.sync kernel. softcap c > 0 caps the scaled scores at c tanh(s / c) (with the hardware's tanh); sinks
+// then uses the mma.sync kernel. softcap c > 0 caps the scaled scores at c tanh(s / c) (with the hardware's tanh; softcap -c: the
+// same with a tanh of 32-bit accuracy, without a table of distances only); sinks
 // (float32 [nq] or null) adds exp(sink) of the head to the softmax's denominator; slopes (float32 [nq] or null) takes
 // slope_h times the key's distance off every score of head h; rel (float32 [nq, rel_len] or null) adds rel[h, min(distance,
 // rel_len - 1)] to every score of head h.
@@ -539,9 +543,10 @@ extern "C" int stride_paged_prefill_attention_tc(const void* q, int q_stride, vo
                                                  int rel_len, int* status,
                                                  cudaStream_t stream) {
     if (tokens < 0 || num_seqs < 0 || nq <= 0 || nkv <= 0 || page_size <= 0 || table_width <= 0 || window < 0 || num_pages <= 0 ||
-        softcap < 0.f || (rel && rel_len <= 0))
+        (rel && rel_len <= 0))
         return STRIDE_BAD_ARGUMENT;
     if (nq % nkv || status == nullptr) return STRIDE_BAD_ARGUMENT;
+    if (rel && softcap < 0.f) return STRIDE_UNSUPPORTED;
     if ((hd != 64 && hd != 128) || page_size > tc::kKeys || page_size < 4 || q_stride % 8 || nq > 65535) return STRIDE_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(k_pages) |
          reinterpret_cast<uintptr_t>(v_pages)) % 16)

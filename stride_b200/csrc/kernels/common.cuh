@@ -130,8 +130,15 @@ __device__ __forceinline__ float from_f32<float>(float x) { return x; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float x) { return __float2bfloat16_rn(x); }
 
-// tanh x = 1 - 2 / (e^2x + 1) by the hardware's exponential and reciprocal: an absolute error of a few 2^-24, where the
-// hardware's own tanh leaves 2^-11 (a capped score is a multiple of it: what counts is the absolute error of the exponent).
+// The hardware's tanh (relative error about 2^-11): for scores that are rounded to bfloat16 anyway.
+__device__ __forceinline__ float tanh_approx(float x) {
+    float y;
+    asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// tanh x = 1 - 2 / (e^2x + 1) by the hardware's exponential and reciprocal: an absolute error of a few 2^-24 (a capped score is a
+// multiple of it: what counts is the absolute error), for designs whose scores are 32-bit throughout.
 __device__ __forceinline__ float tanh_quick(float x) {
     float e, r;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));

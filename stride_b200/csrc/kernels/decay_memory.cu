@@ -80,9 +80,6 @@ chunk_decay_kernel(const ChunkArgs p) {
     }
 }
 
-// z / (1 + e^-z) by the hardware's exponential and quotient: a few units in the last place of float32.
-__device__ __forceinline__ float silu_quick(float z) { return __fdividef(z, 1.f + __expf(-z)); }
-
 // Eight neighbouring values of a row of the projection.
 __device__ __forceinline__ void unpack8(const uint4& r, float* v) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);

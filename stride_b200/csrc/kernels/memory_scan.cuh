@@ -17,6 +17,8 @@ enum MemoryRule {
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// The same by the hardware's exponential and quotient: a few units in the last place of float32.
+__device__ __forceinline__ float silu_quick(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
 __device__ __forceinline__ float load_any(const void* p, size_t i, int is_bf16) {
     return is_bf16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p)[i]) : static_cast<const float*>(p)[i];

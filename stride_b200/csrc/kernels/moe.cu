@@ -12,6 +12,7 @@
 //   moe_plan      one CTA counts the rows of every expert, lays the (token, choice) pairs out expert by expert and
 //                 writes where each pair went: `offsets` [experts + 1], `perm_token` [rows] and `row_of` [tokens, top], and
 //                 on request every row's weight;
+//   moe_route_plan  for a few bfloat16 tokens: the router's product, the choice by the rule above and the plan in one launch;
 //   grouped_gemm  C[p, :] = act(A[src(p), :] W[e(p)]^T) for the rows p of every expert e, the tiles of all experts in
 //                 one launch (the CTA finds its expert from `offsets` on the device, so nothing goes back to the
 //                 host and the step can be replayed from a graph); float32 FMA with a fixed k order for float32
@@ -146,34 +147,18 @@ moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ bi
     }
 }
 
-// logits: [tokens, ld] float32 (the first `experts` columns of a row). One warp per token.
-__global__ void __launch_bounds__(128)
-moe_select_sigmoid_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction,
-                          const int32_t* __restrict__ seq_of_token, int32_t* __restrict__ ids, float* __restrict__ weights, int tokens,
-                          int experts, int top, int groups, int keep, float route_scale, int rule) {
-    pdl_trigger();
-    pdl_wait();
-    __shared__ float choice_s[4][kMaxExperts];
-    __shared__ float group_s[4][kMaxExperts];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t = blockIdx.x * 4 + warp;
-    if (t >= tokens) return;
-    if (seq_of_token && seq_of_token[t] < 0) {
-        for (int k = lane; k < top; k += 32) {
-            ids[static_cast<size_t>(t) * top + k] = -1;
-            weights[static_cast<size_t>(t) * top + k] = 0.f;
-        }
-        return;
-    }
-    float* choice = choice_s[warp];
-    float* gscore = group_s[warp];
+// One warp's choice for a token by the group router's rule: z_row its logits, `choice` and `gscore` shared memory of kMaxExperts
+// floats each, ids and weights the token's `top` places.
+__device__ __forceinline__ void choose_by_rule(const float* z_row, const float* __restrict__ correction, float* choice, float* gscore,
+                                               int32_t* __restrict__ ids, float* __restrict__ weights, int experts, int top, int groups, int keep,
+                                               float route_scale, int rule, int lane) {
     float score[kMaxExperts / 32];       // lane holds experts lane, lane + 32, ...
     if (rule & kRuleSoftmax) {           // softmax over all experts: largest logit, exponentials, their sum in a fixed order
         float top_z = -INFINITY;
 #pragma unroll
         for (int i = 0; i < kMaxExperts / 32; ++i) {
             const int e = i * 32 + lane;
-            score[i] = e < experts ? logits[static_cast<size_t>(t) * ld + e] : -INFINITY;
+            score[i] = e < experts ? z_row[e] : -INFINITY;
             top_z = fmaxf(top_z, score[i]);
         }
 #pragma unroll
@@ -198,7 +183,7 @@ moe_select_sigmoid_kernel(const float* __restrict__ logits, int ld, const float*
             const int e = i * 32 + lane;
             score[i] = 0.f;
             if (e < experts) {
-                score[i] = 1.f / (1.f + expf(-logits[static_cast<size_t>(t) * ld + e]));
+                score[i] = 1.f / (1.f + expf(-z_row[e]));
                 choice[e] = score[i] + (correction ? correction[e] : 0.f);
             }
         }
@@ -274,25 +259,51 @@ moe_select_sigmoid_kernel(const float* __restrict__ logits, int ld, const float*
         if (lane == k) { mine = best_score; mine_id = best_e == 0x7fffffff ? -1 : best_e; }
     }
     if (lane < top) {
-        ids[static_cast<size_t>(t) * top + lane] = mine_id;
-        weights[static_cast<size_t>(t) * top + lane] = (rule & kRuleKeepScores) ? mine * route_scale : mine / (denom + 1e-20f) * route_scale;
+        ids[lane] = mine_id;
+        weights[lane] = (rule & kRuleKeepScores) ? mine * route_scale : mine / (denom + 1e-20f) * route_scale;
     }
 }
 
-// ids: [tokens, top] (-1: a padded token). rank_tmp: [tokens * top] scratch.
-__global__ void __launch_bounds__(256)
-moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
-                int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, const float* __restrict__ weights,
-                float* __restrict__ row_weight, int top) {
+// logits: [tokens, ld] float32 (the first `experts` columns of a row). One warp per token.
+__global__ void __launch_bounds__(128)
+moe_select_sigmoid_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction,
+                          const int32_t* __restrict__ seq_of_token, int32_t* __restrict__ ids, float* __restrict__ weights, int tokens,
+                          int experts, int top, int groups, int keep, float route_scale, int rule) {
     pdl_trigger();
     pdl_wait();
+    __shared__ float choice_s[4][kMaxExperts];
+    __shared__ float group_s[4][kMaxExperts];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * 4 + warp;
+    if (t >= tokens) return;
+    ids += static_cast<size_t>(t) * top;
+    weights += static_cast<size_t>(t) * top;
+    if (seq_of_token && seq_of_token[t] < 0) {
+        for (int k = lane; k < top; k += 32) {
+            ids[k] = -1;
+            weights[k] = 0.f;
+        }
+        return;
+    }
+    choose_by_rule(logits + static_cast<size_t>(t) * ld, correction, choice_s[warp], group_s[warp], ids, weights, experts, top, groups, keep,
+                   route_scale, rule, lane);
+}
+
+// ids: [tokens, top] (-1: a padded token). rank_tmp: [tokens * top] scratch.
+__device__ __forceinline__ void plan_rows(const int32_t* ids, int pairs, int experts, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
+                                          int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, const float* weights,
+                                          float* __restrict__ row_weight, int top) {
     __shared__ int counts[kMaxExperts];
     __shared__ int starts[kMaxExperts + 1];
     for (int e = threadIdx.x; e < experts; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-        const int e = ids[i];
-        if (e >= 0 && e < experts) rank_tmp[i] = atomicAdd(&counts[e], 1);
+    for (int i0 = threadIdx.x; i0 < pairs; i0 += 4 * blockDim.x) {      // four pairs a thread are asked for together
+        int e[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) e[u] = i0 + u * blockDim.x < pairs ? __ldcg(ids + i0 + u * blockDim.x) : -1;
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+            if (e[u] >= 0 && e[u] < experts) rank_tmp[i0 + u * blockDim.x] = atomicAdd(&counts[e[u]], 1);
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -305,17 +316,104 @@ moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t
     }
     __syncthreads();
     for (int e = threadIdx.x; e <= experts; e += blockDim.x) offsets[e] = starts[e];
-    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-        const int e = ids[i];
-        if (e >= 0 && e < experts) {
-            const int row = starts[e] + rank_tmp[i];
+    for (int i0 = threadIdx.x; i0 < pairs; i0 += 4 * blockDim.x) {
+        int e[4], rank[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int i = i0 + u * blockDim.x;
+            e[u] = i < pairs ? __ldcg(ids + i) : -1;
+            rank[u] = e[u] >= 0 && e[u] < experts ? rank_tmp[i] : -1;       // written by this thread
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int i = i0 + u * blockDim.x;
+            if (i >= pairs) continue;
+            const int row = rank[u] >= 0 ? starts[e[u]] + rank[u] : -1;
             row_of[i] = row;
+            if (row < 0) continue;
             perm_token[row] = i / top;
-            if (row_weight) row_weight[row] = weights[i];
-        } else {
-            row_of[i] = -1;
+            if (row_weight) row_weight[row] = __ldcg(weights + i);
         }
     }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
+                int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, const float* __restrict__ weights,
+                float* __restrict__ row_weight, int top) {
+    pdl_trigger();
+    pdl_wait();
+    plan_rows(ids, pairs, experts, offsets, perm_token, row_of, rank_tmp, weights, row_weight, top);
+}
+
+// Router product, choice and plan of a step of a few tokens in one launch: a CTA a token, a warp four experts at a time, every
+// logit a float32 sum in an order that depends on `hidden` only; the CTA that finishes last (a ticket, left at zero) lays out the rows.
+// rows: of w (the experts, then any more whose logits are only written, such as a shared expert's gate).
+constexpr int kRouteThreads = 256, kRouteMaxRows = kMaxExperts + 32;
+__global__ void __launch_bounds__(kRouteThreads)
+moe_route_plan_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int rows, int hidden, float* __restrict__ logits,
+                      const float* __restrict__ correction, const int32_t* __restrict__ seq_of_token, int32_t* ids, float* weights, int experts, int top,
+                      int groups, int keep, float route_scale, int rule, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
+                      int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, float* __restrict__ row_weight, unsigned* ticket) {
+    __shared__ float z[kRouteMaxRows];
+    __shared__ float choice[kMaxExperts], gscore[kMaxExperts];
+    __shared__ bool last;
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const __nv_bfloat16* row = x + static_cast<size_t>(t) * hidden;
+    for (int e0 = warp * 4; e0 < rows; e0 += kRouteThreads / 32 * 4) {
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+        for (int k = lane * 8; k < hidden; k += 256) {
+            const uint4 a = *reinterpret_cast<const uint4*>(row + k);
+            uint4 b[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                b[u] = e0 + u < rows ? __ldg(reinterpret_cast<const uint4*>(w + static_cast<size_t>(e0 + u) * hidden + k)) : make_uint4(0, 0, 0, 0);
+            const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&a);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 fa = __bfloat1622float2(pa[i]);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const float2 fb = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&b[u])[i]);
+                    acc[u] = fmaf(fa.x, fb.x, acc[u]);
+                    acc[u] = fmaf(fa.y, fb.y, acc[u]);
+                }
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            acc[u] = warp_sum(acc[u]);
+            if (lane == 0 && e0 + u < rows) {
+                z[e0 + u] = acc[u];
+                logits[static_cast<size_t>(t) * rows + e0 + u] = acc[u];
+            }
+        }
+    }
+    __syncthreads();
+    if (warp == 0) {
+        int32_t* my_ids = ids + static_cast<size_t>(t) * top;
+        float* my_weights = weights + static_cast<size_t>(t) * top;
+        if (seq_of_token && seq_of_token[t] < 0) {
+            for (int k = lane; k < top; k += 32) {
+                my_ids[k] = -1;
+                my_weights[k] = 0.f;
+            }
+        } else {
+            choose_by_rule(z, correction, choice, gscore, my_ids, my_weights, experts, top, groups, keep, route_scale, rule, lane);
+        }
+        __threadfence();
+        __syncwarp();
+        if (lane == 0) {
+            last = atomicAdd(ticket, 1u) + 1 == gridDim.x;
+            if (last) *ticket = 0;
+            __threadfence();
+        }
+    }
+    __syncthreads();
+    if (last) plan_rows(ids, static_cast<int>(gridDim.x) * top, experts, offsets, perm_token, row_of, rank_tmp, weights, row_weight, top);
 }
 
 __device__ __forceinline__ float clamped_gated(float g, float u, float limit, float alpha) {
@@ -583,8 +681,25 @@ int stride_moe_plan(const int32_t* ids, int tokens, int top, int experts, int32_
                     int32_t* rank_tmp, const float* weights, float* row_weight, cudaStream_t stream) {
     if (tokens < 0 || top <= 0 || experts <= 0 || (row_weight && !weights)) return STRIDE_BAD_ARGUMENT;
     if (experts > kMaxExperts) return STRIDE_UNSUPPORTED;
-    stride::launch(moe_plan_kernel, dim3(1), dim3(256), 0, stream, ids, tokens * top, experts, offsets, perm_token, row_of, rank_tmp, weights,
+    stride::launch(moe_plan_kernel, dim3(1), dim3(static_cast<long long>(tokens) * top > 1024 ? 1024 : 256), 0, stream, ids, tokens * top, experts, offsets, perm_token, row_of, rank_tmp, weights,
                    row_weight, top);
+    return STRIDE_LAUNCH_STATUS();
+}
+
+// ticket: one word, zero between launches. Returns -2 for what it does not take (hidden no multiple of 8, unaligned operands).
+int stride_moe_route_plan(const void* x, const void* w, int rows, int hidden, float* logits, const float* correction, const int32_t* seq_of_token,
+                          int32_t* ids, float* weights, int tokens, int experts, int top, int groups, int keep, float route_scale, int rule,
+                          int32_t* offsets, int32_t* perm_token, int32_t* row_of, int32_t* rank_tmp, float* row_weight, unsigned* ticket,
+                          cudaStream_t stream) {
+    if (tokens < 0 || hidden <= 0 || experts <= 0 || rows < experts || top <= 0 || top > experts || groups <= 0 || keep <= 0 || keep > groups ||
+        experts % groups || top > keep * (experts / groups) || rule < 0 || rule > 7 || !ticket)
+        return STRIDE_BAD_ARGUMENT;
+    if (experts > kMaxExperts || top > kMaxTop || rows > kRouteMaxRows || hidden % 8 || (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) % 16)
+        return STRIDE_UNSUPPORTED;
+    if (tokens == 0) return 0;
+    stride::launch(moe_route_plan_kernel, dim3(tokens), dim3(kRouteThreads), 0, stream, static_cast<const __nv_bfloat16*>(x),
+                   static_cast<const __nv_bfloat16*>(w), rows, hidden, logits, correction, seq_of_token, ids, weights, experts, top, groups, keep,
+                   route_scale, rule, offsets, perm_token, row_of, rank_tmp, row_weight, ticket);
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -92,10 +92,31 @@ __device__ __forceinline__ void store_pack(T* p, const float* v) {
     }
 }
 
+// A pack as it lies in memory, to be widened when it is used.
+template <typename T, int V>
+struct HeldPack {
+    float v[V];
+    __device__ __forceinline__ void load(const T* p) { load_pack<T, V>(p, v); }
+    __device__ __forceinline__ void widen(float* out) const {
+#pragma unroll
+        for (int e = 0; e < V; ++e) out[e] = v[e];
+    }
+};
+template <>
+struct HeldPack<__nv_bfloat16, 8> {
+    uint4 raw;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { raw = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void widen(float* out) const { load_pack<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(&raw), out); }
+};
+
+// SiLU for an output of type T: what is rounded to 16 bits takes the quick form.
+template <typename T>
+__device__ __forceinline__ float silu_for(float z) { return sizeof(T) == 2 ? silu_quick(z) : silu_f(z); }
+
 // A thread: V neighbouring channels of `run` consecutive rows. TAPS > 0: that many taps, the last inputs kept in registers from
-// row to row; TAPS 0: any number, every input read again.
+// row to row, four rows asked for at a time; TAPS 0: any number, every input read again.
 template <typename TI, typename TO, int V, int TAPS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 5)
 ssm_conv_kernel(const SsmConvArgs p, int run) {
     pdl_trigger();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
@@ -125,46 +146,60 @@ ssm_conv_kernel(const SsmConvArgs p, int run) {
     float hist[HELD][V];            // inputs of tokens t - TAPS + 1 .. t (the last slot: t)
     int held_seq = -1;
     const int t0 = blockIdx.y * run, t1 = min(t0 + run, p.tokens);
-    for (int t = t0; t < t1; ++t) {
-        const int seq = p.seq_of_token[t];
-        if (seq < 0) {
-            held_seq = -1;
-            continue;
+    constexpr int ROWS = 4;
+    for (int tb = t0; tb < t1; tb += ROWS) {
+        HeldPack<TI, V> fresh[ROWS];
+        int seqs[ROWS];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            seqs[r] = -1;
+            if (tb + r < t1) {
+                seqs[r] = p.seq_of_token[tb + r];
+                fresh[r].load(u + static_cast<size_t>(tb + r) * p.ld);
+            }
         }
-        float y[V];
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = bias[e];
-        if (TAPS > 0) {
-            if (seq == held_seq) {
+        for (int r = 0; r < ROWS; ++r) {
+            const int t = tb + r, seq = seqs[r];
+            if (seq < 0) {
+                held_seq = -1;
+                continue;
+            }
+            float y[V];
 #pragma unroll
-                for (int j = 0; j + 1 < HELD; ++j)
+            for (int e = 0; e < V; ++e) y[e] = bias[e];
+            if (TAPS > 0) {
+                if (seq == held_seq) {
 #pragma unroll
-                    for (int e = 0; e < V; ++e) hist[j][e] = hist[j + 1][e];
+                    for (int j = 0; j + 1 < HELD; ++j)
+#pragma unroll
+                        for (int e = 0; e < V; ++e) hist[j][e] = hist[j + 1][e];
+                } else {
+                    const int start = p.q_start[seq], slot = p.state_slot[seq], at = p.positions[t];
+#pragma unroll
+                    for (int j = 0; j + 1 < HELD; ++j) earlier(start, t - start, at, slot, HELD - 1 - j, hist[j]);
+                    held_seq = seq;
+                }
+                fresh[r].widen(hist[HELD - 1]);
+#pragma unroll
+                for (int j = 0; j < HELD; ++j)
+#pragma unroll
+                    for (int e = 0; e < V; ++e) y[e] = fmaf(w[j][e], hist[j][e], y[e]);
             } else {
                 const int start = p.q_start[seq], slot = p.state_slot[seq], at = p.positions[t];
+                for (int j = 0; j < taps; ++j) {
+                    float v[V], f[V];
+                    load_pack<float, V>(p.w + static_cast<size_t>(j) * p.channels + c, f);
+                    if (j + 1 < taps) earlier(start, t - start, at, slot, taps - 1 - j, v);
+                    else fresh[r].widen(v);
 #pragma unroll
-                for (int j = 0; j + 1 < HELD; ++j) earlier(start, t - start, at, slot, HELD - 1 - j, hist[j]);
-                held_seq = seq;
+                    for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], v[e], y[e]);
+                }
             }
-            load_pack<TI, V>(u + static_cast<size_t>(t) * p.ld, hist[HELD - 1]);
 #pragma unroll
-            for (int j = 0; j < HELD; ++j)
-#pragma unroll
-                for (int e = 0; e < V; ++e) y[e] = fmaf(w[j][e], hist[j][e], y[e]);
-        } else {
-            const int start = p.q_start[seq], slot = p.state_slot[seq], at = p.positions[t];
-            for (int j = 0; j < taps; ++j) {
-                float v[V], f[V];
-                load_pack<float, V>(p.w + static_cast<size_t>(j) * p.channels + c, f);
-                if (j + 1 < taps) earlier(start, t - start, at, slot, taps - 1 - j, v);
-                else load_pack<TI, V>(u + static_cast<size_t>(t) * p.ld, v);
-#pragma unroll
-                for (int e = 0; e < V; ++e) y[e] = fmaf(f[e], v[e], y[e]);
-            }
+            for (int e = 0; e < V; ++e) y[e] = silu_for<TO>(y[e]);
+            store_pack<TO, V>(out + static_cast<size_t>(t) * p.ld_out, y);
         }
-#pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = silu_f(y[e]);
-        store_pack<TO, V>(out + static_cast<size_t>(t) * p.ld_out, y);
     }
 }
 
@@ -255,13 +290,23 @@ ssm_step_kernel(const SsmStepArgs p) {
         }
         float v = 0.f;
         if (c >= 0) {
-            const float now = load_any(p.u, t * p.ld + c, p.u_bf16);
+            const float now = load_any(p.u, t * p.ld + c, p.u_bf16), last = p.w[static_cast<size_t>(p.taps - 1) * C + c];
             v = p.b[c];
-            for (int j = 0; j + 1 < p.taps; ++j) {
-                const int back = p.taps - 1 - j;
-                if (at >= back) v = fmaf(p.w[static_cast<size_t>(j) * C + c], ring[static_cast<size_t>((at - back) % p.taps) * C + c], v);
+            for (int j0 = 0; j0 + 1 < p.taps; j0 += 3) {        // three earlier inputs are asked for together
+                float was[3], f[3];
+#pragma unroll
+                for (int e = 0; e < 3; ++e) {
+                    const int back = p.taps - 1 - j0 - e;
+                    was[e] = f[e] = 0.f;
+                    if (back > 0 && at >= back) {
+                        was[e] = ring[static_cast<size_t>((at - back) % p.taps) * C + c];
+                        f[e] = p.w[static_cast<size_t>(j0 + e) * C + c];
+                    }
+                }
+#pragma unroll
+                for (int e = 0; e < 3; ++e) v = fmaf(f[e], was[e], v);
             }
-            v = silu_f(fmaf(p.w[static_cast<size_t>(p.taps - 1) * C + c], now, v));
+            v = silu_f(fmaf(last, now, v));
             // one writer a channel: x the CTA whose columns they are, B and C the first CTA of the group
             if (p.taps > 1 && (i < COLS || (blockIdx.x == 0 && h == g * (p.H / p.G)))) ring[static_cast<size_t>(at % p.taps) * C + c] = now;
         }
@@ -372,6 +417,18 @@ __device__ __forceinline__ void stage_bf16(__nv_bfloat16* dst, const __nv_bfloat
     }
 }
 
+// The same by asynchronous copies where rows allow them (cp_async_wait and a barrier before the tile is read).
+template <int ROWS, int COLS, int LDS>
+__device__ __forceinline__ void stage_async(__nv_bfloat16* dst, const __nv_bfloat16* src, int ld, int nt, int width, bool vec) {
+    if (!vec) return stage_bf16<ROWS, COLS, LDS>(dst, src, ld, nt, width, false);
+#pragma unroll
+    for (int n = 0; n < ROWS * COLS / 8 / kSsmThreads; ++n) {
+        const int idx = n * kSsmThreads + threadIdx.x, r = idx / (COLS / 8), c = (idx % (COLS / 8)) * 8;
+        if (r < nt && c < width) cp_async_16(dst + r * LDS + c, src + static_cast<size_t>(r) * ld + c);
+        else *reinterpret_cast<uint4*>(dst + r * LDS + c) = make_uint4(0, 0, 0, 0);
+    }
+}
+
 // v as the sum of two bfloat16 numbers.
 __device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
     hi = __float2bfloat16_rn(v);
@@ -412,20 +469,24 @@ ssm_chunk_sum_kernel(const SsmChunkArgs p) {
     pdl_wait();
     const int N = p.N, P = p.P, g = h / (p.H / p.G);
     const size_t row0 = static_cast<size_t>(p.q_start[seq] + first);
-    stage_bf16<kSsmChunk, NP, LDN>(Bs, p.B + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
-    chunk_decays(p, h, row0, nt, s_d, s_c);
-    __syncthreads();
-    const float end = s_c[nt - 1];
     const __nv_bfloat16* x = p.x + row0 * p.ld + h * P + col0;
     const int width = min(P - col0, kSsmCols);
+    // everything the CTA reads is asked for before anything is waited for
+    constexpr int PACKS = kSsmChunk * kSsmCols / 8 / kSsmThreads;
+    uint4 rx[PACKS];
     if (p.vec) {
-        constexpr int PACKS = kSsmChunk * kSsmCols / 8 / kSsmThreads;
-        uint4 rx[PACKS];
 #pragma unroll
         for (int n = 0; n < PACKS; ++n) {
             const int idx = n * kSsmThreads + threadIdx.x, j = idx / (kSsmCols / 8), c = (idx % (kSsmCols / 8)) * 8;
             rx[n] = j < nt && c < width ? *reinterpret_cast<const uint4*>(x + static_cast<size_t>(j) * p.ld + c) : make_uint4(0, 0, 0, 0);
         }
+    }
+    stage_async<kSsmChunk, NP, LDN>(Bs, p.B + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
+    cp_async_commit();
+    chunk_decays(p, h, row0, nt, s_d, s_c);
+    __syncthreads();
+    const float end = s_c[nt - 1];
+    if (p.vec) {
 #pragma unroll
         for (int n = 0; n < PACKS; ++n) {
             const int idx = n * kSsmThreads + threadIdx.x, j = idx / (kSsmCols / 8), c = (idx % (kSsmCols / 8)) * 8;
@@ -449,6 +510,7 @@ ssm_chunk_sum_kernel(const SsmChunkArgs p) {
             split_bf16(v, xh[j * kLdX + c], xl[j * kLdX + c]);
         }
     }
+    cp_async_wait<0>();
     __syncthreads();
     if (blockIdx.x == 0 && threadIdx.x == 0) p.piece_p[static_cast<size_t>(z) * p.H + h] = expf(end);
     // warps over row tiles of 16 first, over columns with what is left
@@ -568,19 +630,43 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
     const int N = p.N, P = p.P, g = h / (p.H / p.G);
     const size_t row0 = static_cast<size_t>(p.q_start[seq] + first);
     const int width = min(P - col0, kSsmCols);
-    stage_bf16<kSsmChunk, NP, LDN>(BCs, p.C + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
-    stage_bf16<kSsmChunk, kSsmCols, kLdX>(xs, p.x + row0 * p.ld + h * P + col0, p.ld, nt, width, p.vec);
+    // everything the CTA reads is asked for before anything is waited for: C and x go to shared memory by asynchronous copies, S
+    // (of up to 128 rows) and B, whose place C holds at first, to registers
+    stage_async<kSsmChunk, NP, LDN>(BCs, p.C + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
+    stage_async<kSsmChunk, kSsmCols, kLdX>(xs, p.x + row0 * p.ld + h * P + col0, p.ld, nt, width, p.vec);
+    cp_async_commit();
+    constexpr bool HELD = NP <= 128;
+    constexpr int B_PACKS = HELD ? kSsmChunk * NP / 8 / kSsmThreads : 1;
+    const __nv_bfloat16* B = p.B + row0 * p.ld + g * N;
+    uint4 rb[B_PACKS];
+    if (HELD && p.vec) {
+#pragma unroll
+        for (int n = 0; n < B_PACKS; ++n) {
+            const int idx = n * kSsmThreads + threadIdx.x, r = idx / (NP / 8), c = (idx % (NP / 8)) * 8;
+            rb[n] = r < nt && c < N ? *reinterpret_cast<const uint4*>(B + static_cast<size_t>(r) * p.ld + c) : make_uint4(0, 0, 0, 0);
+        }
+    }
     const float* S = p.piece_s + (static_cast<size_t>(z) * p.H + h) * N * P + col0;
     if (P % 4 == 0) {
-#pragma unroll 4
-        for (int idx = threadIdx.x; idx < NP * kSsmCols / 4; idx += kSsmThreads) {
-            const int r = idx / (kSsmCols / 4), c = (idx % (kSsmCols / 4)) * 4;
-            const float4 v = r < N && c < width ? *reinterpret_cast<const float4*>(S + static_cast<size_t>(r) * P + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            uint2 hi, lo;
-            split_pair(v.x, v.y, hi.x, lo.x);
-            split_pair(v.z, v.w, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(Sh + r * kLdX + c) = hi;
-            *reinterpret_cast<uint2*>(Sl + r * kLdX + c) = lo;
+        constexpr int S_PACKS = NP * kSsmCols / 4 / kSsmThreads;        // 16 bytes each
+        constexpr int TURN = S_PACKS < 8 ? S_PACKS : 8;
+#pragma unroll
+        for (int n0 = 0; n0 < S_PACKS; n0 += TURN) {
+            float4 rs[TURN];
+#pragma unroll
+            for (int n = 0; n < TURN; ++n) {
+                const int idx = (n0 + n) * kSsmThreads + threadIdx.x, r = idx / (kSsmCols / 4), c = (idx % (kSsmCols / 4)) * 4;
+                rs[n] = r < N && c < width ? *reinterpret_cast<const float4*>(S + static_cast<size_t>(r) * P + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int n = 0; n < TURN; ++n) {
+                const int idx = (n0 + n) * kSsmThreads + threadIdx.x, r = idx / (kSsmCols / 4), c = (idx % (kSsmCols / 4)) * 4;
+                uint2 hi, lo;
+                split_pair(rs[n].x, rs[n].y, hi.x, lo.x);
+                split_pair(rs[n].z, rs[n].w, hi.y, lo.y);
+                *reinterpret_cast<uint2*>(Sh + r * kLdX + c) = hi;
+                *reinterpret_cast<uint2*>(Sl + r * kLdX + c) = lo;
+            }
         }
     } else {
         for (int idx = threadIdx.x; idx < NP * kSsmCols; idx += kSsmThreads) {
@@ -589,6 +675,7 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
         }
     }
     chunk_decays(p, h, row0, nt, s_d, s_c);
+    cp_async_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i0 = warp * 16;
     const bool busy = i0 < nt;                  // the warp has tokens
@@ -596,7 +683,15 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
 #pragma unroll
     for (int k = 0; k < NP / 16; ++k) ldmatrix_x4(cf[k], smem_addr(BCs + (i0 + (lane & 15)) * LDN + k * 16 + ((lane >> 4) << 3)));
     __syncthreads();
-    stage_bf16<kSsmChunk, NP, LDN>(BCs, p.B + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
+    if (HELD && p.vec) {
+#pragma unroll
+        for (int n = 0; n < B_PACKS; ++n) {
+            const int idx = n * kSsmThreads + threadIdx.x, r = idx / (NP / 8), c = (idx % (NP / 8)) * 8;
+            *reinterpret_cast<uint4*>(BCs + r * LDN + c) = rb[n];
+        }
+    } else {
+        stage_bf16<kSsmChunk, NP, LDN>(BCs, B, p.ld, nt, N, p.vec);
+    }
     float acc[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
@@ -641,8 +736,8 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
             for (int e = 0; e < 2; ++e) {
                 const int j = j0 + 8 * q + 2 * (lane & 3) + e;
                 const float cj = s_c[j], dj = s_d[j];
-                s[q][e] = j <= ia ? s[q][e] * expf(ca - cj) * dj : 0.f;
-                s[q][2 + e] = j <= ib ? s[q][2 + e] * expf(cb - cj) * dj : 0.f;
+                s[q][e] = j <= ia ? s[q][e] * __expf(ca - cj) * dj : 0.f;
+                s[q][2 + e] = j <= ib ? s[q][2 + e] * __expf(cb - cj) * dj : 0.f;
             }
         uint32_t ah[4], al[4];
         split_pair(s[0][0], s[0][1], ah[0], al[0]);
@@ -724,7 +819,7 @@ gated_group_norm_kernel(const float* __restrict__ y, const TZ* __restrict__ z, i
             g[0] = a.x; g[1] = a.y; g[2] = b.x; g[3] = b.y;
         }
 #pragma unroll
-        for (int e = 0; e < V; ++e) u[e] *= silu_f(g[e]);
+        for (int e = 0; e < V; ++e) u[e] *= silu_for<TO>(g[e]);
     };
     float u[HELD][V], sq = 0.f;
 #pragma unroll

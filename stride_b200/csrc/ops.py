@@ -118,11 +118,15 @@ _SIGNATURES = {
     "stride_rglru_scan_pieces": ("rglru", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_moe_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "stride_moe_route_plan": ("moe", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                      c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "stride_moe_plan": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "stride_grouped_gemm": ("moe", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                     c_float, c_void_p, c_int, c_void_p]),
     "stride_grouped_gemm_tc5": ("moe_tc", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                            c_float, c_void_p, c_int, c_void_p, c_void_p]),
+    "stride_moe_stream": ("moe_stream", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                                         c_float, c_void_p, c_int, c_void_p]),
     "stride_gather_rows": ("moe_tc", [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p]),
     "stride_moe_combine": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_relu_squared": ("moe", [c_void_p, c_longlong, c_int, c_void_p]),
@@ -222,7 +226,8 @@ _CLASS_OF = {
     "stride_qkv_rotate_norm": "rotation + head norms + cache write",
     "stride_rglru_conv": "recurrent block: convolution",
     "stride_rglru_gates": "recurrent block: gates", "stride_rglru_scan": "recurrent block: recurrence", "stride_rglru_scan_pieces": "recurrent block: recurrence", "stride_moe_route": "router",
-    "stride_moe_plan": "router", "stride_grouped_gemm": "expert products", "stride_moe_combine": "expert sum",
+    "stride_moe_plan": "router", "stride_moe_route_plan": "router", "stride_grouped_gemm": "expert products", "stride_moe_combine": "expert sum",
+    "stride_moe_stream": "expert products (weight streaming)",
     "stride_grouped_gemm_tc5": "expert products (tcgen05)", "stride_gather_rows": "expert rows gathered",
     "stride_relu_squared": "relu^2", "stride_gated_act": "act * up", "stride_pointwise": "gates and caps", "stride_weighted_sum": "sum of branches",
     "stride_delta_prepare": "delta rule: convolution, unit vectors, decay", "stride_delta_scan": "delta rule: recurrence",
@@ -1156,6 +1161,31 @@ def moe_select_groups(logits, correction, seq_of_token, ids, weights, experts: i
                                            int(keep), float(route_scale), rule, _stream()), "moe_select_groups")
 
 
+# Steps of at most this many tokens run router product, choice and plan in one launch. 0 turns it off.
+MOE_ROUTE_PLAN_MAX_TOKENS = int(_os.environ.get("STRIDE_B200_MOE_ROUTE_PLAN_MAX_TOKENS", "16"))
+
+
+def moe_route_plan(x, w_router, logits, correction, seq_of_token, ids, weights, experts: int, groups: int, keep: int, route_scale: float,
+                   offsets, perm_token, row_of, rank_tmp, row_weight, ticket, softmax: bool = False, group_max: bool = False,
+                   keep_scores: bool = False) -> bool:
+    """``logits = x @ w_router.T`` (float32 sums), ``moe_select_groups`` on them and ``moe_plan``, for a few bfloat16 tokens. ``ticket``: an
+    int32 word, zero between launches. False when it does not take the sizes (nothing was done)."""
+    tokens, hidden = x.shape
+    if x.dtype != torch.bfloat16 or w_router.dtype != torch.bfloat16 or w_router.shape[1] != hidden or logits.shape != (tokens, w_router.shape[0]):
+        return False
+    rule = (1 if softmax else 0) | (2 if group_max else 0) | (4 if keep_scores else 0)
+    code = _fn("stride_moe_route_plan")(
+        _dev(x, "x"), _dev(w_router, "w_router"), w_router.shape[0], hidden, _dev(logits, "logits", torch.float32),
+        _opt(correction, "correction", torch.float32), _opt(seq_of_token, "seq_of_token", torch.int32), _dev(ids, "ids", torch.int32),
+        _dev(weights, "weights", torch.float32), tokens, int(experts), ids.shape[1], int(groups), int(keep), float(route_scale), rule,
+        _dev(offsets, "offsets", torch.int32), _dev(perm_token, "perm_token", torch.int32), _dev(row_of, "row_of", torch.int32),
+        _dev(rank_tmp, "rank_tmp", torch.int32), _opt(row_weight, "row_weight", torch.float32), _dev(ticket, "ticket", torch.int32), _stream())
+    if code == -2:
+        return False
+    _check(code, "moe_route_plan")
+    return True
+
+
 def moe_plan(ids, experts: int, offsets, perm_token, row_of, rank_tmp, weights=None, row_weight=None) -> None:
     """``row_weight`` (float32, one per row; with ``weights`` [tokens, top]) receives every row's weight."""
     tokens, top = ids.shape
@@ -1189,6 +1219,24 @@ GROUPED_TC_MIN_ROWS = int(_os.environ.get("STRIDE_GROUPED_TC_MIN_ROWS", "1024"))
 
 def grouped_tc_wanted(dtype, rows: int) -> bool:
     return dtype == torch.bfloat16 and GROUPED_TC_MIN_ROWS > 0 and rows >= GROUPED_TC_MIN_ROWS
+
+
+# Steps of at most this many tokens run the experts' products on the weight-streaming form (moe_stream.cu). 0 turns it off.
+MOE_STREAM_MAX_TOKENS = int(_os.environ.get("STRIDE_B200_MOE_STREAM_MAX_TOKENS", "64"))
+
+
+def moe_stream(a, row_map, w, offsets, c, act: int = 0, limit: float = 0.0, alpha: float = 1.0, row_weight=None) -> bool:
+    """``grouped_gemm`` for a few bfloat16 rows an expert. False when it does not take the sizes (nothing was done)."""
+    experts, n, k = w.shape
+    if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.shape[1] != k or c.dtype not in (torch.bfloat16, torch.float32):
+        return False
+    code = _fn("stride_moe_stream")(_dev(a, "a"), a.shape[1], _opt(row_map, "row_map", torch.int32), _dev(w, "w"), _dev(offsets, "offsets", torch.int32),
+                                    experts, _dev(c, "c"), c.shape[1], n, k, int(act), float(limit), float(alpha),
+                                    _opt(row_weight, "row_weight", torch.float32), 1 if c.dtype == torch.float32 else 0, _stream())
+    if code == -2:
+        return False
+    _check(code, "moe_stream")
+    return True
 
 
 def gather_rows(x, perm, offsets, experts: int, xs, max_rows: int) -> bool:
@@ -1707,10 +1755,11 @@ def decode_scratch_floats(tokens: int, nq: int, nkv: int, hd: int, max_context: 
 
 def paged_attention_decode(q, q_stride: int, out, k_pages, v_pages, block_table, seq_of_token, positions, scratch, nq: int,
                            nkv: int, hd: int, page_size: int, scale: float, window: int, max_context: int, softcap: float = 0.0,
-                           sinks=None, slopes=None, gate_col: int = -1, rel=None) -> None:
+                           sinks=None, slopes=None, gate_col: int = -1, rel=None, precise_cap: bool = False) -> None:
     """Attention for single decoded tokens (one query per row), split over the keys;
     ``scratch`` (float32, zero when first used) holds the ticket counters and the
-    partial results of the splits. ``softcap``, ``sinks`` and ``slopes`` as for ``paged_attention``. ``gate_col`` >= 0: columns
+    partial results of the splits. ``softcap``, ``sinks`` and ``slopes`` as for ``paged_attention``; ``precise_cap``: the cap's tanh in
+    32-bit accuracy instead of the hardware's short one. ``gate_col`` >= 0: columns
     ``gate_col .. gate_col + nq - 1`` of a row of ``q`` hold one logit per head, and head h's output leaves the kernel
     multiplied by the sigmoid of its logit. ``rel`` as for ``paged_attention``."""
     tokens = out.shape[0]
@@ -1721,7 +1770,7 @@ def paged_attention_decode(q, q_stride: int, out, k_pages, v_pages, block_table,
         _dev(v_pages, "v_pages", torch.bfloat16), k_pages.shape[0], _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], _dev(seq_of_token, "seq_of_token", torch.int32), _dev(positions, "positions", torch.int32),
         _dev(scratch, "scratch", torch.float32), scratch.numel(), tokens, nq, nkv, hd, page_size, float(scale), int(window),
-        float(softcap), _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), int(gate_col), int(max_context),
+        -float(softcap) if precise_cap else float(softcap), _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), int(gate_col), int(max_context),
         _tc_buffers(q.device, 0)["status"].data_ptr(), _stream()),
         "paged_attention_decode")
 
@@ -1731,7 +1780,7 @@ TC_ATTENTION = _os.environ.get("STRIDE_B200_TC_ATTENTION", "1") != "0"
 
 def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_table, q_start, q_len, ctx_len, num_seqs: int,
                                nq: int, nkv: int, hd: int, page_size: int, scale: float, window: int, softcap: float = 0.0,
-                               sinks=None, slopes=None, rel=None) -> bool:
+                               sinks=None, slopes=None, rel=None, precise_cap: bool = False) -> bool:
     """The tcgen05 version of ``paged_attention_prefill`` (same arguments). Returns False
     when it does not take the sizes; the caller then uses the mma.sync kernel."""
     tokens = out.shape[0]
@@ -1742,7 +1791,7 @@ def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_ta
         _dev(q, "q", torch.bfloat16), q_stride, _dev(out, "out", torch.bfloat16), _dev(k_pages, "k_pages", torch.bfloat16),
         _dev(v_pages, "v_pages", torch.bfloat16), k_pages.shape[0], _dev(block_table, "block_table", torch.int32),
         block_table.shape[1], _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32),
-        _dev(ctx_len, "ctx_len", torch.int32), num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), float(softcap),
+        _dev(ctx_len, "ctx_len", torch.int32), num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), -float(softcap) if precise_cap else float(softcap),
         _opt(sinks, "sinks", torch.float32), _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), st["status"].data_ptr(), _stream())
     if code == -2:
         return False
@@ -1752,7 +1801,7 @@ def paged_attention_prefill_tc(q, q_stride: int, out, k_pages, v_pages, block_ta
 
 def paged_attention_prefill(q, q_stride: int, out, k_pages, v_pages, block_table, q_start, q_len, ctx_len, num_seqs: int,
                             nq: int, nkv: int, hd: int, page_size: int, scale: float, window: int, softcap: float = 0.0,
-                            sinks=None, slopes=None, rel=None) -> None:
+                            sinks=None, slopes=None, rel=None, precise_cap: bool = False) -> None:
     """Attention for the first ``num_seqs`` requests of the step (portions of any
     length), which own the rows of ``out``. ``softcap`` and ``sinks`` as for ``paged_attention``."""
     tokens = out.shape[0]
@@ -1762,7 +1811,7 @@ def paged_attention_prefill(q, q_stride: int, out, k_pages, v_pages, block_table
         _dev(q, "q", torch.bfloat16), q_stride, _dev(out, "out", torch.bfloat16), _dev(k_pages, "k_pages", torch.bfloat16),
         _dev(v_pages, "v_pages", torch.bfloat16), _dev(block_table, "block_table", torch.int32), block_table.shape[1],
         _dev(q_start, "q_start", torch.int32), _dev(q_len, "q_len", torch.int32), _dev(ctx_len, "ctx_len", torch.int32),
-        num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), float(softcap), _opt(sinks, "sinks", torch.float32),
+        num_seqs, tokens, nq, nkv, hd, page_size, float(scale), int(window), -float(softcap) if precise_cap else float(softcap), _opt(sinks, "sinks", torch.float32),
         _opt(slopes, "slopes", torch.float32), *_rel_args(rel, nq), _stream()), "paged_attention_prefill")
 
 

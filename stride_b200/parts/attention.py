@@ -11,7 +11,7 @@ Spec params, all optional:
 * ``values`` ``keys``: there is no value projection; a token's value is its key as projected (bias included),
   before the rotation. The key rows are used twice in the fused projection, so keys and values go through the same
   kernels and pages as ever.
-* ``softcap`` c: scaled scores become c tanh(s / c).
+* ``softcap`` c: scaled scores become c tanh(s / c). ``precise_cap``: with a tanh of 32-bit accuracy in the bfloat16 kernels, too.
 * ``sinks``: a tensor ``sink`` [heads]; exp(sink_h) joins the denominator of head h's softmax.
 * ``output_gate``: a matrix ``g`` [heads * head_dim, hidden]; the concatenated heads are multiplied by
   sigmoid(g x) before the output projection.
@@ -104,7 +104,7 @@ class PagedAttention(Mixer):
         self.position = build_part("position", s.position, runtime)
         p = dict(s.params)
         self.values_are_keys = p.get("values") == "keys"
-        self.softcap = float(p.get("softcap", 0.0))
+        self.softcap, self.precise_cap = float(p.get("softcap", 0.0)), bool(p.get("precise_cap", False))
         self.zero_sinks = p.get("sinks") == "zero"
         self.has_sinks, self.gated = bool(p.get("sinks", False)) and not self.zero_sinks, bool(p.get("output_gate", False))
         self.taps, self.weighted_qk = int(p.get("conv", 0)), p.get("qk_norm") == "weighted"
@@ -486,7 +486,7 @@ class PagedAttention(Mixer):
         split = min(ctx.decode_tail_start, tokens)          # portions before, single decoded tokens after
         if split > 0:
             args = (qkv[:split], self.qkv_dim, attn[:split], cache.k_pages, cache.v_pages, table, ctx.q_start, ctx.q_len,
-                    ctx.ctx_len, ctx.decode_tail_seq, *geometry, self.softcap, self.sinks, self.slopes, self.rel)
+                    ctx.ctx_len, ctx.decode_tail_seq, *geometry, self.softcap, self.sinks, self.slopes, self.rel, self.precise_cap)
             # tcgen05 kernel first; the mma.sync kernel takes what it refuses (odd page sizes)
             if not (ops.TC_ATTENTION and ops.paged_attention_prefill_tc(*args)):
                 ops.paged_attention_prefill(*args)
@@ -496,7 +496,7 @@ class PagedAttention(Mixer):
             ops.paged_attention_decode(qkv[split:tokens], self.qkv_dim, attn[split:tokens], cache.k_pages, cache.v_pages, table,
                                        ctx.seq_of_token[split:tokens], ctx.positions[split:tokens], scratch, *geometry,
                                        ctx.context_bound, self.softcap, self.sinks, self.slopes,
-                                       self.q_dim + self.kv_cols if self.fused_gate else -1, self.rel)
+                                       self.q_dim + self.kv_cols if self.fused_gate else -1, self.rel, self.precise_cap)
             return split if self.fused_gate else tokens
         return tokens
 

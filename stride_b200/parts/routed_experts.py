@@ -158,26 +158,30 @@ class RoutedExperts(FeedForward):
         ids = self.rt.buffer("moe_ids", tokens, top, i32)
         weights = self.rt.buffer("moe_weights", tokens, top, torch.float32)
         logits = self.rt.buffer("moe_logits", tokens, self.w_router.shape[0], torch.float32)
-        ops.linear(x, self.w_router, logits)            # float32 sums of exact products, float32 logits
-        if self.router_kind == "sigmoid_groups":
-            ops.moe_select_sigmoid(logits, self.correction, ctx.seq_of_token[:tokens], ids, weights, self.experts, self.groups, self.keep,
-                                   self.route_scale)
-        elif self.router_kind in ("softmax_groups", "sigmoid_scores"):
-            ops.moe_select_groups(logits, None, ctx.seq_of_token[:tokens], ids, weights, self.experts, self.groups, self.keep,
-                                  self.route_scale, softmax=self.router_kind == "softmax_groups", group_max=True, keep_scores=True)
-        else:
-            ops.moe_select(logits if not self.shared_gate else logits[:, :self.experts].contiguous(), self.bias,
-                           ctx.seq_of_token[:tokens], ids, weights)
         row_of = self.rt.buffer("moe_row_of", tokens, top, i32)
         perm = self.rt.buffer("moe_perm", tokens, top, i32).view(-1)
         rank = self.rt.buffer("moe_rank", tokens, top, i32).view(-1)
         offsets = self.rt.scratch(f"moe_offsets_{self.experts}", self.experts + 1, i32)
         row_weight = self.rt.buffer("moe_row_weight", tokens, top, torch.float32).view(-1) if self.weigh_inputs else None
-        ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank, weights if self.weigh_inputs else None, row_weight)
+        seq_of = ctx.seq_of_token[:tokens]
+        rule = dict(softmax=self.router_kind == "softmax_groups", group_max=self.router_kind != "sigmoid_groups",
+                    keep_scores=self.router_kind != "sigmoid_groups")
+        if not (self.router_kind != "softmax_top" and tokens <= ops.MOE_ROUTE_PLAN_MAX_TOKENS
+                and ops.moe_route_plan(x, self.w_router, logits, self.correction, seq_of, ids, weights, self.experts, self.groups, self.keep,
+                                       self.route_scale, offsets, perm, row_of, rank, row_weight, self.rt.scratch("moe_ticket", 1, i32), **rule)):
+            ops.linear(x, self.w_router, logits)            # float32 sums of exact products, float32 logits
+            if self.router_kind == "softmax_top":
+                ops.moe_select(logits if not self.shared_gate else logits[:, :self.experts].contiguous(), self.bias, seq_of, ids, weights)
+            else:
+                ops.moe_select_groups(logits, self.correction, seq_of, ids, weights, self.experts, self.groups, self.keep, self.route_scale, **rule)
+            ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank, weights if self.weigh_inputs else None, row_weight)
         hidden_rows = self.rt.buffer("moe_hidden", tokens, top * self.ff).view(pairs, self.ff)
         y = self.rt.buffer("moe_y", tokens, top * self.hidden, torch.float32).view(pairs, self.hidden)
         act = (2 if self.clamped else 3) if self.gated else 1
-        if not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight):
+        if tokens <= ops.MOE_STREAM_MAX_TOKENS and ops.moe_stream(x, perm, self.w_up, offsets, hidden_rows, act, self.limit, self.alpha, row_weight):
+            if not ops.moe_stream(hidden_rows, None, self.w_down, offsets, y):
+                ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
+        elif not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight):
             ops.grouped_gemm(x, perm, self.w_up, offsets, hidden_rows, pairs, act=act, limit=self.limit, alpha=self.alpha, row_weight=row_weight)
             ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
         shared = None
