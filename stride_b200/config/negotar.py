@@ -60,8 +60,10 @@ def _check_attention(m: dict, where: str) -> None:
     if not isinstance(m.get("v_mix", False), bool):
         raise ConfigError(f"{where}: v_mix must be true or false")
     rot = m.get("rot")
+    if rot is None:             # no rotation
+        return
     if not isinstance(rot, dict):
-        raise ConfigError(f"{where}: `rot` must be an object with `base` and `dims`")
+        raise ConfigError(f"{where}: `rot` must be an object with `base` and `dims`, or null")
     dims = _int(rot, "dims", where + ".rot", minimum=0)
     if dims % 2 or dims > dim or not _num(rot, "base", where + ".rot") > 0:
         raise ConfigError(f"{where}: rot.dims must be even and at most dim, rot.base positive")
@@ -170,7 +172,7 @@ class NegotarConfig:
         return NormSpec(kind="rmsnorm", width=self.width, eps=self.norm_eps, prefix=name, params=(("tensor", name), ("weight_offset", 1.0), *params))
 
     def _attention(self, m: dict, prefix: str, mixing: str | None) -> MixerSpec:
-        rot, scaling = m["rot"], None
+        rot, scaling = m.get("rot") or {"base": 1.0, "dims": 0}, None
         sc = rot.get("scaling")
         if sc:
             scaling = RopeScaling(rope_type="llama3", factor=float(sc["factor"]), low_freq_factor=float(sc["low"]),

@@ -1,4 +1,4 @@
-"""Named shapes, as config.json dictionaries (Llama 3, two of the Nidilix design, a tiny one of the Netusun and of the Dopudra design): the tiny shapes used
+"""Named shapes, as config.json dictionaries (Llama 3, two of the Nidilix design, a tiny one of the Netusun, of the Dopudra and of the Negotar design): the tiny shapes used
 for correctness runs (tiny-d has the head size and widths that the tensor-core
 kernels take) and the 8B / 3B / 70B shapes used for measurements. The
 reference keeps such presets in crates/stride-model/src/presets.rs:73-91."""
@@ -72,7 +72,19 @@ def _dopudra_tiny() -> dict:
             "embedding": {"scale": 0.8}, "layers": layers}
 
 
+def _negotar_tiny() -> dict:
+    """Four layers: state space, two attention layers with mixed values around another state space; mixtures in three of them."""
+    attention = {"heads": 4, "kv_heads": 2, "dim": 48, "vdim": 32, "scale": 48 ** -0.5, "softcap": 25.0, "v_mix": True,
+                 "rot": {"base": 10000.0, "dims": 32, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 128}}}
+    memory = {"heads": 4, "vdim": 64, "groups": 2, "state": 64, "conv": 4, "norm_groups": 2}
+    moe = {"kind": "moe", "expert": {"ff": 64}, "router": {"experts": 8, "top": 2}}
+    kinds = [("mamba2", memory, moe), ("attention", attention, moe), ("mamba2", memory, None), ("attention", attention, moe)]
+    layers = [{"type": kind, "mixer": copy.deepcopy(mixer), "mlp": copy.deepcopy(mlp)} for kind, mixer, mlp in kinds]
+    return {"architecture": "Negotar", "width": 128, "vocab": 384, "norm": {"eps": 1e-6}, "logit_scale": 0.8, "layers": layers}
+
+
 PRESETS = {
+    "negotar-tiny": _negotar_tiny(),
     "dopudra-tiny": _dopudra_tiny(),
     "netusun-tiny": _netusun_tiny(),
     "nidilix-tiny": _nidilix(128, 512, "rarb", {"width": 160, "blocks": 5, "conv": 3},

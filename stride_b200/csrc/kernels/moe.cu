@@ -12,7 +12,7 @@
 //   moe_plan      one CTA counts the rows of every expert, lays the (token, choice) pairs out expert by expert and
 //                 writes where each pair went: `offsets` [experts + 1], `perm_token` [rows] and `row_of` [tokens, top], and
 //                 on request every row's weight;
-//   moe_route_plan  for a few bfloat16 tokens: the router's product, the choice by the rule above and the plan in one launch;
+//   moe_route_rule  for a few bfloat16 tokens: the router's product and the choice by the rule above in one launch;
 //   grouped_gemm  C[p, :] = act(A[src(p), :] W[e(p)]^T) for the rows p of every expert e, the tiles of all experts in
 //                 one launch (the CTA finds its expert from `offsets` on the device, so nothing goes back to the
 //                 host and the step can be replayed from a graph); float32 FMA with a fixed k order for float32
@@ -21,7 +21,7 @@
 //                 and writes g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), N / 2 wide;
 //                 act 3 reads the same pairs and writes g sigmoid(g) u; with `row_weight` the sums of row p are multiplied by
 //                 row_weight[p] first (the product of a row that was multiplied by it);
-//   moe_combine   out[t] = sum_k weight[t, k] * Y[row_of[t, k]] (no weights: the plain sum) (+ a shared expert's output, optionally times the
+//   moe_combine   out[t] = sum_k weight[t, k] * Y[row_of[t, k]] (no weights: the plain sum; no row_of: pair (t, k) is row t * top + k) (+ a shared expert's output, optionally times the
 //                 sigmoid of a per-token logit), in the order of k.
 // A row's result depends only on that row: not on the batch, nor on where the plan put it.
 #include "common.cuh"
@@ -148,15 +148,16 @@ moe_select_kernel(const float* __restrict__ logits, const float* __restrict__ bi
 }
 
 // One warp's choice for a token by the group router's rule: z_row its logits, `choice` and `gscore` shared memory of kMaxExperts
-// floats each, ids and weights the token's `top` places.
-__device__ __forceinline__ void choose_by_rule(const float* z_row, const float* __restrict__ correction, float* choice, float* gscore,
+// floats each, ids and weights the token's `top` places. SLOTS: experts a lane looks after.
+template <int SLOTS>
+__device__ __forceinline__ void choose_by_rule_n(const float* z_row, const float* __restrict__ correction, float* choice, float* gscore,
                                                int32_t* __restrict__ ids, float* __restrict__ weights, int experts, int top, int groups, int keep,
                                                float route_scale, int rule, int lane) {
-    float score[kMaxExperts / 32];       // lane holds experts lane, lane + 32, ...
+    float score[SLOTS];       // lane holds experts lane, lane + 32, ...
     if (rule & kRuleSoftmax) {           // softmax over all experts: largest logit, exponentials, their sum in a fixed order
         float top_z = -INFINITY;
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             const int e = i * 32 + lane;
             score[i] = e < experts ? z_row[e] : -INFINITY;
             top_z = fmaxf(top_z, score[i]);
@@ -165,21 +166,21 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
         for (int o = 16; o > 0; o >>= 1) top_z = fmaxf(top_z, __shfl_xor_sync(0xffffffffu, top_z, o));
         float sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             score[i] = i * 32 + lane < experts ? expf(score[i] - top_z) : 0.f;
             sum += score[i];
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             const int e = i * 32 + lane;
             score[i] /= sum;
             if (e < experts) choice[e] = score[i] + (correction ? correction[e] : 0.f);
         }
     } else {
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             const int e = i * 32 + lane;
             score[i] = 0.f;
             if (e < experts) {
@@ -218,7 +219,7 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
             if (best_g != 0x7fffffff) kept[best_g >> 5] |= 1u << (best_g & 31);        // every lane keeps the whole set
         }
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             const int e = i * 32 + lane;
             if (e < experts) {
                 const int g = e / size;
@@ -227,10 +228,10 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
         }
         __syncwarp();
     }
-    float z[kMaxExperts / 32];
-    bool open_[kMaxExperts / 32];
+    float z[SLOTS];
+    bool open_[SLOTS];
 #pragma unroll
-    for (int i = 0; i < kMaxExperts / 32; ++i) {
+    for (int i = 0; i < SLOTS; ++i) {
         const int e = i * 32 + lane;
         open_[i] = e < experts;
         z[i] = e < experts ? choice[e] : -INFINITY;
@@ -241,7 +242,7 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
         float best = -INFINITY, best_score = 0.f;
         int best_e = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i) {
+        for (int i = 0; i < SLOTS; ++i) {
             const int e = i * 32 + lane;
             if (open_[i] && (best_e == 0x7fffffff || z[i] > best)) { best = z[i]; best_e = e; best_score = score[i]; }
         }
@@ -253,7 +254,7 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
             if (oe != 0x7fffffff && (best_e == 0x7fffffff || ob > best || (ob == best && oe < best_e))) { best = ob; best_e = oe; best_score = os; }
         }
 #pragma unroll
-        for (int i = 0; i < kMaxExperts / 32; ++i)
+        for (int i = 0; i < SLOTS; ++i)
             if (i * 32 + lane == best_e) open_[i] = false;       // taken
         denom += best_score;
         if (lane == k) { mine = best_score; mine_id = best_e == 0x7fffffff ? -1 : best_e; }
@@ -262,6 +263,14 @@ __device__ __forceinline__ void choose_by_rule(const float* z_row, const float* 
         ids[lane] = mine_id;
         weights[lane] = (rule & kRuleKeepScores) ? mine * route_scale : mine / (denom + 1e-20f) * route_scale;
     }
+}
+
+__device__ __forceinline__ void choose_by_rule(const float* z_row, const float* __restrict__ correction, float* choice, float* gscore,
+                                               int32_t* __restrict__ ids, float* __restrict__ weights, int experts, int top, int groups, int keep,
+                                               float route_scale, int rule, int lane) {
+    if (experts <= 32) choose_by_rule_n<1>(z_row, correction, choice, gscore, ids, weights, experts, top, groups, keep, route_scale, rule, lane);
+    else if (experts <= 64) choose_by_rule_n<2>(z_row, correction, choice, gscore, ids, weights, experts, top, groups, keep, route_scale, rule, lane);
+    else choose_by_rule_n<kMaxExperts / 32>(z_row, correction, choice, gscore, ids, weights, experts, top, groups, keep, route_scale, rule, lane);
 }
 
 // logits: [tokens, ld] float32 (the first `experts` columns of a row). One warp per token.
@@ -346,37 +355,39 @@ moe_plan_kernel(const int32_t* __restrict__ ids, int pairs, int experts, int32_t
     plan_rows(ids, pairs, experts, offsets, perm_token, row_of, rank_tmp, weights, row_weight, top);
 }
 
-// Router product, choice and plan of a step of a few tokens in one launch: a CTA a token, a warp four experts at a time, every
-// logit a float32 sum in an order that depends on `hidden` only; the CTA that finishes last (a ticket, left at zero) lays out the rows.
-// rows: of w (the experts, then any more whose logits are only written, such as a shared expert's gate).
-constexpr int kRouteThreads = 256, kRouteMaxRows = kMaxExperts + 32;
+// Router product and choice of a step of a few tokens in one launch: a CTA a token, a warp PER rows of w at a time, every logit a
+// float32 sum in an order that depends on `hidden` only. rows: of w (the experts, then any more whose logits are only written, such
+// as a shared expert's gate).
+constexpr int kRouteThreads = 512, kRouteMaxRows = kMaxExperts + 32;
+template <int PER>
 __global__ void __launch_bounds__(kRouteThreads)
-moe_route_plan_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int rows, int hidden, float* __restrict__ logits,
-                      const float* __restrict__ correction, const int32_t* __restrict__ seq_of_token, int32_t* ids, float* weights, int experts, int top,
-                      int groups, int keep, float route_scale, int rule, int32_t* __restrict__ offsets, int32_t* __restrict__ perm_token,
-                      int32_t* __restrict__ row_of, int32_t* __restrict__ rank_tmp, float* __restrict__ row_weight, unsigned* ticket) {
+moe_route_rule_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, int rows, int hidden, float* __restrict__ logits,
+                      const float* __restrict__ correction, const int32_t* __restrict__ seq_of_token, int32_t* __restrict__ ids,
+                      float* __restrict__ weights, int experts, int top, int groups, int keep, float route_scale, int rule) {
     __shared__ float z[kRouteMaxRows];
     __shared__ float choice[kMaxExperts], gscore[kMaxExperts];
-    __shared__ bool last;
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool padded = seq_of_token && seq_of_token[t] < 0;
     const __nv_bfloat16* row = x + static_cast<size_t>(t) * hidden;
-    for (int e0 = warp * 4; e0 < rows; e0 += kRouteThreads / 32 * 4) {
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
+    for (int e0 = warp * PER; e0 < rows; e0 += kRouteThreads / 32 * PER) {
+        float acc[PER];
+#pragma unroll
+        for (int u = 0; u < PER; ++u) acc[u] = 0.f;
+#pragma unroll 16 / PER
         for (int k = lane * 8; k < hidden; k += 256) {
             const uint4 a = *reinterpret_cast<const uint4*>(row + k);
-            uint4 b[4];
+            uint4 b[PER];
 #pragma unroll
-            for (int u = 0; u < 4; ++u)
+            for (int u = 0; u < PER; ++u)
                 b[u] = e0 + u < rows ? __ldg(reinterpret_cast<const uint4*>(w + static_cast<size_t>(e0 + u) * hidden + k)) : make_uint4(0, 0, 0, 0);
             const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&a);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const float2 fa = __bfloat1622float2(pa[i]);
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
+                for (int u = 0; u < PER; ++u) {
                     const float2 fb = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&b[u])[i]);
                     acc[u] = fmaf(fa.x, fb.x, acc[u]);
                     acc[u] = fmaf(fa.y, fb.y, acc[u]);
@@ -384,7 +395,7 @@ moe_route_plan_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* 
             }
         }
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
+        for (int u = 0; u < PER; ++u) {
             acc[u] = warp_sum(acc[u]);
             if (lane == 0 && e0 + u < rows) {
                 z[e0 + u] = acc[u];
@@ -393,27 +404,17 @@ moe_route_plan_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* 
         }
     }
     __syncthreads();
-    if (warp == 0) {
-        int32_t* my_ids = ids + static_cast<size_t>(t) * top;
-        float* my_weights = weights + static_cast<size_t>(t) * top;
-        if (seq_of_token && seq_of_token[t] < 0) {
-            for (int k = lane; k < top; k += 32) {
-                my_ids[k] = -1;
-                my_weights[k] = 0.f;
-            }
-        } else {
-            choose_by_rule(z, correction, choice, gscore, my_ids, my_weights, experts, top, groups, keep, route_scale, rule, lane);
+    if (warp != 0) return;
+    ids += static_cast<size_t>(t) * top;
+    weights += static_cast<size_t>(t) * top;
+    if (padded) {
+        for (int k = lane; k < top; k += 32) {
+            ids[k] = -1;
+            weights[k] = 0.f;
         }
-        __threadfence();
-        __syncwarp();
-        if (lane == 0) {
-            last = atomicAdd(ticket, 1u) + 1 == gridDim.x;
-            if (last) *ticket = 0;
-            __threadfence();
-        }
+        return;
     }
-    __syncthreads();
-    if (last) plan_rows(ids, static_cast<int>(gridDim.x) * top, experts, offsets, perm_token, row_of, rank_tmp, weights, row_weight, top);
+    choose_by_rule(z, correction, choice, gscore, ids, weights, experts, top, groups, keep, route_scale, rule, lane);
 }
 
 __device__ __forceinline__ float clamped_gated(float g, float u, float limit, float alpha) {
@@ -591,7 +592,7 @@ moe_combine_kernel(const float* __restrict__ Y, const int32_t* __restrict__ row_
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < hidden; c += gridDim.y * blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
-            const int row = row_of[static_cast<size_t>(t) * top + k];
+            const int row = row_of ? row_of[static_cast<size_t>(t) * top + k] : t * top + k;
             if (row >= 0) acc = fmaf(weights ? weights[static_cast<size_t>(t) * top + k] : 1.f, Y[static_cast<size_t>(row) * hidden + c], acc);
         }
         if (shared) acc = fmaf(share, to_f32(shared[static_cast<size_t>(t) * hidden + c]), acc);
@@ -686,20 +687,19 @@ int stride_moe_plan(const int32_t* ids, int tokens, int top, int experts, int32_
     return STRIDE_LAUNCH_STATUS();
 }
 
-// ticket: one word, zero between launches. Returns -2 for what it does not take (hidden no multiple of 8, unaligned operands).
-int stride_moe_route_plan(const void* x, const void* w, int rows, int hidden, float* logits, const float* correction, const int32_t* seq_of_token,
+// logits: [tokens, rows]. Returns -2 for what it does not take (hidden no multiple of 8, unaligned operands).
+int stride_moe_route_rule(const void* x, const void* w, int rows, int hidden, float* logits, const float* correction, const int32_t* seq_of_token,
                           int32_t* ids, float* weights, int tokens, int experts, int top, int groups, int keep, float route_scale, int rule,
-                          int32_t* offsets, int32_t* perm_token, int32_t* row_of, int32_t* rank_tmp, float* row_weight, unsigned* ticket,
                           cudaStream_t stream) {
     if (tokens < 0 || hidden <= 0 || experts <= 0 || rows < experts || top <= 0 || top > experts || groups <= 0 || keep <= 0 || keep > groups ||
-        experts % groups || top > keep * (experts / groups) || rule < 0 || rule > 7 || !ticket)
+        experts % groups || top > keep * (experts / groups) || rule < 0 || rule > 7)
         return STRIDE_BAD_ARGUMENT;
     if (experts > kMaxExperts || top > kMaxTop || rows > kRouteMaxRows || hidden % 8 || (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) % 16)
         return STRIDE_UNSUPPORTED;
     if (tokens == 0) return 0;
-    stride::launch(moe_route_plan_kernel, dim3(tokens), dim3(kRouteThreads), 0, stream, static_cast<const __nv_bfloat16*>(x),
-                   static_cast<const __nv_bfloat16*>(w), rows, hidden, logits, correction, seq_of_token, ids, weights, experts, top, groups, keep,
-                   route_scale, rule, offsets, perm_token, row_of, rank_tmp, row_weight, ticket);
+    auto kernel = rows <= 16 ? moe_route_rule_kernel<1> : rows <= 32 ? moe_route_rule_kernel<2> : moe_route_rule_kernel<4>;
+    stride::launch(kernel, dim3(tokens), dim3(kRouteThreads), 0, stream, static_cast<const __nv_bfloat16*>(x), static_cast<const __nv_bfloat16*>(w), rows,
+                   hidden, logits, correction, seq_of_token, ids, weights, experts, top, groups, keep, route_scale, rule);
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -1,6 +1,8 @@
 // The experts' products of a routed feed-forward for steps of a few tokens (decoding), bfloat16, where the time goes into
 // reading the chosen experts' weights once:
-//   C[p, :] = act(A[src(p), :] W[e(p)]^T)   for the rows p of every expert e, rows lying expert by expert (`offsets`).
+//   C[p, :] = act(A[src(p), :] W[e(p)]^T)   for the rows p of every expert e.
+// Either rows lie expert by expert (`offsets`, a plan's), or there is no plan: row p is (token, choice) pair p, which belongs to
+// expert ids[p], and every CTA picks its expert's pairs out of the list itself (`pairs` of them, up to 512; src(p) = p / top).
 //
 // A CTA takes 16 rows of one expert's weights and all of K, its four warps every fourth block of 32 columns. The weights are the
 // 16-row operand of mma.sync m16n8k16 and go from global memory straight into fragments, 16 bytes a lane and row: a lane's eight
@@ -19,6 +21,7 @@ namespace stride {
 constexpr int kStreamWarps = 4;
 constexpr int kStreamRows = 16;          // weight rows a CTA
 constexpr int kStreamTokens = 32;        // rows of A a turn
+constexpr int kStreamMaxPairs = 512;
 constexpr int kStreamAhead = 4;          // blocks of 32 columns whose weights a warp asks for together
 
 __device__ __forceinline__ float stream_pair(int act, float g, float u, float limit, float alpha) {
@@ -62,14 +65,36 @@ __device__ __forceinline__ void stream_rows(const __nv_bfloat16* w_lo, const __n
 template <typename OutT>
 __global__ void __launch_bounds__(kStreamWarps * 32)
 moe_stream_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32_t* __restrict__ row_map, const __nv_bfloat16* __restrict__ W,
-                  const int32_t* __restrict__ offsets, OutT* __restrict__ C, int ldc, int N, int K, int act, float limit, float alpha,
-                  const float* __restrict__ row_weight) {
+                  const int32_t* __restrict__ offsets, const int32_t* __restrict__ ids, int pairs, int top, OutT* __restrict__ C, int ldc, int N, int K,
+                  int act, float limit, float alpha, const float* __restrict__ row_weight) {
     __shared__ float red[kStreamWarps][kStreamRows][kStreamTokens + 1];
+    __shared__ int picked[kStreamMaxPairs];
     pdl_trigger();
     pdl_wait();
-    const int e = blockIdx.y, lo = offsets[e], hi = offsets[e + 1];
-    if (lo >= hi) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tg = lane & 3;
+    const int e = blockIdx.y;
+    int lo = 0, hi = 0;
+    if (ids) {              // this expert's pairs in ascending order; every warp finds (and notes) all of them, so nobody waits
+        for (int p0 = 0; p0 < pairs; p0 += 128) {
+            int own[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) own[i] = p0 + i * 32 + lane < pairs ? ids[p0 + i * 32 + lane] : -1;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (p0 + i * 32 >= pairs) break;
+                const unsigned mine = __ballot_sync(0xffffffffu, own[i] == e);
+                if ((mine >> lane) & 1u) picked[hi + __popc(mine & ((1u << lane) - 1u))] = p0 + i * 32 + lane;
+                hi += __popc(mine);
+            }
+        }
+        if (hi == 0) return;
+        __syncwarp();
+    } else {
+        lo = offsets[e];
+        hi = offsets[e + 1];
+        if (lo >= hi) return;
+    }
+    auto row_at = [&](int p) { return ids ? picked[p] : p; };
     const int n0 = blockIdx.x * kStreamRows;
     const __nv_bfloat16* We = W + (static_cast<size_t>(e) * N + n0) * K;
     const __nv_bfloat16* w_lo = n0 + g < N ? We + static_cast<size_t>(g) * K : nullptr;
@@ -80,7 +105,8 @@ moe_stream_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32_t* _
 #pragma unroll
         for (int n = 0; n < 4; ++n) {
             const int p = p0 + n * 8 + g;
-            src[n] = n * 8 + g < rows ? A + static_cast<size_t>(row_map ? row_map[p] : p) * lda : nullptr;
+            src[n] = nullptr;
+            if (n * 8 + g < rows) src[n] = A + static_cast<size_t>(ids ? picked[p] / top : row_map ? row_map[p] : p) * lda;
         }
         float acc[4][4];
 #pragma unroll
@@ -100,13 +126,13 @@ moe_stream_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32_t* _
             float v = 0.f;
 #pragma unroll
             for (int w = 0; w < kStreamWarps; ++w) v += red[w][r][t];
-            return row_weight ? v * row_weight[p0 + t] : v;
+            return row_weight ? v * row_weight[row_at(p0 + t)] : v;
         };
         if (act >= 2) {                         // rows 2i and 2i + 1: gate and up of a unit
             for (int i = threadIdx.x; i < kStreamRows / 2 * rows; i += blockDim.x) {
                 const int unit = i % (kStreamRows / 2), t = i / (kStreamRows / 2);
                 if (n0 + 2 * unit + 1 < N)
-                    C[static_cast<size_t>(p0 + t) * ldc + n0 / 2 + unit] = from_f32<OutT>(stream_pair(act, sum(2 * unit, t), sum(2 * unit + 1, t), limit, alpha));
+                    C[static_cast<size_t>(row_at(p0 + t)) * ldc + n0 / 2 + unit] = from_f32<OutT>(stream_pair(act, sum(2 * unit, t), sum(2 * unit + 1, t), limit, alpha));
             }
         } else {
             for (int i = threadIdx.x; i < kStreamRows * rows; i += blockDim.x) {
@@ -117,7 +143,7 @@ moe_stream_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int32_t* _
                     v = fmaxf(v, 0.f);
                     v *= v;
                 }
-                C[static_cast<size_t>(p0 + t) * ldc + n0 + r] = from_f32<OutT>(v);
+                C[static_cast<size_t>(row_at(p0 + t)) * ldc + n0 + r] = from_f32<OutT>(v);
             }
         }
     }
@@ -130,18 +156,22 @@ using namespace stride;
 extern "C" {
 
 // C: [rows, N] (N / 2 with act 2 and 3), bfloat16 or float32. Returns -2 for what it does not take (K or lda no multiple of 8,
-// unaligned operands); the caller then uses the other grouped product.
-int stride_moe_stream(const void* A, int lda, const int32_t* row_map, const void* W, const int32_t* offsets, int experts, void* C, int ldc, int N,
-                      int K, int act, float limit, float alpha, const float* row_weight, int out_is_f32, cudaStream_t stream) {
+// unaligned operands, too many pairs); the caller then uses the other grouped product. ids null: rows by offsets and row_map;
+// else pairs by ids [pairs], row p of A being pair p's token (top 1: the pair itself).
+int stride_moe_stream(const void* A, int lda, const int32_t* row_map, const void* W, const int32_t* offsets, const int32_t* ids, int pairs, int top,
+                      int experts, void* C, int ldc, int N, int K, int act, float limit, float alpha, const float* row_weight, int out_is_f32,
+                      cudaStream_t stream) {
+    if ((!ids && !offsets) || (ids && (pairs < 0 || top <= 0))) return STRIDE_BAD_ARGUMENT;
+    if (ids && pairs > kStreamMaxPairs) return STRIDE_UNSUPPORTED;
     if (experts <= 0 || N <= 0 || K <= 0 || lda < K || act < 0 || act > 3 || ldc < (act >= 2 ? N / 2 : N) || (act >= 2 && N % 2)) return STRIDE_BAD_ARGUMENT;
     if (experts > 65535 || K % 8 || lda % 8 || (reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) % 16) return STRIDE_UNSUPPORTED;
     const dim3 grid((N + kStreamRows - 1) / kStreamRows, experts), block(kStreamWarps * 32);
     if (out_is_f32)
         stride::launch(moe_stream_kernel<float>, grid, block, 0, stream, static_cast<const __nv_bfloat16*>(A), lda, row_map,
-                       static_cast<const __nv_bfloat16*>(W), offsets, static_cast<float*>(C), ldc, N, K, act, limit, alpha, row_weight);
+                       static_cast<const __nv_bfloat16*>(W), offsets, ids, pairs, top, static_cast<float*>(C), ldc, N, K, act, limit, alpha, row_weight);
     else
         stride::launch(moe_stream_kernel<__nv_bfloat16>, grid, block, 0, stream, static_cast<const __nv_bfloat16*>(A), lda, row_map,
-                       static_cast<const __nv_bfloat16*>(W), offsets, static_cast<__nv_bfloat16*>(C), ldc, N, K, act, limit, alpha, row_weight);
+                       static_cast<const __nv_bfloat16*>(W), offsets, ids, pairs, top, static_cast<__nv_bfloat16*>(C), ldc, N, K, act, limit, alpha, row_weight);
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -335,8 +335,9 @@ qkv_unit_norm_vec_kernel(T* __restrict__ qkv, int row_stride, const float* __res
     }
 }
 
-// One head a group of LANES lanes (16: two heads a warp, for heads of at most 16 packs). A head's entries pass through shared
-// memory between bias and rotation, since an entry's partner lies in another lane. hd / vd: columns of a head in the row and in
+// One head a group of LANES lanes (16: two heads a warp, for heads of at most 16 packs). An entry's partner lies in another lane: where
+// a lane holds one pack and half the turned entries are whole packs (SHUFFLE), the partner's pack is the same pack of one other
+// lane; otherwise a head's entries pass through shared memory between bias and rotation. hd / vd: columns of a head in the row and in
 // the pages; qd / vdim: its entries (the rest are zeros). V entries a pack: 16 bytes of the compute type where sizes and
 // pointers allow, else single entries. The order of a head's sum depends on qd, LANES and V only.
 struct RotateNormArgs {
@@ -356,10 +357,10 @@ struct RotateNormArgs {
     const float* share;
 };
 
-template <typename T, int LANES, int V>
+template <typename T, int LANES, int V, bool SHUFFLE>
 __global__ void __launch_bounds__(kNormWarps * 32)
 qkv_rotate_norm_kernel(const RotateNormArgs p) {
-    __shared__ __align__(16) float stage[kNormWarps * (32 / LANES)][kMaxHead];
+    __shared__ __align__(16) float stage[SHUFFLE ? 1 : kNormWarps * (32 / LANES)][SHUFFLE ? 4 : kMaxHead];
     pdl_trigger();
     pdl_wait();
     constexpr int kPerWarp = 32 / LANES;
@@ -372,7 +373,7 @@ qkv_rotate_norm_kernel(const RotateNormArgs p) {
     const int width = live ? (is_value ? p.vdim : p.qd) : 0, cols = is_value ? p.vd : p.hd;
     const int column = is_value ? (p.nq + p.nkv) * p.hd + (head - p.nq - p.nkv) * p.vd : head * p.hd;
     T* x = static_cast<T*>(p.qkv) + static_cast<size_t>(t) * p.row_stride + (live ? column : 0);
-    float* mine = stage[warp * kPerWarp + sub];
+    float* mine = stage[SHUFFLE ? 0 : warp * kPerWarp + sub];
     auto load = [](const auto* from, float* v) {
         if constexpr (V == 1) v[0] = to_f32(*from);
         else Pack<T>::load(from, v);
@@ -396,15 +397,39 @@ qkv_rotate_norm_kernel(const RotateNormArgs p) {
 #pragma unroll
                 for (int j = 0; j < V; ++j) v[i][j] = __fadd_rn(v[i][j], b[j]);
             }
-            if (!is_value) {
+            if (!SHUFFLE && !is_value) {
 #pragma unroll
                 for (int j = 0; j < V; ++j) mine[d + j] = v[i][j];
             }
+        } else if (SHUFFLE) {
+#pragma unroll
+            for (int j = 0; j < V; ++j) v[i][j] = 0.f;
         }
     }
-    __syncwarp();
+    if (!SHUFFLE) __syncwarp();
     float sq = 0.f;
-    if (!is_value) {
+    if constexpr (SHUFFLE) {
+        const int half = p.rot / 2, d = lane * V;
+        const bool low = d < half, turns = !is_value && d < p.rot;
+        float c[V], s[V], other[V];
+        if (turns) {
+            const size_t at = static_cast<size_t>(p.positions[t]) * half + (low ? d : d - half);
+            load_floats(p.cos_t + at, c);
+            load_floats(p.sin_t + at, s);
+        }
+        const int from = turns ? (low ? lane + half / V : lane - half / V) : lane;
+#pragma unroll
+        for (int j = 0; j < V; ++j) other[j] = __shfl_sync(0xffffffffu, v[0][j], from, LANES);
+        if (turns) {
+#pragma unroll
+            for (int j = 0; j < V; ++j)
+                v[0][j] = low ? __fmul_rn(v[0][j], c[j]) - __fmul_rn(other[j], s[j]) : __fmul_rn(v[0][j], c[j]) + __fmul_rn(other[j], s[j]);
+        }
+        if (!is_value) {
+#pragma unroll
+            for (int j = 0; j < V; ++j) sq = fmaf(v[0][j], v[0][j], sq);
+        }
+    } else if (!is_value) {
         const int half = p.rot / 2, at = half ? p.positions[t] : 0;
 #pragma unroll
         for (int i = 0; i < kPacks; ++i) {
@@ -451,13 +476,16 @@ qkv_rotate_norm_kernel(const RotateNormArgs p) {
             for (int j = 0; j < V; ++j) v[i][j] = 0.f;
         } else if (is_value) {
             if (first && p.share) {
+                float kept[V];
+                load_floats(first + d, kept);
 #pragma unroll
-                for (int j = 0; j < V; ++j)
-                    if (d + j < width) v[i][j] = __fadd_rn(__fmul_rn(1.f - share, v[i][j]), __fmul_rn(share, first[d + j]));
+                for (int j = 0; j < V; ++j) v[i][j] = __fadd_rn(__fmul_rn(1.f - share, v[i][j]), __fmul_rn(share, kept[j]));
             } else if (first) {
+                if constexpr (V == 1) first[d] = v[i][0];
+                else {
 #pragma unroll
-                for (int j = 0; j < V; ++j)
-                    if (d + j < width) first[d + j] = v[i][j];
+                    for (int j = 0; j < V; j += 4) Pack<float>::store(first + d + j, v[i] + j);
+                }
             }
         } else {
 #pragma unroll
@@ -540,20 +568,27 @@ int stride_qkv_rotate_norm(void* qkv, int row_stride, const float* bias, const i
     const int pack = dtype == STRIDE_DTYPE_F32 ? 4 : 8;
     // packs never straddle a head's end, nor the middle of what turns
     const bool vec = hd % pack == 0 && vd % pack == 0 && qd % pack == 0 && vdim % pack == 0 && row_stride % pack == 0 && aligned(qkv) &&
-                     aligned(bias) && aligned(k_pages) && aligned(v_pages);
+                     aligned(bias) && aligned(k_pages) && aligned(v_pages) && aligned(first);
     const bool halves = vec && hd <= 16 * pack && vd <= 16 * pack;       // two heads a warp
+    const bool shuffle = vec && (rot / 2) % pack == 0 && (halves || dtype == STRIDE_DTYPE_BF16) && aligned(cos_t) && aligned(sin_t);     // one pack a lane
     const int groups = halves ? (nq + 2 * nkv + 1) / 2 : nq + 2 * nkv;
     const dim3 grid(tokens, (groups + kNormWarps - 1) / kNormWarps), block(kNormWarps * 32);
-    if (dtype == STRIDE_DTYPE_F32)
-        stride::launch(halves ? qkv_rotate_norm_kernel<float, 16, 4> : vec ? qkv_rotate_norm_kernel<float, 32, 4> : qkv_rotate_norm_kernel<float, 32, 1>,
-                       grid, block, 0, stream, p);
-    else if (dtype == STRIDE_DTYPE_BF16)
-        stride::launch(halves ? qkv_rotate_norm_kernel<__nv_bfloat16, 16, 8>
-                       : vec  ? qkv_rotate_norm_kernel<__nv_bfloat16, 32, 8>
-                              : qkv_rotate_norm_kernel<__nv_bfloat16, 32, 1>,
-                       grid, block, 0, stream, p);
-    else
+    if (dtype == STRIDE_DTYPE_F32) {
+        auto kernel = shuffle  ? qkv_rotate_norm_kernel<float, 16, 4, true>
+                      : halves ? qkv_rotate_norm_kernel<float, 16, 4, false>
+                      : vec    ? qkv_rotate_norm_kernel<float, 32, 4, false>
+                               : qkv_rotate_norm_kernel<float, 32, 1, false>;
+        stride::launch(kernel, grid, block, 0, stream, p);
+    } else if (dtype == STRIDE_DTYPE_BF16) {
+        using T = __nv_bfloat16;
+        auto kernel = shuffle  ? (halves ? qkv_rotate_norm_kernel<T, 16, 8, true> : qkv_rotate_norm_kernel<T, 32, 8, true>)
+                      : halves ? qkv_rotate_norm_kernel<T, 16, 8, false>
+                      : vec    ? qkv_rotate_norm_kernel<T, 32, 8, false>
+                               : qkv_rotate_norm_kernel<T, 32, 1, false>;
+        stride::launch(kernel, grid, block, 0, stream, p);
+    } else {
         return STRIDE_BAD_ARGUMENT;
+    }
     return STRIDE_LAUNCH_STATUS();
 }
 

@@ -118,15 +118,15 @@ _SIGNATURES = {
     "stride_rglru_scan_pieces": ("rglru", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_moe_route": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
-    "stride_moe_route_plan": ("moe", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                      c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "stride_moe_route_rule": ("moe", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                      c_int, c_float, c_int, c_void_p]),
     "stride_moe_plan": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "stride_grouped_gemm": ("moe", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                     c_float, c_void_p, c_int, c_void_p]),
     "stride_grouped_gemm_tc5": ("moe_tc", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                            c_float, c_void_p, c_int, c_void_p, c_void_p]),
-    "stride_moe_stream": ("moe_stream", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                                         c_float, c_void_p, c_int, c_void_p]),
+    "stride_moe_stream": ("moe_stream", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                                         c_int, c_float, c_float, c_void_p, c_int, c_void_p]),
     "stride_gather_rows": ("moe_tc", [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p]),
     "stride_moe_combine": ("moe", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "stride_relu_squared": ("moe", [c_void_p, c_longlong, c_int, c_void_p]),
@@ -226,7 +226,7 @@ _CLASS_OF = {
     "stride_qkv_rotate_norm": "rotation + head norms + cache write",
     "stride_rglru_conv": "recurrent block: convolution",
     "stride_rglru_gates": "recurrent block: gates", "stride_rglru_scan": "recurrent block: recurrence", "stride_rglru_scan_pieces": "recurrent block: recurrence", "stride_moe_route": "router",
-    "stride_moe_plan": "router", "stride_moe_route_plan": "router", "stride_grouped_gemm": "expert products", "stride_moe_combine": "expert sum",
+    "stride_moe_plan": "router", "stride_moe_route_rule": "router", "stride_grouped_gemm": "expert products", "stride_moe_combine": "expert sum",
     "stride_moe_stream": "expert products (weight streaming)",
     "stride_grouped_gemm_tc5": "expert products (tcgen05)", "stride_gather_rows": "expert rows gathered",
     "stride_relu_squared": "relu^2", "stride_gated_act": "act * up", "stride_pointwise": "gates and caps", "stride_weighted_sum": "sum of branches",
@@ -1161,28 +1161,25 @@ def moe_select_groups(logits, correction, seq_of_token, ids, weights, experts: i
                                            int(keep), float(route_scale), rule, _stream()), "moe_select_groups")
 
 
-# Steps of at most this many tokens run router product, choice and plan in one launch. 0 turns it off.
-MOE_ROUTE_PLAN_MAX_TOKENS = int(_os.environ.get("STRIDE_B200_MOE_ROUTE_PLAN_MAX_TOKENS", "16"))
+# Steps of at most this many tokens run router product and choice in one launch. 0 turns it off.
+MOE_ROUTE_RULE_MAX_TOKENS = int(_os.environ.get("STRIDE_B200_MOE_ROUTE_RULE_MAX_TOKENS", "16"))
 
 
-def moe_route_plan(x, w_router, logits, correction, seq_of_token, ids, weights, experts: int, groups: int, keep: int, route_scale: float,
-                   offsets, perm_token, row_of, rank_tmp, row_weight, ticket, softmax: bool = False, group_max: bool = False,
-                   keep_scores: bool = False) -> bool:
-    """``logits = x @ w_router.T`` (float32 sums), ``moe_select_groups`` on them and ``moe_plan``, for a few bfloat16 tokens. ``ticket``: an
-    int32 word, zero between launches. False when it does not take the sizes (nothing was done)."""
+def moe_route_rule(x, w_router, logits, correction, seq_of_token, ids, weights, experts: int, groups: int, keep: int, route_scale: float,
+                   softmax: bool = False, group_max: bool = False, keep_scores: bool = False) -> bool:
+    """``logits = x @ w_router.T`` (float32 sums) and ``moe_select_groups`` on them, for a few bfloat16 tokens. False when it does not
+    take the sizes (nothing was done)."""
     tokens, hidden = x.shape
     if x.dtype != torch.bfloat16 or w_router.dtype != torch.bfloat16 or w_router.shape[1] != hidden or logits.shape != (tokens, w_router.shape[0]):
         return False
     rule = (1 if softmax else 0) | (2 if group_max else 0) | (4 if keep_scores else 0)
-    code = _fn("stride_moe_route_plan")(
+    code = _fn("stride_moe_route_rule")(
         _dev(x, "x"), _dev(w_router, "w_router"), w_router.shape[0], hidden, _dev(logits, "logits", torch.float32),
         _opt(correction, "correction", torch.float32), _opt(seq_of_token, "seq_of_token", torch.int32), _dev(ids, "ids", torch.int32),
-        _dev(weights, "weights", torch.float32), tokens, int(experts), ids.shape[1], int(groups), int(keep), float(route_scale), rule,
-        _dev(offsets, "offsets", torch.int32), _dev(perm_token, "perm_token", torch.int32), _dev(row_of, "row_of", torch.int32),
-        _dev(rank_tmp, "rank_tmp", torch.int32), _opt(row_weight, "row_weight", torch.float32), _dev(ticket, "ticket", torch.int32), _stream())
+        _dev(weights, "weights", torch.float32), tokens, int(experts), ids.shape[1], int(groups), int(keep), float(route_scale), rule, _stream())
     if code == -2:
         return False
-    _check(code, "moe_route_plan")
+    _check(code, "moe_route_rule")
     return True
 
 
@@ -1225,18 +1222,30 @@ def grouped_tc_wanted(dtype, rows: int) -> bool:
 MOE_STREAM_MAX_TOKENS = int(_os.environ.get("STRIDE_B200_MOE_STREAM_MAX_TOKENS", "64"))
 
 
-def moe_stream(a, row_map, w, offsets, c, act: int = 0, limit: float = 0.0, alpha: float = 1.0, row_weight=None) -> bool:
-    """``grouped_gemm`` for a few bfloat16 rows an expert. False when it does not take the sizes (nothing was done)."""
+def moe_stream(a, row_map, w, offsets, c, act: int = 0, limit: float = 0.0, alpha: float = 1.0, row_weight=None, ids=None,
+               by_pair: bool = False) -> bool:
+    """``grouped_gemm`` for a few bfloat16 rows an expert. With ``ids`` (int32 [tokens, top], -1: none) there is no plan: row p of ``c`` is
+    pair p, computed from row p // top of ``a`` (``by_pair``: from row p) with the weights of expert ``ids.view(-1)[p]``. False when it
+    does not take the sizes (nothing was done)."""
     experts, n, k = w.shape
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.shape[1] != k or c.dtype not in (torch.bfloat16, torch.float32):
         return False
-    code = _fn("stride_moe_stream")(_dev(a, "a"), a.shape[1], _opt(row_map, "row_map", torch.int32), _dev(w, "w"), _dev(offsets, "offsets", torch.int32),
-                                    experts, _dev(c, "c"), c.shape[1], n, k, int(act), float(limit), float(alpha),
-                                    _opt(row_weight, "row_weight", torch.float32), 1 if c.dtype == torch.float32 else 0, _stream())
+    pairs, top = (0, 0) if ids is None else (ids.numel(), 1 if by_pair else ids.shape[1])
+    code = _fn("stride_moe_stream")(_dev(a, "a"), a.shape[1], _opt(row_map, "row_map", torch.int32), _dev(w, "w"), _opt(offsets, "offsets", torch.int32),
+                                    _opt(ids, "ids", torch.int32), pairs, top, experts, _dev(c, "c"), c.shape[1], n, k, int(act), float(limit),
+                                    float(alpha), _opt(row_weight, "row_weight", torch.float32), 1 if c.dtype == torch.float32 else 0, _stream())
     if code == -2:
         return False
     _check(code, "moe_stream")
     return True
+
+
+MOE_STREAM_MAX_PAIRS = 512          # (token, choice) pairs that run without a plan
+
+
+def moe_stream_supported(dtype, tokens: int, top: int, hidden: int, ff: int) -> bool:
+    """Sizes whose experts' products all run on the weight-streaming form without a plan."""
+    return dtype == torch.bfloat16 and tokens <= MOE_STREAM_MAX_TOKENS and tokens * top <= MOE_STREAM_MAX_PAIRS and hidden % 8 == 0 and ff % 8 == 0
 
 
 def gather_rows(x, perm, offsets, experts: int, xs, max_rows: int) -> bool:
@@ -1269,15 +1278,15 @@ def grouped_gemm_tc(a, w, offsets, c, max_rows: int, act: int = 0, limit: float 
 
 
 def moe_combine(y, row_of, weights, shared, out, shared_gate=None) -> None:
-    """``weights`` None: the plain sum of a token's rows. ``shared_gate``: a float32 column (one logit per token, possibly a column of a wider buffer); the shared expert's
+    """``weights`` None: the plain sum of a token's rows. ``row_of`` None: pair (t, k) is row t * top + k of ``y``. ``shared_gate``: a float32 column (one logit per token, possibly a column of a wider buffer); the shared expert's
     output is then multiplied by its sigmoid."""
     tokens, hidden = out.shape
     gate_ptr, gate_stride = (None, 0) if shared_gate is None else (shared_gate.data_ptr(), shared_gate.stride(0))
     if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.shape[0] != tokens):
         raise KernelError("moe_combine: the shared expert's gate must be one float32 logit per token")
-    _check(_fn("stride_moe_combine")(_dev(y, "y", torch.float32), _dev(row_of, "row_of", torch.int32), _opt(weights, "weights", torch.float32),
+    _check(_fn("stride_moe_combine")(_dev(y, "y", torch.float32), _opt(row_of, "row_of", torch.int32), _opt(weights, "weights", torch.float32),
                                      _opt(shared, "shared", out.dtype), gate_ptr, gate_stride, _dev(out, "out"), tokens, hidden,
-                                     row_of.shape[1], _code(out.dtype), _stream()), "moe_combine")
+                                     y.shape[0] // tokens if row_of is None else row_of.shape[1], _code(out.dtype), _stream()), "moe_combine")
 
 
 def relu_squared(x) -> None:

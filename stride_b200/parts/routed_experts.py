@@ -7,7 +7,8 @@ a shared expert of the same form runs for every token and is added.
 On the device: the router's product leaves float32 logits, a kernel chooses, a one-CTA plan lays the (token, choice) pairs out expert by expert, two
 grouped products run all experts' rows in one launch each (the first gathers its rows through the plan and applies
 the activation, the second leaves float32 rows), and one kernel sums a token's rows with its weights and the
-shared expert's output. Nothing returns to the host, so a step can be captured in a graph.
+shared expert's output. Steps of a few tokens in bfloat16 models choose in the kernel of the router's product and stream the chosen
+experts' weights through products that find their rows in the list of choices (``csrc/kernels/moe_stream.cu``): no plan. Nothing returns to the host, so a step can be captured in a graph.
 
 Spec: ``hidden``, ``intermediate`` (an expert's width), ``activation`` (``relu_squared``), params ``experts``, ``top``,
 ``shared`` (the shared expert's width, 0 for none), ``router_bias``. Tensors under the prefix: ``router``, ``router.b``,
@@ -158,32 +159,27 @@ class RoutedExperts(FeedForward):
         ids = self.rt.buffer("moe_ids", tokens, top, i32)
         weights = self.rt.buffer("moe_weights", tokens, top, torch.float32)
         logits = self.rt.buffer("moe_logits", tokens, self.w_router.shape[0], torch.float32)
-        row_of = self.rt.buffer("moe_row_of", tokens, top, i32)
-        perm = self.rt.buffer("moe_perm", tokens, top, i32).view(-1)
-        rank = self.rt.buffer("moe_rank", tokens, top, i32).view(-1)
-        offsets = self.rt.scratch(f"moe_offsets_{self.experts}", self.experts + 1, i32)
-        row_weight = self.rt.buffer("moe_row_weight", tokens, top, torch.float32).view(-1) if self.weigh_inputs else None
         seq_of = ctx.seq_of_token[:tokens]
         rule = dict(softmax=self.router_kind == "softmax_groups", group_max=self.router_kind != "sigmoid_groups",
                     keep_scores=self.router_kind != "sigmoid_groups")
-        if not (self.router_kind != "softmax_top" and tokens <= ops.MOE_ROUTE_PLAN_MAX_TOKENS
-                and ops.moe_route_plan(x, self.w_router, logits, self.correction, seq_of, ids, weights, self.experts, self.groups, self.keep,
-                                       self.route_scale, offsets, perm, row_of, rank, row_weight, self.rt.scratch("moe_ticket", 1, i32), **rule)):
+        if not (self.router_kind != "softmax_top" and tokens <= ops.MOE_ROUTE_RULE_MAX_TOKENS
+                and ops.moe_route_rule(x, self.w_router, logits, self.correction, seq_of, ids, weights, self.experts, self.groups, self.keep,
+                                       self.route_scale, **rule)):
             ops.linear(x, self.w_router, logits)            # float32 sums of exact products, float32 logits
             if self.router_kind == "softmax_top":
                 ops.moe_select(logits if not self.shared_gate else logits[:, :self.experts].contiguous(), self.bias, seq_of, ids, weights)
             else:
                 ops.moe_select_groups(logits, self.correction, seq_of, ids, weights, self.experts, self.groups, self.keep, self.route_scale, **rule)
-            ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank, weights if self.weigh_inputs else None, row_weight)
         hidden_rows = self.rt.buffer("moe_hidden", tokens, top * self.ff).view(pairs, self.ff)
         y = self.rt.buffer("moe_y", tokens, top * self.hidden, torch.float32).view(pairs, self.hidden)
         act = (2 if self.clamped else 3) if self.gated else 1
-        if tokens <= ops.MOE_STREAM_MAX_TOKENS and ops.moe_stream(x, perm, self.w_up, offsets, hidden_rows, act, self.limit, self.alpha, row_weight):
-            if not ops.moe_stream(hidden_rows, None, self.w_down, offsets, y):
-                ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
-        elif not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight):
-            ops.grouped_gemm(x, perm, self.w_up, offsets, hidden_rows, pairs, act=act, limit=self.limit, alpha=self.alpha, row_weight=row_weight)
-            ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
+        row_of = None
+        if ops.moe_stream_supported(x.dtype, tokens, top, self.hidden, self.ff):
+            # a few tokens: the products find their rows in the list of choices, pair by pair
+            ops.moe_stream(x, None, self.w_up, None, hidden_rows, act, self.limit, self.alpha, weights if self.weigh_inputs else None, ids)
+            ops.moe_stream(hidden_rows, None, self.w_down, None, y, ids=ids, by_pair=True)
+        else:
+            row_of = self._products_by_plan(x, ids, weights, hidden_rows, y, tokens, pairs, act)
         shared = None
         if self.shared_ff:
             mid = self.rt.buffer("moe_shared_mid", tokens, self.shared_ff)
@@ -206,6 +202,19 @@ class RoutedExperts(FeedForward):
         ops.moe_combine(y, row_of, None if self.weigh_inputs else weights, shared, out, logits[:, self.experts] if self.shared_gate else None)
         return out
 
+    def _products_by_plan(self, x, ids, weights, hidden_rows, y, tokens, pairs, act):
+        """Rows laid out expert by expert; returns where every pair's row lies."""
+        top, i32 = self.top, torch.int32
+        row_of = self.rt.buffer("moe_row_of", tokens, top, i32)
+        perm = self.rt.buffer("moe_perm", tokens, top, i32).view(-1)
+        rank = self.rt.buffer("moe_rank", tokens, top, i32).view(-1)
+        offsets = self.rt.scratch(f"moe_offsets_{self.experts}", self.experts + 1, i32)
+        row_weight = self.rt.buffer("moe_row_weight", tokens, top, torch.float32).view(-1) if self.weigh_inputs else None
+        ops.moe_plan(ids, self.experts, offsets, perm, row_of, rank, weights if self.weigh_inputs else None, row_weight)
+        if not self._products_tc(x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight):
+            ops.grouped_gemm(x, perm, self.w_up, offsets, hidden_rows, pairs, act=act, limit=self.limit, alpha=self.alpha, row_weight=row_weight)
+            ops.grouped_gemm(hidden_rows, None, self.w_down, offsets, y, pairs, act=0)
+        return row_of
 
     def _products_tc(self, x, perm, offsets, hidden_rows, y, tokens, pairs, act, row_weight) -> bool:
         """Both products of all experts on the tcgen05 kernel, for steps of many rows: the tokens' rows are laid out

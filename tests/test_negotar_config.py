@@ -41,6 +41,9 @@ def test_layout():
     position = spec.layers[3].mixer.position
     assert dict(position.params)["rotated"] == 8 and position.scaling == RopeScaling("llama3", 4.0, 2.0, 3.0, 100)
     assert spec.layers[1].mixer.position.scaling is None and spec.layers[1].feed_forward is None and spec.layers[1].ffn_norm is None
+    d = copy.deepcopy(cases.CASE_A)
+    d["layers"][1]["mixer"]["rot"] = None
+    assert dict(config_from_dict(d).to_model_spec().layers[1].mixer.position.params)["rotated"] == 0
     f = spec.layers[3].feed_forward
     assert (f.kind, f.intermediate, f.activation) == ("routed_experts", 16, "silu")
     assert dict(f.params) == {"experts": 7, "top": 4, "router": "sigmoid_scores", "weigh": "inputs"}
@@ -117,6 +120,7 @@ def test_plain_mechanisms_have_the_properties_they_name():
     (lambda d: d["layers"][1]["mixer"].update(v_mix=1), "v_mix"),
     (lambda d: d["layers"][3]["mixer"].update(vdim=20), "cannot be mixed"),
     (lambda d: d["layers"][3]["mixer"].update(softcap=-1.0), "softcap"),
+    (lambda d: d["layers"][1]["mixer"].update(rot=3), "rot"),
     (lambda d: d["layers"][1]["mixer"]["rot"].update(dims=7), "even"),
     (lambda d: d["layers"][1]["mixer"]["rot"].update(dims=22), "at most"),
     (lambda d: d["layers"][3]["mixer"]["rot"]["scaling"].update(factor=0), "factor"),

@@ -332,6 +332,95 @@ def test_the_mixture_alone(gpu, dtype, tol, rows, width, ff, experts, top):
     close(got.cpu()[clear], want[clear], tol)
 
 
+@pytest.mark.parametrize("act,row_weights", [(3, True), (2, False), (1, True), (0, False)])
+@pytest.mark.parametrize("experts,n,k,counts", [(4, 48, 64, [3, 0, 9, 1]), (3, 40, 2056, [1, 17, 33]), (5, 22, 136, [8, 70, 0, 16, 2]), (2, 2, 8, [1, 1]),
+                                                (6, 130, 328, [0, 0, 5, 31, 32, 0])])
+def test_expert_products_for_a_few_rows(gpu, act, row_weights, experts, n, k, counts):
+    """The weight-streaming form against float64: empty experts, more rows than a turn takes, rows found through a map, widths that end
+    inside a tile; both output types. Rows behind the last one stay as they are."""
+    from stride_b200.csrc import ops
+    g = torch.Generator().manual_seed(n + k + act)
+    rows = sum(counts)
+    offsets = dev([0] + [sum(counts[:e + 1]) for e in range(experts)])
+    a, w = torch.randn(rows + 2, k, generator=g).bfloat16(), (torch.randn(experts, n, k, generator=g) * k ** -0.5).bfloat16()
+    perm = torch.randperm(rows, generator=g)
+    f = torch.rand(rows, generator=g) if row_weights else torch.ones(rows)
+    want, at = [], 0
+    for e, c in enumerate(counts):
+        z = (a[perm[at:at + c]].double() @ w[e].double().T) * f[at:at + c, None].double()
+        if act == 1:
+            z = torch.relu(z) ** 2
+        elif act == 2:
+            gate, up = z[:, 0::2].clamp(max=0.9), z[:, 1::2].clamp(-0.9, 0.9)
+            z = gate * torch.sigmoid(1.7 * gate) * (up + 1.0)
+        elif act == 3:
+            z = plain.silu(z[:, 0::2]) * z[:, 1::2]
+        want.append(z)
+        at += c
+    want = torch.cat(want)
+    for out_type, tol in ((torch.float32, 2e-5), (torch.bfloat16, 6e-3)):
+        out = torch.full((rows + 2, want.shape[1]), 5.0, dtype=out_type, device="cuda")
+        assert ops.moe_stream(a.cuda(), perm.to(torch.int32).cuda(), w.cuda(), offsets, out, act, 0.9, 1.7, f.cuda() if row_weights else None)
+        close(out[:rows], want, tol)
+        assert (out[rows:] == 5.0).all()
+
+
+@pytest.mark.parametrize("tokens,experts,top", [(3, 4, 2), (16, 32, 32), (64, 8, 8), (1, 1, 1), (20, 7, 3)])
+@pytest.mark.parametrize("act", [3, 1])
+def test_expert_products_pair_by_pair(gpu, tokens, experts, top, act):
+    """The same without a plan: row p of the output is pair p, a padded token's pairs are left alone, up to 512 pairs; experts chosen by
+    more tokens than a turn takes."""
+    from stride_b200.csrc import ops
+    g = torch.Generator().manual_seed(tokens + experts)
+    n, k = 40, 72
+    x, w = torch.randn(tokens, k, generator=g).bfloat16(), (torch.randn(experts, n, k, generator=g) * k ** -0.5).bfloat16()
+    ids = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(tokens)]).to(torch.int32)
+    if tokens > 2:
+        ids[1] = -1
+    f = torch.rand(tokens, top, generator=g)
+    out = torch.full((tokens * top, n if act == 1 else n // 2), 5.0, device="cuda")
+    assert ops.moe_stream(x.cuda(), None, w.cuda(), None, out, act, row_weight=f.cuda(), ids=ids.cuda())
+    back = torch.full((tokens * top, n), 5.0, dtype=torch.bfloat16, device="cuda")
+    pair_rows = torch.randn(tokens * top, k, generator=g).bfloat16()
+    assert ops.moe_stream(pair_rows.cuda(), None, w.cuda(), None, back, ids=ids.cuda(), by_pair=True)
+    for t in range(tokens):
+        for c in range(top):
+            p, e = t * top + c, int(ids[t, c])
+            if e < 0:
+                assert (out[p] == 5.0).all() and (back[p] == 5.0).all()
+                continue
+            z = (w[e].double() @ x[t].double()) * f[t, c].double()
+            close(out[p], plain.silu(z[0::2]) * z[1::2] if act == 3 else torch.relu(z) ** 2, 3e-5)
+            close(back[p], w[e].double() @ pair_rows[p].double(), 6e-3)
+
+
+@pytest.mark.parametrize("experts,top,extra,hidden,tokens", [(5, 2, 0, 64, 3), (32, 4, 1, 2056, 16), (256, 32, 0, 328, 9), (1, 1, 0, 8, 1), (33, 7, 3, 1024, 16),
+                                                             (16, 16, 0, 264, 5), (64, 3, 0, 40, 2)])
+@pytest.mark.parametrize("keep_scores", [True, False])
+def test_router_and_choice_in_one_launch(gpu, experts, top, extra, hidden, tokens, keep_scores):
+    """Logits against float64; choices and weights against the separate launch on the same logits; a padded token chooses nothing."""
+    from stride_b200.csrc import ops
+    g = torch.Generator().manual_seed(experts + hidden)
+    w = (torch.randn(experts + extra, hidden, generator=g) * 2.0 * hidden ** -0.5).bfloat16()
+    x, seq = torch.randn(tokens, hidden, generator=g).bfloat16(), [0] * tokens
+    if tokens > 1:
+        seq[tokens // 2] = -1
+    live = [t for t in range(tokens) if seq[t] == 0]
+    logits, weights = torch.zeros(tokens, experts + extra, device="cuda"), torch.full((tokens, top), 7.0, device="cuda")
+    ids = torch.full((tokens, top), -7, dtype=torch.int32, device="cuda")
+    assert ops.moe_route_rule(x.cuda(), w.cuda(), logits, None, dev(seq), ids, weights, experts, 1, 1, 1.3, group_max=True, keep_scores=keep_scores)
+    z = x.double() @ w.double().T
+    close(logits, z, 1e-5)
+    ids2, weights2 = torch.zeros_like(ids), torch.zeros_like(weights)
+    ops.moe_select_groups(logits, None, dev(seq), ids2, weights2, experts, 1, 1, 1.3, group_max=True, keep_scores=keep_scores)
+    assert torch.equal(ids, ids2) and torch.equal(weights, weights2)
+    scores = torch.sigmoid(logits[live][:, :experts].double().cpu())
+    assert all(len(set(row)) == top for row in ids[live].tolist())
+    close(scores.gather(1, ids[live].long().cpu()).sum(1), scores.sort(dim=1, descending=True).values[:, :top].sum(1), 1e-6)
+    if keep_scores:
+        close(weights[live], 1.3 * scores.gather(1, ids[live].long().cpu()), 1e-5)
+
+
 @pytest.mark.parametrize("cap", [4.0, 30.0])
 def test_a_cap_on_the_scores_is_exact(gpu, cap):
     """The tensor-core attention kernels against the exact one on the same bfloat16 inputs: scores up to several times the cap, small
