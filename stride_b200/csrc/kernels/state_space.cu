@@ -370,16 +370,22 @@ struct SsmChunkArgs {
     int vec;                    // rows of B, C and x can be read in packs of 8
 };
 
-// d_j and the running sums c_j of a chunk's tokens, by the first warp: four neighbouring tokens a lane.
-__device__ __forceinline__ void chunk_decays(const SsmChunkArgs& p, int h, size_t row0, int nt, float* s_d, float* s_c) {
+// The raw step sizes of a chunk's tokens, four neighbouring tokens a lane of the first warp; then their d_j and the running sums c_j.
+__device__ __forceinline__ void chunk_raw(const SsmChunkArgs& p, int h, size_t row0, int nt, float (&raw)[4]) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const int j = 4 * threadIdx.x + e;
+        raw[e] = threadIdx.x < 32 && j < nt ? p.raw[(row0 + j) * p.ld_raw + h] : 0.f;
+    }
+}
+__device__ __forceinline__ void chunk_decays(const SsmChunkArgs& p, int h, int nt, const float (&raw)[4], float* s_d, float* s_c) {
     if (threadIdx.x >= 32) return;
     const float rate = expf(p.a_log[h]), bias = p.dt_bias[h];
     const int lane = threadIdx.x;
     float d[4], c[4], sum = 0.f;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-        const int j = 4 * lane + e;
-        d[e] = j < nt ? softplus_f(p.raw[(row0 + j) * p.ld_raw + h] + bias) : 0.f;
+        d[e] = 4 * lane + e < nt ? softplus_f(raw[e] + bias) : 0.f;
         sum -= rate * d[e];
         c[e] = sum;
     }
@@ -472,6 +478,8 @@ ssm_chunk_sum_kernel(const SsmChunkArgs p) {
     const __nv_bfloat16* x = p.x + row0 * p.ld + h * P + col0;
     const int width = min(P - col0, kSsmCols);
     // everything the CTA reads is asked for before anything is waited for
+    float raw[4];
+    chunk_raw(p, h, row0, nt, raw);
     constexpr int PACKS = kSsmChunk * kSsmCols / 8 / kSsmThreads;
     uint4 rx[PACKS];
     if (p.vec) {
@@ -483,7 +491,7 @@ ssm_chunk_sum_kernel(const SsmChunkArgs p) {
     }
     stage_async<kSsmChunk, NP, LDN>(Bs, p.B + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
     cp_async_commit();
-    chunk_decays(p, h, row0, nt, s_d, s_c);
+    chunk_decays(p, h, nt, raw, s_d, s_c);
     __syncthreads();
     const float end = s_c[nt - 1];
     if (p.vec) {
@@ -632,6 +640,8 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
     const int width = min(P - col0, kSsmCols);
     // everything the CTA reads is asked for before anything is waited for: C and x go to shared memory by asynchronous copies, S
     // (of up to 128 rows) and B, whose place C holds at first, to registers
+    float raw[4];
+    chunk_raw(p, h, row0, nt, raw);
     stage_async<kSsmChunk, NP, LDN>(BCs, p.C + row0 * p.ld + g * N, p.ld, nt, N, p.vec);
     stage_async<kSsmChunk, kSsmCols, kLdX>(xs, p.x + row0 * p.ld + h * P + col0, p.ld, nt, width, p.vec);
     cp_async_commit();
@@ -647,6 +657,7 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
         }
     }
     const float* S = p.piece_s + (static_cast<size_t>(z) * p.H + h) * N * P + col0;
+    chunk_decays(p, h, nt, raw, s_d, s_c);
     if (P % 4 == 0) {
         constexpr int S_PACKS = NP * kSsmCols / 4 / kSsmThreads;        // 16 bytes each
         constexpr int TURN = S_PACKS < 8 ? S_PACKS : 8;
@@ -674,7 +685,6 @@ ssm_chunk_out_kernel(const SsmChunkArgs p) {
             split_bf16(r < N && c < width ? S[static_cast<size_t>(r) * P + c] : 0.f, Sh[r * kLdX + c], Sl[r * kLdX + c]);
         }
     }
-    chunk_decays(p, h, row0, nt, s_d, s_c);
     cp_async_wait<0>();
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, i0 = warp * 16;
